@@ -77,11 +77,15 @@ class ReaLMoEConfig:
 
 @dataclasses.dataclass
 class RotaryConfig:
-    """Rotation of the pairs (2i, 2i + 1) (`interleaved`) of the first `dims` dimensions of a vector by the angle pos * f_i,
-    f_i = base^(-2i / dims).  With `factor` (YaRN rescaling of a model trained on `original` positions): with
-    dim(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(dim(fast)), 0), hi = min(ceil(dim(slow)), dims - 1) and
-    ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) the frequency becomes f_i / factor * ramp_i + f_i (1 - ramp_i), and cos and
-    sin are multiplied by 0.1 ln(factor) + 1."""
+    """Rotation of the pairs (2i, 2i + 1) (`interleaved`; else (i, i + dims / 2)) of the first `dims` dimensions of a vector by the
+    angle pos * f_i, f_i = base^(-2i / dims).  With `factor` the frequencies of a model trained on `original` positions are rescaled:
+
+      * `scaling` "yarn": with dim(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(dim(fast)), 0),
+        hi = min(ceil(dim(slow)), dims - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) the frequency becomes
+        f_i / factor * ramp_i + f_i (1 - ramp_i), and cos and sin are multiplied by 0.1 ln(factor) + 1;
+      * `scaling` "llama3": n_i = original f_i / (2 pi) is the number of turns over the original length; f_i stays where
+        n_i > `fast`, becomes f_i / factor where n_i < `slow`, and (1 - s) f_i / factor + s f_i with s = (n_i - slow) / (fast - slow)
+        in between; cos and sin are not scaled."""
     dims: int
     base: float = 10000.0
     interleaved: bool = True
@@ -89,6 +93,11 @@ class RotaryConfig:
     original: int = 0
     fast: float = 32.0
     slow: float = 1.0
+    scaling: str = "yarn"          # yarn | llama3 (only with `factor`)
+
+    def __post_init__(self):
+        if self.scaling not in ("yarn", "llama3"):
+            raise ValueError("rotary scaling: yarn | llama3")
 
     def frequencies(self) -> Tuple[List[float], float]:
         """(f_i for i < dims / 2 in double precision, the factor on cos and sin)."""
@@ -97,6 +106,13 @@ class RotaryConfig:
         f = [self.base ** (-2.0 * i / self.dims) for i in range(n)]
         if self.factor is None:
             return f, 1.0
+        if self.scaling == "llama3":
+            out = []
+            for fi in f:
+                turns = self.original * fi / (2.0 * math.pi)
+                s = 1.0 if turns > self.fast else 0.0 if turns < self.slow else (turns - self.slow) / (self.fast - self.slow)
+                out.append((1.0 - s) * fi / self.factor + s * fi)
+            return out, 1.0
 
         def dim_of(turns: float) -> float:
             return self.dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
@@ -121,7 +137,9 @@ class LatentAttentionConfig:
         whole score;
       * `q_rank`: queries are the up-projection of an RMS-normalised latent of this rank (None: one projection);
       * `sink`: a learned per-head logit in the softmax denominator (no key, no value);
-      * `out_gate`: the concatenated heads are multiplied element by element by sigmoid(W_g x), x the mixer's input."""
+      * `out_gate`: the concatenated heads are multiplied element by element by sigmoid(W_g x), x the mixer's input; with
+        `head_gate` W_g has one row per head and head h's output is multiplied by sigmoid(W_g x)_h.
+    The rotation takes either pair layout."""
     n_heads: int
     qk_dim: int
     v_dim: int
@@ -134,13 +152,16 @@ class LatentAttentionConfig:
     q_rank: Optional[int] = None
     sink: bool = False
     out_gate: bool = False
+    head_gate: bool = False
 
     def __post_init__(self):
         if isinstance(self.rotary, dict):
             self.rotary = RotaryConfig(**self.rotary)
+        if self.head_gate and not self.out_gate:
+            raise ValueError("head_gate is a form of out_gate")
         if self.rot_dim:
-            if self.rotary is None or self.rotary.dims != self.rot_dim or self.rot_dim % 2 or not self.rotary.interleaved:
-                raise ValueError("rot_dim > 0 needs an interleaved `rotary` over exactly rot_dim (even) dimensions")
+            if self.rotary is None or self.rotary.dims != self.rot_dim or self.rot_dim % 2:
+                raise ValueError("rot_dim > 0 needs a `rotary` over exactly rot_dim (even) dimensions")
             if self.kv_from is not None or self.window is not None:
                 raise ValueError("the rotated form has its own latent and no window")
 
@@ -153,6 +174,11 @@ class LatentAttentionConfig:
     def cache_width(self) -> int:
         return self.kv_rank + self.rot_dim
 
+    @property
+    def gate_width(self) -> int:
+        """Output-gate logits per token (0: no gate)."""
+        return 0 if not self.out_gate else self.n_heads if self.head_gate else self.n_heads * self.v_dim
+
 
 @dataclasses.dataclass
 class WindowAttentionConfig:
@@ -164,12 +190,20 @@ class WindowAttentionConfig:
 
       * `window` / `keep_first`: query i sees key j <= i when i - j < window or j < keep_first (window None: all j <= i).  The
         cache of a sequence is then `keep_first` fixed rows plus a ring of `window` rows, whatever the sequence's length;
+      * `chunk`: query i sees key j <= i when floor(i / chunk) = floor(j / chunk), positions counted from the start of the sequence
+        (instead of a window).  The cache is a ring of `chunk` rows;
       * `value_norm`: every head's value is divided by its root mean square (no weight) before it is cached;
       * `head_temp`: a learned per-head factor on the scaled score;
       * `slope_base` b: the score loses slope_h * (i - j), slope_h = 2^(-b (h + 1) / n_heads) (None: no distance term);
       * `sink`: a learned per-head logit added to the softmax denominator as exp(sink_h): a key-less, value-less entry;
-      * `out_gate`: head h's output is multiplied by sigmoid(w_g . x)_h, x being the mixer's input;
-      * `qk_norm`: every query / key head is RMS-normalised over qk_dim with a weight (one for queries, one for keys);
+      * `sink_const`: a fixed sink logit instead of the learned ones (0: one is added to the denominator);
+      * `softcap` c: the scaled score becomes c tanh(score / c) (not together with a distance term);
+      * `out_gate`: head h's output is multiplied by sigmoid(w_g . x)_h, x being the mixer's input; with `element_gate` W_g has a row
+        per output element (n_heads * v_dim) and the concatenated heads are multiplied element by element;
+      * `qk_norm`: every query / key head is RMS-normalised over qk_dim with a weight (one for queries, one for keys); with
+        `full_norm` all query heads (all key heads) of a token are one vector with one root mean square, the weights span them;
+      * `value_rotary`: value heads are rotated by their position too (and cached rotated), and every head's output is turned back by
+        the query's position before the gate: the output then depends on distances only;
       * `n_maps` = 2: differential attention.  Queries and keys have two maps per head ([map 1 | map 2], 2 qk_dim wide), each a
         softmax attention of its own over the same values; with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + `diff` (learned vectors
         of size qk_dim, one number per layer) head h's output is o = a1 - lambda a2, then o / sqrt(mean(o^2) + eps) * (1 - diff)."""
@@ -190,10 +224,33 @@ class WindowAttentionConfig:
     n_maps: int = 1
     diff: float = 0.0
     rotary: Optional[RotaryConfig] = None
+    chunk: Optional[int] = None
+    softcap: Optional[float] = None
+    sink_const: Optional[float] = None
+    element_gate: bool = False
+    full_norm: bool = False
+    value_rotary: Optional[RotaryConfig] = None
 
     def __post_init__(self):
         if isinstance(self.rotary, dict):
             self.rotary = RotaryConfig(**self.rotary)
+        if isinstance(self.value_rotary, dict):
+            self.value_rotary = RotaryConfig(**self.value_rotary)
+        vr = self.value_rotary
+        if vr is not None and (vr.dims % 2 or not 0 < vr.dims <= self.v_dim or vr.frequencies()[1] != 1.0):
+            raise ValueError("value_rotary.dims: even, at most v_dim; no factor on cos and sin")
+        if self.chunk is not None and (self.chunk < 1 or self.window is not None or self.keep_first):
+            raise ValueError("chunk >= 1, and instead of a window")
+        if self.softcap is not None and (self.softcap <= 0 or self.slope_base is not None):
+            raise ValueError("softcap > 0, without a distance term")
+        if self.sink_const is not None and self.sink:
+            raise ValueError("sink_const replaces the learned sink")
+        if (self.element_gate and not self.out_gate) or (self.full_norm and not self.qk_norm):
+            raise ValueError("element_gate is a form of out_gate, full_norm of qk_norm")
+        if self.n_maps == 1 and self.qk_norm and not self.full_norm:
+            raise ValueError("plain attention normalises the whole query / key projection (full_norm)")
+        if self.n_maps == 2 and (self.chunk or self.softcap or self.sink_const is not None or self.full_norm or self.value_rotary):
+            raise ValueError("differential attention combines with qk_norm and the window only")
         if self.rotary is not None and (self.rotary.dims % 2 or not 0 < self.rotary.dims <= self.qk_dim or self.n_maps != 1):
             raise ValueError("rotary.dims: even, at most qk_dim, one score map")
         if self.n_heads % self.n_kv_heads:
@@ -210,7 +267,19 @@ class WindowAttentionConfig:
     def cache_rows(self, max_len: int) -> int:
         """Rows a sequence of at most max_len tokens needs: position p lives in row p when p < keep_first, else in row
         keep_first + (p - keep_first) % (rows - keep_first)."""
+        if self.chunk is not None:
+            return max(1, min(max_len, self.chunk))
         return max_len if self.window is None else max(1, min(max_len, self.keep_first + self.window))
+
+    @property
+    def gate_width(self) -> int:
+        """Output-gate logits per token (0: no gate)."""
+        return 0 if not self.out_gate else self.n_heads * self.v_dim if self.element_gate else self.n_heads
+
+    @property
+    def prepared(self) -> bool:
+        """Query / key norm, rotations and cache rows of a token are one kernel (`ops.attention.window_prepare_`)."""
+        return self.n_maps == 1 and (self.full_norm or self.value_rotary is not None or (self.rotary is not None and not self.value_norm))
 
 
 @dataclasses.dataclass
@@ -407,7 +476,16 @@ class ReaLModelConfig:
     embed_scale: Optional[float] = None  # the embedding output is multiplied by this constant
     residual_mult: float = 1.0           # x <- x + residual_mult * branch ("layer" stacks)
     layer_scale: bool = False            # every branch output (after its output norm) times a learned vector (`attn.ls.weight`,
-                                         # `mlp.ls.weight`) before it joins the stream ("layer" stacks)
+                                         # `mlp.ls.weight`) before it joins the stream (wrapped stacks, see `wrapped`)
+    scalar_norm: bool = False            # the sublayers' norms and the final one have ONE learned factor instead of a vector (RMSNorm)
+    gated_residual: bool = False         # every branch output is multiplied element by element by sigmoid(W h + b), h the sublayer's
+                                         # input, before its output norm (`sharding.residual_gate_fused`: where W lives)
+
+    @property
+    def wrapped(self) -> bool:
+        """Every sublayer is x <- x + residual_mult * ls * N_post(gate * branch(N(x))) with at least one mechanism beyond the two norms:
+        the stack's branch outputs travel to the kernel that forms the next norm (`models.hetero_block.PendingBranch`)."""
+        return self.layer_norm_type == "layer" or self.scalar_norm or self.gated_residual or self.layer_scale
 
     def layer_runs(self) -> List[Tuple[int, bool]]:
         """(1-based block index, the run starts a pass of the loop) for every block run, in execution order."""
@@ -435,16 +513,19 @@ class ReaLModelConfig:
             self.blocks = [BlockConfig(**b) if isinstance(b, dict) else b for b in self.blocks]
             if len(self.blocks) != self.n_layers:
                 raise ValueError("`blocks` must describe every layer")
-            if self.layer_norm_type == "layer" and (self.norm_groups != 1 or self.conv_taps or not self.sandwich_norm):
-                raise ValueError("\"layer\" stacks: one norm group, no convolution, norms on both sides of every sublayer")
-            if self.layer_norm_type != "layer" and (self.layer_scale or self.residual_mult != 1.0
-                                                    or any(b.mixer in ("decay", "parallel") for b in self.blocks)):
-                raise ValueError("layer_scale, residual_mult and the decay / parallel mixers live in \"layer\" stacks")
+            if self.wrapped and (self.norm_groups != 1 or self.conv_taps or not self.sandwich_norm or self.layer_norm_type not in ("layer", "rms")):
+                raise ValueError("wrapped stacks: one norm group, no convolution, norms (\"layer\" or \"rms\") on both sides of every sublayer")
+            if not self.wrapped and (self.residual_mult != 1.0 or any(b.mixer in ("decay", "parallel") for b in self.blocks)):
+                raise ValueError("residual_mult and the decay / parallel mixers live in wrapped stacks")
+            if self.scalar_norm and self.layer_norm_type != "rms":
+                raise ValueError("scalar_norm is a form of RMSNorm")
             for i, b in enumerate(self.blocks):
                 if b.mixer != "latent_attention":
                     continue
-                if b.attn.rotated and (self.norm_groups != 1 or self.sandwich_norm or self.conv_taps):
-                    raise ValueError("rotated latent attention lives in plain pre-norm stacks")
+                if b.attn.rotated and not self.wrapped and (self.norm_groups != 1 or self.sandwich_norm or self.conv_taps):
+                    raise ValueError("rotated latent attention lives in plain pre-norm and in wrapped stacks")
+                if self.wrapped and not b.attn.rotated:
+                    raise ValueError("wrapped stacks take latent attention in its rotated form")
                 src = b.attn.kv_from
                 if src is not None and not (0 <= src < i and self.blocks[src].attn.kv_from is None
                                             and self.blocks[src].attn.kv_rank == b.attn.kv_rank):
@@ -458,8 +539,12 @@ class ReaLModelConfig:
         """Parameter count (used by the PP partitioner, the FLOP model and the allocation search)."""
         h, f, v = self.hidden_dim, self.intermediate_dim, self.vocab_size
         if self.blocks is not None:
-            n = 2 * v * h + h
-            norms = (2 if self.sandwich_norm else 1) + self.conv_taps + int(self.layer_scale)   # per sublayer: norm(s), taps, scale
+            n = 2 * v * h + (1 if self.scalar_norm else h)
+            # per sublayer, in units of h: norm(s), taps, scale, residual gate (a matrix and a bias)
+            norms = (2 if self.sandwich_norm else 1) + self.conv_taps + int(self.layer_scale) + (h + 1 if self.gated_residual else 0)
+            if self.scalar_norm:
+                norms -= 2
+                n += 2 * (len(self.blocks) + sum(b.mlp is not None for b in self.blocks))
             for b in self.blocks:
                 if b.mixer in ("decay", "parallel"):
                     a = b.decay
@@ -471,9 +556,9 @@ class ReaLModelConfig:
                     a = b.wattn
                     qkv = a.n_heads * a.qk_dim + a.n_kv_heads * (a.qk_dim + a.v_dim)
                     qkv += (a.n_maps - 1) * (a.n_heads + a.n_kv_heads) * a.qk_dim
-                    n += h * (qkv + (a.n_heads if a.out_gate else 0)) + (qkv if a.qkv_bias else 0) + a.n_heads * a.v_dim * h
+                    n += h * (qkv + a.gate_width) + (qkv if a.qkv_bias else 0) + a.n_heads * a.v_dim * h
                     n += a.n_heads * (int(a.head_temp) + int(a.sink)) + norms * h
-                    n += (2 * a.qk_dim if a.qk_norm else 0) + (4 * a.qk_dim if a.n_maps == 2 else 0)
+                    n += ((a.n_heads + a.n_kv_heads if a.full_norm else 2) * a.qk_dim if a.qk_norm else 0) + (4 * a.qk_dim if a.n_maps == 2 else 0)
                 elif b.mixer == "delta":
                     a = b.delta
                     n += h * (2 * a.n_kv_heads * a.qk_dim + 2 * a.n_heads * a.v_dim + 2 * a.n_heads) + a.n_heads * a.v_dim * h
@@ -487,7 +572,7 @@ class ReaLModelConfig:
                     dq = a.qk_dim + a.rot_dim
                     n += (h * a.q_rank + a.q_rank + a.q_rank * a.n_heads * dq) if a.q_rank else h * a.n_heads * dq
                     n += h * a.cache_width + a.kv_rank + a.kv_rank * a.n_heads * (a.qk_dim + a.v_dim) + a.n_heads * a.v_dim * h
-                    n += (a.n_heads if a.sink else 0) + (h * a.n_heads * a.v_dim if a.out_gate else 0) + norms * h
+                    n += (a.n_heads if a.sink else 0) + h * a.gate_width + norms * h
                 else:
                     a = b.attn
                     n += h * a.n_heads * a.qk_dim + (h * a.kv_rank + a.kv_rank if a.kv_from is None else 0)

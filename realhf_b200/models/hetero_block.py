@@ -10,7 +10,8 @@ per run (`state.k[r]`, `state.v[r]`), by mixer:
     `kv_from = j` holds the SAME tensor as block j), `v[r]` the convolution state [2, n_slots, taps - 1, hidden] fp32 (the normalised
     inputs of the last taps - 1 tokens of the mixer [0] and the feed-forward [1]);
   * window attention: `k[r]` keys [n_slots, G, rows, d], `v[r]` normalised values [n_slots, G, rows, dv] (model dtype); position p
-    in row p below `keep_first`, else in a ring of the remaining rows (`WindowAttentionConfig.cache_rows`);
+    in row p below `keep_first`, else in a ring of the remaining rows (`WindowAttentionConfig.cache_rows`; chunked attention: a ring
+    of `chunk` rows); keys, and with `value_rotary` values, are cached rotated;
   * delta rule: `k[r]` the matrix states [n_slots, H, d, dv] fp32, `v[r]` the last taps - 1 projection outputs
     [n_slots, taps - 1, C] fp32;
   * differential window attention (`n_maps` = 2): `k[r]` [n_slots, 2G, rows, d] (both maps' keys), `v[r]` [n_slots, G, rows, dv];
@@ -21,9 +22,10 @@ per run (`state.k[r]`, `state.v[r]`), by mixer:
   * `parallel` (window attention beside decayed linear attention): `k[r]`, `v[r]` the rotated keys / values as for window
     attention, and a third tensor `state.m[r]` with the matrix states [n_slots, H, d, dv] fp32 (`m[r]` is None for other mixers).
 
-A stack with `layer_norm_type == "layer"` runs  x <- x + mult * ls * LN_post(mixer(LN(x)))  and the same for the feed-forward, LN
-being the bias-free LayerNorm; the add, the branch's output norm and the next sublayer's input norm are one kernel
-(`ops.functional.residual_add_centred_norm_`).
+A wrapped stack (`ReaLModelConfig.wrapped`) runs  x <- x + mult * ls * N_post(sigmoid(W h + b) * mixer(h)), h = N(x),  and the same
+for the feed-forward, N being the bias-free LayerNorm (`layer_norm_type` "layer") or RMSNorm ("rms"; `scalar_norm`: with one factor
+for all coordinates); mult, ls and the sigmoid gate are optional.  The gate, the output norm, the add and the next sublayer's input
+norm are one kernel (`ops.functional.residual_add_centred_norm_`); the gate's logits come out of the projection that reads h anyway.
 
 Inference only (no autograd through these kernels) and not tensor-parallel.  A stack with a loop runs on one pipeline stage.
 """
@@ -35,6 +37,7 @@ from typing import Dict, List, Optional
 
 import torch
 
+from realhf_b200.models.sharding import latent_rope_sections, residual_gate_fused
 from realhf_b200.ops import attention as attn_ops
 from realhf_b200.ops import functional as OF
 from realhf_b200.ops import recurrent as rec_ops
@@ -72,6 +75,31 @@ def packed_meta(cu_seqlens: torch.Tensor, total: int, slots: Optional[torch.Tens
                       m=getattr(state, "m", None) if state is not None else None)
 
 
+@dataclasses.dataclass
+class BranchOut:
+    """What a sublayer of a wrapped stack hands to its output norm: y, or a y + b y2 (`branch_scales`), times sigmoid(gate)."""
+    y: torch.Tensor
+    y2: Optional[torch.Tensor] = None
+    gate: Optional[torch.Tensor] = None
+
+
+def _with_residual_gate(model, i: int, y: torch.Tensor, proj: torch.Tensor):
+    """y with the residual gate's logits, the last section of the mixer's fused input projection (where the stack has the gate)."""
+    c = model.config
+    return BranchOut(y, gate=proj[:, proj.shape[1] - c.hidden_dim:]) if residual_gate_fused(c, i)[0] else y
+
+
+def _mlp_branch(model, i: int, h: torch.Tensor, mcfg) -> BranchOut:
+    """Feed-forward of a wrapped stack, with the residual gate's logits: fused into the up-projection of a relu2 unit."""
+    c, p = model.config, model.p
+    if residual_gate_fused(c, i)[1]:
+        w = p[f"{i}.mlp.up_rg.weight"]
+        u = OF.relu2_linear(h, w, p[f"{i}.mlp.up_rg.bias"], act_cols=w.shape[0] - c.hidden_dim)
+        return BranchOut(OF.linear(u[:, :mcfg.ff], p[f"{i}.mlp.down.weight"]), gate=u[:, w.shape[0] - c.hidden_dim:])
+    gate = OF.linear(h, p[f"{i}.mlp.rg.weight"], p[f"{i}.mlp.rg.bias"]) if c.gated_residual else None
+    return BranchOut(_mlp(model, i, h, mcfg), gate=gate)
+
+
 def _mlp(model, i: int, h: torch.Tensor, mcfg) -> torch.Tensor:
     p = model.p
     if mcfg.kind == "moe":
@@ -95,13 +123,19 @@ def _window_attention_packed(model, i: int, li: int, h: torch.Tensor, meta: Pack
                                            c.layer_norm_epsilon, meta.k[li] if keep else None, meta.v[li] if keep else None, meta.tok_slot,
                                            meta.pos, meta.remain, meta.cu_seqlens, meta.max_seqlen)
         return OF.linear(o, p[f"{i}.attn.o.weight"])
-    if a.rotary is not None:
-        attn_ops.rotate_qk_(qkvg, a, pos=meta.pos)
-    v_n = attn_ops.value_norm_store(qkvg, a, c.layer_norm_epsilon, meta.k[li] if keep else None, meta.v[li] if keep else None,
-                                    meta.tok_slot, meta.pos, meta.remain)
+    if a.prepared:
+        attn_ops.window_prepare_(qkvg, a, p.get(f"{i}.attn.q_norm.weight"), p.get(f"{i}.attn.k_norm.weight"), c.layer_norm_epsilon, pos=meta.pos,
+                                 k_cache=meta.k[li] if keep else None, v_cache=meta.v[li] if keep else None, tok_slot=meta.tok_slot,
+                                 remain=meta.remain)
+        v_n = attn_ops.window_values(qkvg, a)
+    else:
+        if a.rotary is not None:
+            attn_ops.rotate_qk_(qkvg, a, pos=meta.pos)
+        v_n = attn_ops.value_norm_store(qkvg, a, c.layer_norm_epsilon, meta.k[li] if keep else None, meta.v[li] if keep else None,
+                                        meta.tok_slot, meta.pos, meta.remain)
     o = attn_ops.sink_window_attention(qkvg, v_n, a, p.get(f"{i}.attn.temp.weight"), p.get(f"{i}.attn.sink.weight"), meta.pos,
                                        meta.cu_seqlens, meta.max_seqlen)
-    return OF.linear(o, p[f"{i}.attn.o.weight"])
+    return _with_residual_gate(model, i, OF.linear(o, p[f"{i}.attn.o.weight"]), qkvg)
 
 
 def _window_attention_decode(model, i: int, li: int, h: torch.Tensor, k_caches, v_caches, cache_lens, slots) -> torch.Tensor:
@@ -112,11 +146,14 @@ def _window_attention_decode(model, i: int, li: int, h: torch.Tensor, k_caches, 
         o = attn_ops.diff_window_decode_attention(qkvg, a, p[f"{i}.attn.q_norm.weight"], p[f"{i}.attn.k_norm.weight"], p[f"{i}.attn.lambda.weight"],
                                                   c.layer_norm_epsilon, k_caches[li], v_caches[li], cache_lens, slots)
         return OF.linear(o, p[f"{i}.attn.o.weight"])
-    if a.rotary is not None:
+    if a.prepared:
+        attn_ops.window_prepare_(qkvg, a, p.get(f"{i}.attn.q_norm.weight"), p.get(f"{i}.attn.k_norm.weight"), c.layer_norm_epsilon,
+                                 cache_lens=cache_lens, slots=slots)
+    elif a.rotary is not None:
         attn_ops.rotate_qk_(qkvg, a, cache_lens=cache_lens, slots=slots)
     o = attn_ops.sink_window_decode_attention(qkvg, a, p.get(f"{i}.attn.temp.weight"), p.get(f"{i}.attn.sink.weight"), k_caches[li],
                                               v_caches[li], cache_lens, slots, c.layer_norm_epsilon)
-    return OF.linear(o, p[f"{i}.attn.o.weight"])
+    return _with_residual_gate(model, i, OF.linear(o, p[f"{i}.attn.o.weight"]), qkvg)
 
 
 def _delta_packed(model, i: int, li: int, h: torch.Tensor, meta: PackedMeta) -> torch.Tensor:
@@ -174,39 +211,39 @@ def _latent_rope_queries(model, i: int, a, proj: torch.Tensor, cq: Optional[torc
     """[rows, H (d + rot)] queries, not yet rotated: the up-projection of the normalised query latent, or a section of `proj`."""
     if a.q_rank:
         return OF.linear(cq, model.p[f"{i}.attn.uq.weight"])
-    q0 = a.cache_width + (a.n_heads * a.v_dim if a.out_gate else 0)
+    q0 = sum(latent_rope_sections(a)[:-1])
     return proj[:, q0:q0 + a.n_heads * (a.qk_dim + a.rot_dim)]
 
 
-def _latent_rope_gate(a, o: torch.Tensor, proj: torch.Tensor) -> torch.Tensor:
-    if a.out_gate:
-        g0 = (a.q_rank or 0) + a.cache_width
-        attn_ops.sigmoid_gate_(o, proj[:, g0:g0 + a.n_heads * a.v_dim])
-    return o
+def _latent_rope_gate(a, proj: torch.Tensor) -> Optional[torch.Tensor]:
+    g0 = (a.q_rank or 0) + a.cache_width
+    return proj[:, g0:g0 + a.gate_width] if a.out_gate else None
 
 
-def _latent_rope_packed(model, i: int, li: int, h: torch.Tensor, meta: PackedMeta) -> torch.Tensor:
+def _latent_rope_packed(model, i: int, li: int, h: torch.Tensor, meta: PackedMeta):
     c, p = model.config, model.p
     a = c.blocks[i - 1].attn
     keep = meta.k is not None
-    proj = OF.linear(h, p[f"{i}.attn.in.weight"])
+    proj = OF.linear(h, p[f"{i}.attn.in.weight"], p.get(f"{i}.attn.in.bias"))
     cq, lat = attn_ops.latent_rope_prepare(proj, a, p.get(f"{i}.attn.q_ln.weight"), p[f"{i}.attn.dkv_ln.weight"], c.layer_norm_epsilon, meta.pos,
                                            meta.k[li] if keep else None, meta.tok_slot, meta.remain)
     q = _latent_rope_queries(model, i, a, proj, cq)
     kv = OF.linear(lat[:, : a.kv_rank], p[f"{i}.attn.ukv.weight"])
-    o = attn_ops.latent_rope_attention(q, kv, lat, a, p.get(f"{i}.attn.sink.weight"), meta.pos, meta.cu_seqlens, meta.max_seqlen)
-    return OF.linear(_latent_rope_gate(a, o, proj), p[f"{i}.attn.o.weight"])
+    o = attn_ops.latent_rope_attention(q, kv, lat, a, p.get(f"{i}.attn.sink.weight"), meta.pos, meta.cu_seqlens, meta.max_seqlen,
+                                       gate=_latent_rope_gate(a, proj))
+    return _with_residual_gate(model, i, OF.linear(o, p[f"{i}.attn.o.weight"]), proj)
 
 
-def _latent_rope_decode(model, i: int, li: int, h: torch.Tensor, k_caches, cache_lens, slots) -> torch.Tensor:
+def _latent_rope_decode(model, i: int, li: int, h: torch.Tensor, k_caches, cache_lens, slots):
     c, p = model.config, model.p
     a = c.blocks[i - 1].attn
-    proj = OF.linear(h, p[f"{i}.attn.in.weight"])
+    proj = OF.linear(h, p[f"{i}.attn.in.weight"], p.get(f"{i}.attn.in.bias"))
     cq, _ = attn_ops.latent_rope_prepare(proj, a, p.get(f"{i}.attn.q_ln.weight"), p[f"{i}.attn.dkv_ln.weight"], c.layer_norm_epsilon, None,
                                          k_caches[li], cache_lens=cache_lens, slots=slots, want_lat=False)
     q = _latent_rope_queries(model, i, a, proj, cq)
-    o = attn_ops.latent_rope_decode_attention(q, a, p[f"{i}.attn.ukv.weight"], p.get(f"{i}.attn.sink.weight"), k_caches[li], cache_lens, slots)
-    return OF.linear(_latent_rope_gate(a, o, proj), p[f"{i}.attn.o.weight"])
+    o = attn_ops.latent_rope_decode_attention(q, a, p[f"{i}.attn.ukv.weight"], p.get(f"{i}.attn.sink.weight"), k_caches[li], cache_lens, slots,
+                                              gate=_latent_rope_gate(a, proj))
+    return _with_residual_gate(model, i, OF.linear(o, p[f"{i}.attn.o.weight"]), proj)
 
 
 def _decay_branch(model, i: int, d, proj: torch.Tensor, o: torch.Tensor) -> torch.Tensor:
@@ -242,7 +279,7 @@ def _parallel_split(b, proj: torch.Tensor):
 
 
 def _parallel_packed(model, i: int, li: int, h: torch.Tensor, meta: PackedMeta):
-    """Both branches of a `parallel` block on the packed batch -> (left output, right output), each after its own projection."""
+    """Both branches of a `parallel` block on the packed batch, each after its own output projection."""
     c, p = model.config, model.p
     b = c.blocks[i - 1]
     w, d = b.wattn, b.decay
@@ -256,7 +293,7 @@ def _parallel_packed(model, i: int, li: int, h: torch.Tensor, meta: PackedMeta):
     y_l = OF.linear(o, p[f"{i}.attn.o.weight"])
     s = rec_ops.decay_scan(rec_ops.decay_prepare(right, d, pos=meta.pos), d, meta.cu_seqlens, meta.m[li] if keep else None,
                            meta.seq_slot if keep else None)
-    return y_l, OF.linear(_decay_branch(model, i, d, right, s), p[f"{i}.attn.o2.weight"])
+    return BranchOut(y_l, OF.linear(_decay_branch(model, i, d, right, s), p[f"{i}.attn.o2.weight"]))
 
 
 def _parallel_decode(model, i: int, li: int, h: torch.Tensor, k_caches, v_caches, m_caches, cache_lens, slots):
@@ -269,49 +306,55 @@ def _parallel_decode(model, i: int, li: int, h: torch.Tensor, k_caches, v_caches
     o = attn_ops.sink_window_decode_attention(left, w, None, None, k_caches[li], v_caches[li], cache_lens, slots, c.layer_norm_epsilon)
     y_l = OF.linear(o, p[f"{i}.attn.o.weight"])
     s = rec_ops.decay_step(rec_ops.decay_prepare(right, d, cache_lens=cache_lens, slots=slots), d, m_caches[li], slots)
-    return y_l, OF.linear(_decay_branch(model, i, d, right, s), p[f"{i}.attn.o2.weight"])
+    return BranchOut(y_l, OF.linear(_decay_branch(model, i, d, right, s), p[f"{i}.attn.o2.weight"]))
 
 
 @dataclasses.dataclass
 class PendingBranch:
-    """A branch output of a "layer" stack that is still owed to the stream: x += mult * scale * LN(a y + b y2) * w.  The kernel that
-    computes the next norm (the next block's, the final one) adds it on the way."""
-    y: torch.Tensor
+    """A branch output of a wrapped stack that is still owed to the stream: x += mult * scale * N((a y + b y2) * sigmoid(gate)) * w.  The
+    kernel that computes the next norm (the next block's, the final one) adds it on the way."""
+    out: BranchOut
     w: torch.Tensor
     scale: Optional[torch.Tensor]
-    y2: Optional[torch.Tensor] = None
     a: float = 1.0
     b: float = 1.0
 
 
+def _rms(c) -> bool:
+    return c.layer_norm_type != "layer"
+
+
 def _add_pending(model, x: torch.Tensor, pb: PendingBranch, next_w: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     c = model.config
-    return OF.residual_add_centred_norm_(x, pb.y, pb.w, c.layer_norm_epsilon, pb.scale, c.residual_mult, pb.y2, pb.a, pb.b, next_w, model.dtype)
+    return OF.residual_add_centred_norm_(x, pb.out.y, pb.w, c.layer_norm_epsilon, pb.scale, c.residual_mult, pb.out.y2, pb.a, pb.b, next_w,
+                                         model.dtype, _rms(c), pb.out.gate)
 
 
-def _finish_layer_block(model, i: int, b, x: torch.Tensor, y, defer: bool = False) -> Optional[PendingBranch]:
-    """"layer" stacks: x += mult * ls * LN_post(mixer output), then the feed-forward sublayer likewise.  `y` is the mixer's output,
-    or the pair of branch outputs of a `parallel` block (summed with `branch_scales` inside the norm kernel).  With `defer` the
-    block's last branch is returned instead of added."""
-    p = model.p
-    y, y2 = y if isinstance(y, tuple) else (y, None)
-    sa, sb = b.branch_scales if y2 is not None else (1.0, 1.0)
-    pb = PendingBranch(y, p[f"{i}.attn.ln_post.weight"], p.get(f"{i}.attn.ls.weight"), y2, sa, sb)
+def _finish_wrapped_block(model, i: int, b, x: torch.Tensor, h: torch.Tensor, y, defer: bool = False) -> Optional[PendingBranch]:
+    """Wrapped stacks: x += mult * ls * N_post(gated mixer output), then the feed-forward sublayer likewise.  `y` is what the mixer made
+    of h: its output, or a `BranchOut` (two outputs of a `parallel` block, summed with `branch_scales` inside the norm kernel; the
+    residual gate's logits).  With `defer` the block's last branch is returned instead of added."""
+    c, p = model.config, model.p
+    out = y if isinstance(y, BranchOut) else BranchOut(y)
+    if c.gated_residual and out.gate is None:
+        out.gate = OF.linear(h, p[f"{i}.attn.rg.weight"], p[f"{i}.attn.rg.bias"])
+    sa, sb = b.branch_scales if out.y2 is not None else (1.0, 1.0)
+    pb = PendingBranch(out, p[f"{i}.attn.ln_post.weight"], p.get(f"{i}.attn.ls.weight"), sa, sb)
     if b.mlp is not None:
         h = _add_pending(model, x, pb, p[f"{i}.mlp.ln.weight"])
-        pb = PendingBranch(_mlp(model, i, h, b.mlp), p[f"{i}.mlp.ln_post.weight"], p.get(f"{i}.mlp.ls.weight"))
+        pb = PendingBranch(_mlp_branch(model, i, h, b.mlp), p[f"{i}.mlp.ln_post.weight"], p.get(f"{i}.mlp.ls.weight"))
     if defer:
         return pb
     _add_pending(model, x, pb)
     return None
 
 
-def _first_layer_norm(model, i: int, x: torch.Tensor, pending) -> torch.Tensor:
-    """Input of block i's mixer in a "layer" stack; a branch the previous block left pending is added by the same kernel."""
+def _first_wrapped_norm(model, i: int, x: torch.Tensor, pending) -> torch.Tensor:
+    """Input of block i's mixer in a wrapped stack; a branch the previous block left pending is added by the same kernel."""
     w = model.p[f"{i}.attn.ln.weight"]
     if isinstance(pending, PendingBranch):
         return _add_pending(model, x, pending, w)
-    return OF.centred_norm(settle(model, x, pending), w, model.config.layer_norm_epsilon, model.dtype)
+    return OF.centred_norm(settle(model, x, pending), w, model.config.layer_norm_epsilon, model.dtype, _rms(model.config))
 
 
 def norm_offset(c) -> float:
@@ -331,7 +374,7 @@ def loop_inject(model, i: int, x: torch.Tensor, x0: torch.Tensor) -> torch.Tenso
 
 def plain_prenorm(c) -> bool:
     """One RMSNorm per sublayer and nothing else around it: a sublayer's residual add can wait for the next norm kernel."""
-    return c.norm_groups == 1 and not c.sandwich_norm and not c.conv_taps
+    return not c.wrapped and c.norm_groups == 1 and not c.sandwich_norm and not c.conv_taps
 
 
 def first_norm(model, i: int, x: torch.Tensor, pending: Optional[torch.Tensor]) -> torch.Tensor:
@@ -386,11 +429,11 @@ def block_packed(model, i: int, li: int, x: torch.Tensor, meta: PackedMeta, pend
     a = b.attn
     G, eps = c.norm_groups, c.layer_norm_epsilon
     keep = meta.k is not None
-    if c.layer_norm_type == "layer":
-        h = _first_layer_norm(model, i, x, pending)
+    if c.wrapped:
+        h = _first_wrapped_norm(model, i, x, pending)
         mixer = {"window_attention": _window_attention_packed, "delta": _delta_packed, "mlstm": _mlstm_packed, "latent_attention": _latent_rope_packed,
                  "decay": _decay_packed, "parallel": _parallel_packed}[b.mixer]
-        return x, _finish_layer_block(model, i, b, x, mixer(model, i, li, h, meta), defer)
+        return x, _finish_wrapped_block(model, i, b, x, h, mixer(model, i, li, h, meta), defer)
     if b.mixer != "latent_attention" or a.rotated:
         defer = defer and plain_prenorm(c)
         h = first_norm(model, i, x, pending) if plain_prenorm(c) else OF.sublayer_input(settle(model, x, pending), p[f"{i}.attn.ln.weight"], G, eps,
@@ -444,9 +487,9 @@ def block_decode(model, i: int, li: int, x: torch.Tensor, k_caches: List[torch.T
     b = c.blocks[i - 1]
     a = b.attn
     G, eps = c.norm_groups, c.layer_norm_epsilon
-    if c.layer_norm_type == "layer":
-        h = _first_layer_norm(model, i, x, pending)
-        return x, _finish_layer_block(model, i, b, x, _mixer_decode(model, b, i, li, h, k_caches, v_caches, m_caches, cache_lens, slots), defer)
+    if c.wrapped:
+        h = _first_wrapped_norm(model, i, x, pending)
+        return x, _finish_wrapped_block(model, i, b, x, h, _mixer_decode(model, b, i, li, h, k_caches, v_caches, m_caches, cache_lens, slots), defer)
     if b.mixer != "latent_attention" or a.rotated:
         defer = defer and plain_prenorm(c)
         h = first_norm(model, i, x, pending) if plain_prenorm(c) else OF.sublayer_input_step(settle(model, x, pending), p[f"{i}.attn.ln.weight"], G,
@@ -472,10 +515,10 @@ def block_decode(model, i: int, li: int, x: torch.Tensor, k_caches: List[torch.T
 def final_norm(model, x: torch.Tensor, pending: Optional[torch.Tensor] = None) -> torch.Tensor:
     c = model.config
     w = model.p[f"{c.n_layers}.ln_f.weight"]
-    if c.layer_norm_type == "layer":
+    if c.wrapped:
         if isinstance(pending, PendingBranch):
             return _add_pending(model, x, pending, w)
-        return OF.centred_norm(x, w, c.layer_norm_epsilon, model.dtype)
+        return OF.centred_norm(x, w, c.layer_norm_epsilon, model.dtype, _rms(c))
     if pending is not None and plain_prenorm(c):
         return OF.add_rms_norm_(x, pending, w, c.layer_norm_epsilon, model.dtype, norm_offset(c))
     return OF.sublayer_input(settle(model, x, pending), w, c.norm_groups, c.layer_norm_epsilon, None, None, model.dtype, w_offset=norm_offset(c))

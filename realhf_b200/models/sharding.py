@@ -100,10 +100,28 @@ def _pad8(n: int) -> int:
 
 def wattn_sections(w) -> Tuple[int, ...]:
     """Rows of the fused input projection of a window-attention block: [queries | keys | values | output-gate logits].  The gate
-    section (one row per head) is padded to a multiple of 8 rows so that the fused tensor keeps 16-byte row groups; the padding
-    rows are never read."""
+    section (one row per head, or per output element) is padded so that it ends at a multiple of 8 rows counted from its own start
+    (per head) or from the tensor's (per element): what follows it starts on a 16-byte boundary; the padding rows are never read."""
     sec = (w.n_heads * w.n_maps * w.qk_dim, w.n_kv_heads * w.n_maps * w.qk_dim, w.n_kv_heads * w.v_dim)   # n_maps = 2: two score maps per head
-    return sec + ((_pad8(w.n_heads),) if w.out_gate else ())
+    if not w.out_gate:
+        return sec
+    return sec + ((_pad8(sum(sec) + w.gate_width) - sum(sec),) if w.element_gate else (_pad8(w.n_heads),))
+
+
+def residual_gate_fused(cfg: ReaLModelConfig, layer_idx: int) -> Tuple[bool, bool]:
+    """Whether the residual gate's rows (`cfg.gated_residual`) are the last section of the projection that reads the same input: of
+    the mixer's fused input projection (window attention, rotated latent attention), of the feed-forward's up-projection
+    (`mlp.up_rg`, kind relu2).  Elsewhere they are tensors of their own (`attn.rg` / `mlp.rg`)."""
+    b = cfg.blocks[layer_idx - 1]
+    mixer = (b.mixer == "window_attention" and b.wattn.n_maps == 1) or (b.mixer == "latent_attention" and b.attn.rotated)
+    return cfg.gated_residual and mixer, cfg.gated_residual and b.mlp is not None and b.mlp.kind == "relu2"
+
+
+def in_sections(cfg: ReaLModelConfig, layer_idx: int) -> Tuple[int, ...]:
+    """Sections of the fused input projection of a window-attention or rotated latent-attention block, the residual gate's last."""
+    b = cfg.blocks[layer_idx - 1]
+    sec = wattn_sections(b.wattn) if b.mixer == "window_attention" else latent_rope_sections(b.attn)
+    return sec + ((cfg.hidden_dim,) if residual_gate_fused(cfg, layer_idx)[0] else ())
 
 
 def mlstm_sections(m) -> Tuple[int, ...]:
@@ -116,8 +134,8 @@ def latent_rope_sections(a) -> Tuple[int, ...]:
     """Rows of the fused input projection of a rotated latent-attention block: [query latent | latent, rotated key part | gate
     logits | queries].  The first section exists with `q_rank`, the third with `out_gate`, the last without `q_rank`."""
     dq = a.qk_dim + a.rot_dim
-    return (((a.q_rank,) if a.q_rank else ()) + (a.kv_rank + a.rot_dim,) + ((a.n_heads * a.v_dim,) if a.out_gate else ())
-            + (() if a.q_rank else (a.n_heads * dq,)))
+    return (((a.q_rank,) if a.q_rank else ()) + (a.kv_rank + a.rot_dim,)
+            + ((_pad8(a.n_heads) if a.head_gate else a.gate_width,) if a.out_gate else ()) + (() if a.q_rank else (a.n_heads * dq,)))
 
 
 def delta_sections(d) -> Tuple[int, ...]:
@@ -147,7 +165,9 @@ def _hetero_block_specs(cfg: ReaLModelConfig, layer_idx: int, P) -> List[ParamSp
     if cfg.loop is not None and cfg.loop.inject and cfg.loop.inject_mode == "linear" and layer_idx == cfg.loop.start + 1:
         add("loop_in.weight", (H, 2 * H), None)
     norm_init = "zeros" if cfg.layer_norm_type == "gemma" else "ones"    # "gemma": the factor is 1 + weight
-    add("attn.ln.weight", (H,), None, init=norm_init)
+    NW = 1 if cfg.scalar_norm else H
+    rg_mixer, rg_mlp = residual_gate_fused(cfg, layer_idx)
+    add("attn.ln.weight", (NW,), None, init=norm_init)
     if cfg.conv_taps:
         add("attn.canon.weight", (H, cfg.conv_taps), None)
     if b.mixer in ("decay", "parallel"):
@@ -165,17 +185,17 @@ def _hetero_block_specs(cfg: ReaLModelConfig, layer_idx: int, P) -> List[ParamSp
             add("attn.o.weight", (H, d.n_heads * d.v_dim), None)
     elif b.mixer == "window_attention":
         w = b.wattn
-        sec = wattn_sections(w)
+        sec = in_sections(cfg, layer_idx)
         add("attn.qkvg.weight", (sum(sec), H), None, sec)
-        if w.qkv_bias:
+        if w.qkv_bias or rg_mixer:
             add("attn.qkvg.bias", (sum(sec),), None, sec, init="zeros")
         if w.head_temp:
             add("attn.temp.weight", (w.n_heads,), None, init="ones")
         if w.sink:
             add("attn.sink.weight", (w.n_heads,), None, init="zeros")
         if w.qk_norm:
-            add("attn.q_norm.weight", (w.qk_dim,), None, init="ones")
-            add("attn.k_norm.weight", (w.qk_dim,), None, init="ones")
+            add("attn.q_norm.weight", (w.qk_dim * (w.n_heads if w.full_norm else 1),), None, init="ones")
+            add("attn.k_norm.weight", (w.qk_dim * (w.n_kv_heads if w.full_norm else 1),), None, init="ones")
         if w.n_maps == 2:
             add("attn.lambda.weight", (4, w.qk_dim), None)     # lq1, lk1, lq2, lk2
         add("attn.o.weight", (H, w.n_heads * w.v_dim), None)
@@ -187,8 +207,10 @@ def _hetero_block_specs(cfg: ReaLModelConfig, layer_idx: int, P) -> List[ParamSp
         add("attn.o_norm.weight", (m.n_heads * m.v_dim,), None, init="ones")
         add("attn.o.weight", (H, m.n_heads * m.v_dim), None)
     elif b.mixer == "latent_attention" and a.rotated:
-        sec = latent_rope_sections(a)
+        sec = in_sections(cfg, layer_idx)
         add("attn.in.weight", (sum(sec), H), None, sec)
+        if rg_mixer:
+            add("attn.in.bias", (sum(sec),), None, sec, init="zeros")
         if a.q_rank:
             add("attn.q_ln.weight", (a.q_rank,), None, init="ones")
             add("attn.uq.weight", (a.n_heads * (a.qk_dim + a.rot_dim), a.q_rank), None)
@@ -216,13 +238,16 @@ def _hetero_block_specs(cfg: ReaLModelConfig, layer_idx: int, P) -> List[ParamSp
         kv_sec = (a.n_heads * a.qk_dim, a.n_heads * a.v_dim)
         add("attn.ukv.weight", (sum(kv_sec), a.kv_rank), None, kv_sec)
         add("attn.o.weight", (H, a.n_heads * a.v_dim), None)
+    if cfg.gated_residual and not rg_mixer:
+        add("attn.rg.weight", (H, H), None)
+        add("attn.rg.bias", (H,), None, init="zeros")
     if cfg.sandwich_norm:
-        add("attn.ln_post.weight", (H,), None, init="ones")
+        add("attn.ln_post.weight", (NW,), None, init="ones")
     if cfg.layer_scale:
         add("attn.ls.weight", (H,), None, init="ones")
     if b.mlp is not None:
         F = b.mlp.ff
-        add("mlp.ln.weight", (H,), None, init=norm_init)
+        add("mlp.ln.weight", (NW,), None, init=norm_init)
         if cfg.conv_taps:
             add("mlp.canon.weight", (H, cfg.conv_taps), None)
         if b.mlp.kind == "moe":
@@ -243,17 +268,25 @@ def _hetero_block_specs(cfg: ReaLModelConfig, layer_idx: int, P) -> List[ParamSp
                 if mo.shared_gate:
                     add("mlp.shared.sg.weight", (1, H), None)
         elif b.mlp.kind == "relu2":
-            add("mlp.up.weight", (F, H), None)
+            if rg_mlp:                              # [up, padded to a multiple of 8 rows | residual gate]
+                sec = (_pad8(F), H)
+                add("mlp.up_rg.weight", (sum(sec), H), None, sec)
+                add("mlp.up_rg.bias", (sum(sec),), None, sec, init="zeros")
+            else:
+                add("mlp.up.weight", (F, H), None)
             add("mlp.down.weight", (H, F), None)
         else:
             add("mlp.gate_up.weight", (2 * F, H), None, (F, F))
             add("mlp.down.weight", (H, F), None)
+        if cfg.gated_residual and not rg_mlp:
+            add("mlp.rg.weight", (H, H), None)
+            add("mlp.rg.bias", (H,), None, init="zeros")
         if cfg.sandwich_norm:
-            add("mlp.ln_post.weight", (H,), None, init="ones")
+            add("mlp.ln_post.weight", (NW,), None, init="ones")
         if cfg.layer_scale:
             add("mlp.ls.weight", (H,), None, init="ones")
     if layer_idx == cfg.n_layers:
-        add("ln_f.weight", (H,), None, init=norm_init)
+        add("ln_f.weight", (NW,), None, init=norm_init)
     return out
 
 

@@ -324,9 +324,10 @@ def latent_decode_attention(qc, w_ln, w_ukv, cache, cache_lens, slots, n_heads: 
 
 
 # ------------------------------------------------------------------------------------------------ window attention with a sink
-# (`WindowAttentionConfig`): grouped key / value heads, no rotation; per-head temperature, linear distance penalty, sliding window
-# that keeps the first tokens, sink logit in the denominator, sigmoid output gate.  Scores, weights and the value norm are fp32.
-# The projection output `qkvg` [T, ld] holds [q (H x d) | k (G x d) | v (G x dv) | gate logits (H, padded)] per row.
+# (`WindowAttentionConfig`): grouped key / value heads; per-head temperature, linear distance penalty, soft cap, sliding window
+# that keeps the first tokens or chunks of positions, sink logit in the denominator, sigmoid output gate per head or element.
+# Scores, weights and the value norm are fp32.  Rotations and query / key norms happen before (`window_prepare_`, `rotate_qk_`).
+# The projection output `qkvg` [T, ld] holds [q (H x d) | k (G x d) | v (G x dv) | gate logits (H or H x dv, padded)] per row.
 # Caches: k_cache [n_slots, G, rows, d], v_cache [n_slots, G, rows, dv]; position p of a sequence lives in row p when
 # p < keep_first, else in row keep_first + (p - keep_first) % (rows - keep_first).
 
@@ -348,6 +349,99 @@ def head_slopes(n_heads: int, slope_base: Optional[float], device) -> torch.Tens
 def _wa_offsets(a):
     nq, nk, nv = a.n_heads * a.qk_dim, a.n_kv_heads * a.qk_dim, a.n_kv_heads * a.v_dim
     return nq, nq + nk, nq + nk + nv
+
+
+def window_gate(qkvg, a):
+    """The gate logits of a window-attention block's projection rows ([T, H] or [T, H * dv]; None without an output gate)."""
+    ov = _wa_offsets(a)[2]
+    return qkvg[:, ov:ov + a.gate_width] if a.out_gate else None
+
+
+def window_values(qkvg, a):
+    """The value heads of a window-attention block's projection rows, [T, G * dv] (a view)."""
+    _, ok_, ov = _wa_offsets(a)
+    return qkvg[:, ok_:ov]
+
+
+def _sink_logits(a, sink, like):
+    """The sink logits the kernels take: the learned ones, or a constant vector in the operand type."""
+    if a.sink_const is None:
+        return sink
+    key = ("sink", a.n_heads, float(a.sink_const), like.dtype, str(like.device))
+    if key not in _ROPE_TABLES:
+        _ROPE_TABLES[key] = torch.full((a.n_heads,), float(a.sink_const), dtype=like.dtype, device=like.device)
+    return _ROPE_TABLES[key]
+
+
+def first_visible(i: int, a) -> int:
+    """First position of the window / chunk part that query i sees (`keep_first` keys come on top)."""
+    if a.chunk is not None:
+        return i // a.chunk * a.chunk
+    return 0 if a.window is None else max(0, i - a.window + 1)
+
+
+def window_prepare_(qkvg, a, wq, wk, eps: float, pos=None, cache_lens=None, slots=None, k_cache=None, v_cache=None, tok_slot=None, remain=None):
+    """In place on the projection rows: q and k RMS-normalised over all their heads (`a.full_norm`, weights wq / wk), q and k rotated
+    (`a.rotary`), values rotated (`a.value_rotary`).  Packed form (`pos` [T]): with caches also stores the keys and values that a
+    later decode step can still see; step form (`pos` None): row b's position is cache_lens[slots[b]], nothing is stored."""
+    H, G, d, dv = a.n_heads, a.n_kv_heads, a.qk_dim, a.v_dim
+    rot, vrot = a.rotary, a.value_rotary
+    fq = rotary_table(rot, qkvg.device)[0] if rot is not None else None
+    fv = rotary_table(vrot, qkvg.device)[0] if vrot is not None else None
+    if rot is not None and rotary_table(rot, qkvg.device)[1] != 1.0:
+        raise ValueError("window attention takes rotations without a factor on cos and sin")
+    if not a.full_norm:
+        wq = wk = None
+    if use_native(qkvg) and d <= 1024 and dv <= 1024:
+        lib().window_prepare_(qkvg, wq, wk, fq, fv, pos, cache_lens if pos is None else None, slots if pos is None else None, k_cache, v_cache,
+                              tok_slot if k_cache is not None else None, remain if k_cache is not None else None, H, G, d, dv,
+                              rot.dims if rot else 0, bool(rot.interleaved) if rot else False, vrot.dims if vrot else 0,
+                              bool(vrot.interleaved) if vrot else False, a.keep_first, eps)
+        return qkvg
+    from realhf_b200.ops.recurrent import _rotate_heads_ref
+    T = qkvg.shape[0]
+    oq, ok_, ov = _wa_offsets(a)
+    n = pos if pos is not None else cache_lens[slots.long() if slots is not None else torch.arange(T, device=qkvg.device)]
+    q, k, v = qkvg[:, :oq].float(), qkvg[:, oq:ok_].float(), qkvg[:, ok_:ov].float().reshape(T, G, dv)
+    if wq is not None:
+        q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps) * wq.float()
+        k = k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps) * wk.float()
+    q, k = q.reshape(T, H, d), k.reshape(T, G, d)
+    if rot is not None:
+        q, k = _rotate_heads_ref(q, n, rot, fq), _rotate_heads_ref(k, n, rot, fq)
+    if vrot is not None:
+        v = _rotate_heads_ref(v, n, vrot, fv)
+    qkvg[:, :ov] = torch.cat([q.reshape(T, -1), k.reshape(T, -1), v.reshape(T, -1)], -1).to(qkvg.dtype)
+    if k_cache is not None:
+        import dataclasses
+        value_norm_store_ref(qkvg, dataclasses.replace(a, value_norm=False), eps, k_cache, v_cache, tok_slot, n, remain)
+    return qkvg
+
+
+def turn_gate_(x, a, gate, pos=None, cache_lens=None, slots=None):
+    """Attention output x [T, H * dv] in place: every head turned back by the row's position (`a.value_rotary`), then times the sigmoid
+    of the gate logits (per head or per element; None: no gate)."""
+    T, H, dv, vrot = x.shape[0], a.n_heads, a.v_dim, a.value_rotary
+    fv = rotary_table(vrot, x.device)[0] if vrot is not None else None
+    if use_native(x) and dv <= 1024:
+        lib().turn_gate_(x, gate, a.element_gate, fv, pos, cache_lens if pos is None else None, slots if pos is None else None, H, dv,
+                         vrot.dims if vrot else 0, bool(vrot.interleaved) if vrot else False)
+        return x
+    from realhf_b200.ops.recurrent import _rotate_heads_ref
+    o = x.float().reshape(T, H, dv)
+    if vrot is not None:
+        n = pos if pos is not None else cache_lens[slots.long() if slots is not None else torch.arange(T, device=x.device)]
+        o = _rotate_heads_ref(o, -n, vrot, fv)
+    x.copy_(_apply_gate_ref(o, gate).reshape(T, -1).to(x.dtype))
+    return x
+
+
+def _apply_gate_ref(o, gate):
+    """o [T, H, dv] fp32 times sigmoid of [T, H] or [T, H * dv] gate logits."""
+    if gate is None:
+        return o
+    g = torch.sigmoid(gate.float())
+    return o * (g.unsqueeze(-1) if gate.shape[1] == o.shape[1] else g.reshape(o.shape))
 
 
 def value_norm_store_ref(qkvg, a, eps, k_cache, v_cache, tok_slot, pos, remain):
@@ -424,8 +518,8 @@ def sink_window_attention_ref(qkvg, v_n, a, temp, sink, cu_seqlens):
     oq, ok_, ov = _wa_offsets(a)
     q = qkvg[:, :oq].float().view(T, H, d)
     k = qkvg[:, oq:ok_].float().view(T, G, d)
-    v = v_n.float().view(T, G, dv)
-    gate = torch.sigmoid(qkvg[:, ov:ov + H].float()) if a.out_gate else None
+    v = v_n.float().reshape(T, G, dv)
+    sink = _sink_logits(a, sink, qkvg)
     slopes = head_slopes(H, a.slope_base, qkvg.device)
     out = torch.zeros(T, H, dv, dtype=torch.float32, device=qkvg.device)
     cu = cu_seqlens.tolist()
@@ -439,16 +533,20 @@ def sink_window_attention_ref(qkvg, v_n, a, temp, sink, cu_seqlens):
         ok = j <= i
         if a.window is not None:
             ok = ok & ((i - j < a.window) | (j < a.keep_first))
+        if a.chunk is not None:
+            ok = ok & (i // a.chunk == j // a.chunk)
         dist = (i - j).float()
         for h in range(H):
             g = h // (H // G)
             sc = (q[s0:e0, h] @ k[s0:e0, g].T) * a.scale
             if temp is not None:
                 sc = sc * temp[h].float()
+            if a.softcap is not None:
+                sc = a.softcap * torch.tanh(sc / a.softcap)
             sc = sc - slopes[h] * dist
             out[s0:e0, h] = _sink_softmax_pv(sc, ok, sink[h].float() if sink is not None else None, v[s0:e0, g])
-    if gate is not None:
-        out = out * gate.unsqueeze(-1)
+    if a.value_rotary is None:                      # (else the output is turned back first: turn_gate_)
+        out = _apply_gate_ref(out, window_gate(qkvg, a))
     return out.reshape(T, H * dv).to(qkvg.dtype)
 
 
@@ -457,26 +555,32 @@ def _sink_tc_ok(qkvg, v_n, a) -> bool:
     weights rounded to the operand type for the P.V product); `REAL_WINDOW_ATTN=simt` selects the all-fp32 CUDA-core kernel."""
     return (os.environ.get("REAL_WINDOW_ATTN", "tcgen05") == "tcgen05" and qkvg.dtype in (torch.bfloat16, torch.float16)
             and a.qk_dim == a.v_dim and a.qk_dim in (64, 128) and qkvg.stride(0) % 8 == 0 and qkvg.data_ptr() % 16 == 0
-            and (a.n_heads * a.qk_dim) % 8 == 0 and v_n.data_ptr() % 16 == 0)
+            and (a.n_heads * a.qk_dim) % 8 == 0 and v_n.data_ptr() % 16 == 0 and v_n.stride(0) % 8 == 0)
 
 
 def sink_window_attention(qkvg, v_n, a, temp, sink, pos, cu_seqlens, max_seqlen=None):
     """Packed causal attention of a window-attention block over the batch's own keys (every sequence starts at position 0):
-    softmax_j(q_i . k_j * scale * temp_h - slope_h (i - j)) with the sink logit in the denominator, over j <= i with
-    i - j < window or j < keep_first; head h's output times sigmoid(gate logit h).  Returns [T, H * dv] in the model dtype."""
+    softmax_j(q_i . k_j * scale * temp_h - slope_h (i - j)) with the sink logit in the denominator (soft-capped with `a.softcap`), over
+    j <= i with i - j < window or j < keep_first (or of the same chunk); times the sigmoid gate.  With `a.value_rotary` the output
+    comes turned back by the query's position, before the gate.  Returns [T, H * dv] in the model dtype."""
+    out = _sink_window_attention(qkvg, v_n, a, temp, sink, pos, cu_seqlens, max_seqlen)
+    return turn_gate_(out, a, window_gate(qkvg, a), pos=pos) if a.value_rotary is not None else out
+
+
+def _sink_window_attention(qkvg, v_n, a, temp, sink, pos, cu_seqlens, max_seqlen):
     if use_native(qkvg) and a.qk_dim <= 512 and a.v_dim <= 256:     # (larger heads: the PyTorch form, on the device)
         T = qkvg.shape[0]
         out = torch.empty(T, a.n_heads * a.v_dim, dtype=qkvg.dtype, device=qkvg.device)
         if max_seqlen is None:
             max_seqlen = int((cu_seqlens[1:] - cu_seqlens[:-1]).max())
-        if _sink_tc_ok(qkvg, v_n, a):
-            lib().sink_window_attention_tc(qkvg, v_n, out, temp, sink, cu_seqlens, max_seqlen, a.n_heads, a.n_kv_heads, a.qk_dim, a.scale,
-                                           a.window if a.window is not None else -1, a.keep_first,
-                                           a.slope_base if a.slope_base is not None else -1.0, bool(a.out_gate))
-            return out
-        lib().sink_window_attention(qkvg, v_n, out, temp, sink, cu_seqlens, max_seqlen, a.n_heads, a.n_kv_heads, a.qk_dim, a.v_dim, a.scale,
-                                    a.window if a.window is not None else -1, a.keep_first,
-                                    a.slope_base if a.slope_base is not None else -1.0, bool(a.out_gate))
+        sink = _sink_logits(a, sink, qkvg)
+        gate = window_gate(qkvg, a) if a.value_rotary is None else None
+        shape = (a.scale, a.window if a.window is not None else -1, a.keep_first, a.slope_base if a.slope_base is not None else -1.0, gate,
+                 a.element_gate, a.chunk or 0, a.softcap or 0.0)
+        if _sink_tc_ok(qkvg, v_n, a) and not (gate is not None and a.element_gate and gate.data_ptr() % 16):
+            lib().sink_window_attention_tc(qkvg, v_n, out, temp, sink, cu_seqlens, max_seqlen, a.n_heads, a.n_kv_heads, a.qk_dim, *shape)
+        else:
+            lib().sink_window_attention(qkvg, v_n, out, temp, sink, cu_seqlens, max_seqlen, a.n_heads, a.n_kv_heads, a.qk_dim, a.v_dim, *shape)
         return out
     return sink_window_attention_ref(qkvg, v_n, a, temp, sink, cu_seqlens)
 
@@ -486,6 +590,7 @@ def sink_window_decode_attention_ref(qkvg, a, temp, sink, k_cache, v_cache, cach
     H, G, d, dv = a.n_heads, a.n_kv_heads, a.qk_dim, a.v_dim
     oq, ok_, ov = _wa_offsets(a)
     rows = k_cache.shape[2]
+    sink = _sink_logits(a, sink, qkvg)
     slopes = head_slopes(H, a.slope_base, qkvg.device)
     out = torch.zeros(B, H, dv, dtype=torch.float32, device=qkvg.device)
     for b in range(B):
@@ -498,8 +603,7 @@ def sink_window_decode_attention_ref(qkvg, a, temp, sink, k_cache, v_cache, cach
         k_cache[s, :, r] = qkvg[b, oq:ok_].view(G, d)
         v_cache[s, :, r] = v_new.to(v_cache.dtype)
         j = torch.arange(n + 1, device=qkvg.device)
-        if a.window is not None:
-            j = j[(n - j < a.window) | (j < a.keep_first)]
+        j = j[(j >= first_visible(n, a)) | (j < a.keep_first)]
         rj = cache_row(j, a.keep_first, rows)
         kk = k_cache[s][:, rj].float()                             # [G, n_keys, d]
         vv = v_cache[s][:, rj].float()
@@ -509,23 +613,28 @@ def sink_window_decode_attention_ref(qkvg, a, temp, sink, k_cache, v_cache, cach
             sc = (kk[g] @ q[h]) * a.scale
             if temp is not None:
                 sc = sc * temp[h].float()
+            if a.softcap is not None:
+                sc = a.softcap * torch.tanh(sc / a.softcap)
             sc = (sc - slopes[h] * (n - j).float()).unsqueeze(0)
             out[b, h] = _sink_softmax_pv(sc, torch.ones_like(sc, dtype=torch.bool), sink[h].float() if sink is not None else None, vv[g])[0]
-        if a.out_gate:
-            out[b] = out[b] * torch.sigmoid(qkvg[b, ov:ov + H].float()).unsqueeze(-1)
-    return out.reshape(B, H * dv).to(qkvg.dtype)
+    out = out.reshape(B, H * dv)
+    return turn_gate_(out, a, window_gate(qkvg, a), cache_lens=cache_lens, slots=slots).to(qkvg.dtype)
 
 
 def sink_window_decode_attention(qkvg, a, temp, sink, k_cache, v_cache, cache_lens, slots, eps: float):
     """One new token per row against the caches of its slot (slots None: row b is slot b).  The row's key and normalised value
     are appended in place at the row of position cache_lens[slot] (cache_lens itself is not changed), then the token attends to
-    every cached position its window and `keep_first` allow, itself included.  Returns [B, H * dv] in the model dtype."""
+    every cached position its window and `keep_first` (or its chunk) allow, itself included; turning back and gate as in the packed
+    form.  Returns [B, H * dv] in the model dtype."""
     if use_native(qkvg) and a.v_dim <= 256:
         B = qkvg.shape[0]
         out = torch.empty(B, a.n_heads * a.v_dim, dtype=qkvg.dtype, device=qkvg.device)
-        lib().sink_window_decode_attention(qkvg, out, temp, sink, k_cache, v_cache, cache_lens, slots, a.n_heads, a.n_kv_heads, a.qk_dim,
-                                           a.v_dim, a.scale, a.window if a.window is not None else -1, a.keep_first,
-                                           a.slope_base if a.slope_base is not None else -1.0, bool(a.out_gate), bool(a.value_norm), eps)
+        vr = a.value_rotary
+        lib().sink_window_decode_attention(qkvg, out, temp, _sink_logits(a, sink, qkvg), k_cache, v_cache, cache_lens, slots, a.n_heads, a.n_kv_heads,
+                                           a.qk_dim, a.v_dim, a.scale, a.window if a.window is not None else -1, a.keep_first,
+                                           a.slope_base if a.slope_base is not None else -1.0, window_gate(qkvg, a), a.element_gate, a.chunk or 0,
+                                           a.softcap or 0.0, rotary_table(vr, qkvg.device)[0] if vr is not None else None,
+                                           vr.dims if vr is not None else 0, bool(vr.interleaved) if vr is not None else False, bool(a.value_norm), eps)
         return out
     return sink_window_decode_attention_ref(qkvg, a, temp, sink, k_cache, v_cache, cache_lens, slots, eps)
 
@@ -589,10 +698,10 @@ def diff_window_attention(qkv, a, wq, wk, w_lambda, eps: float, k_cache, v_cache
         if _sink_tc_ok(qkv, v_n, av):
             # 16-bit operands, head size 64 / 128: the tcgen05 kernel; both maps' weighted sums come back in the operand type
             att = torch.empty(T, 2 * H * dv, dtype=qkv.dtype, device=qkv.device)
-            lib().sink_window_attention_tc(qkv, v_n, att, None, None, cu_seqlens, max_seqlen, 2 * H, 2 * G, d, a.scale, win, a.keep_first, -1.0, False, 2)
+            lib().sink_window_attention_tc(qkv, v_n, att, None, None, cu_seqlens, max_seqlen, 2 * H, 2 * G, d, a.scale, win, a.keep_first, -1.0, vshare=2)
         else:
             att = torch.empty(T, 2 * H * dv, dtype=torch.float32, device=qkv.device)
-            lib().sink_window_attention(qkv, v_n, att, None, None, cu_seqlens, max_seqlen, 2 * H, 2 * G, d, dv, a.scale, win, a.keep_first, -1.0, False, 2)
+            lib().sink_window_attention(qkv, v_n, att, None, None, cu_seqlens, max_seqlen, 2 * H, 2 * G, d, dv, a.scale, win, a.keep_first, -1.0, vshare=2)
         out = torch.empty(T, H * dv, dtype=qkv.dtype, device=qkv.device)
         lib().diff_combine(att, lam, out, H, G, dv, a.diff, eps)
         return out
@@ -638,7 +747,7 @@ def diff_window_decode_attention(qkv, a, wq, wk, w_lambda, eps: float, k_cache, 
         fast = qkv.dtype != torch.float32 and d == dv and d in (64, 128) and (H // G) in (1, 2, 4, 8)    # the streaming 16-bit kernel
         att = torch.empty(B, 2 * H * dv, dtype=qkv.dtype if fast else torch.float32, device=qkv.device)
         lib().sink_window_decode_attention(qkv, att, None, None, k_cache, v_cache, cache_lens, slots, 2 * H, 2 * G, d, dv, a.scale,
-                                           a.window if a.window is not None else -1, a.keep_first, -1.0, False, False, eps, 2)
+                                           a.window if a.window is not None else -1, a.keep_first, -1.0, None, False, 0, 0.0, None, 0, False, False, eps, 2)
         out = torch.empty(B, H * dv, dtype=qkv.dtype, device=qkv.device)
         lib().diff_combine(att, lam, out, H, G, dv, a.diff, eps)
         return out
@@ -674,7 +783,7 @@ _ROPE_TABLES: dict = {}
 
 def rotary_table(rot, device):
     """(fp32 frequencies [dims / 2] on `device`, rounded once from double precision; factor on cos / sin)."""
-    key = (rot.dims, rot.base, rot.factor, rot.original, rot.fast, rot.slow, str(device))
+    key = (rot.dims, rot.base, rot.factor, rot.original, rot.fast, rot.slow, rot.scaling, str(device))
     hit = _ROPE_TABLES.get(key)
     if hit is None:
         f, m = rot.frequencies()
@@ -682,13 +791,20 @@ def rotary_table(rot, device):
     return hit
 
 
-def _rotate_ref(x, pos, inv_freq, mscale):
-    """x [N, ..., rot] fp32, pos [N]: interleaved pairs turn by pos * f_i (fp32)."""
+def _rotate_ref(x, pos, inv_freq, mscale, inter=True):
+    """x [N, ..., rot] fp32, pos [N]: interleaved pairs (else (i, i + rot / 2)) turn by pos * f_i (fp32)."""
     ang = pos.float().unsqueeze(-1) * inv_freq
     shape = [x.shape[0]] + [1] * (x.dim() - 2) + [inv_freq.numel()]
     cs, sn = (torch.cos(ang) * mscale).view(shape), (torch.sin(ang) * mscale).view(shape)
+    if not inter:
+        u, v = x.chunk(2, -1)
+        return torch.cat([u * cs - v * sn, v * cs + u * sn], -1)
     u, v = x[..., 0::2], x[..., 1::2]
     return torch.stack([u * cs - v * sn, v * cs + u * sn], -1).flatten(-2)
+
+
+def _latent_inter(a) -> bool:
+    return a.rotary is None or bool(a.rotary.interleaved)
 
 
 def latent_rope_prepare(proj, a, wq, wc, eps: float, pos, cache, tok_slot=None, remain=None, cache_lens=None, slots=None, want_lat=True):
@@ -704,7 +820,7 @@ def latent_rope_prepare(proj, a, wq, wc, eps: float, pos, cache, tok_slot=None, 
         lat = torch.empty(T, r + rot, dtype=proj.dtype, device=proj.device) if want_lat else None
         lib().latent_rope_prepare(proj, wq if qr else None, wc, inv_freq, ms, pos, cache_lens if pos is None else None,
                                   slots if pos is None else None, tok_slot if (cache is not None and pos is not None) else None,
-                                  remain if (cache is not None and pos is not None) else None, cq, lat, cache, qr, r, rot, eps)
+                                  remain if (cache is not None and pos is not None) else None, cq, lat, cache, qr, r, rot, eps, _latent_inter(a))
         return cq, lat
     cq = None
     if qr:
@@ -719,7 +835,7 @@ def latent_rope_prepare(proj, a, wq, wc, eps: float, pos, cache, tok_slot=None, 
         p = pos
     parts = [c]
     if rot:
-        parts.append(_rotate_ref(proj[:, qr + r:qr + r + rot].float(), p, inv_freq, ms))
+        parts.append(_rotate_ref(proj[:, qr + r:qr + r + rot].float(), p, inv_freq, ms, _latent_inter(a)))
     lat = torch.cat(parts, -1).to(proj.dtype)
     if cache is not None:
         R = cache.shape[1]
@@ -731,30 +847,32 @@ def latent_rope_prepare(proj, a, wq, wc, eps: float, pos, cache, tok_slot=None, 
     return cq, lat
 
 
-def latent_rope_attention(q, kv, lat, a, sink, pos, cu_seqlens, max_seqlen=None):
+def latent_rope_attention(q, kv, lat, a, sink, pos, cu_seqlens, max_seqlen=None, gate=None):
     """Packed causal attention: q [T, H (d + rot)] (rotated here), kv [T, H d | H dv] the up-projected unrotated keys and values,
     lat [T, kv_rank + rot] whose last rot columns are the rotated key part of every head.  The softmax denominator holds
-    exp(sink_h) when `sink` is given.  Returns [T, H * dv] in q's dtype."""
+    exp(sink_h) when `sink` is given; the output is multiplied by the sigmoid of `gate` ([T, H] or [T, H * dv] logits, or None).
+    Returns [T, H * dv] in q's dtype."""
     T = q.shape[0]
     H, d, rot, dv, r = a.n_heads, a.qk_dim, a.rot_dim, a.v_dim, a.kv_rank
     dq = d + rot
     inv_freq, ms = rotary_table(a.rotary, q.device) if rot else (torch.zeros(1, device=q.device), 1.0)
     if use_native(q) and dq <= 512 and dv <= 256:
         qk = torch.empty(T, 2 * H * dq, dtype=q.dtype, device=q.device)
-        lib().latent_rope_assemble(q, kv, lat, pos, inv_freq, ms, qk, H, d, rot, r)
+        lib().latent_rope_assemble(q, kv, lat, pos, inv_freq, ms, qk, H, d, rot, r, _latent_inter(a))
         out = torch.empty(T, H * dv, dtype=q.dtype, device=q.device)
         if max_seqlen is None:
             max_seqlen = int((cu_seqlens[1:] - cu_seqlens[:-1]).max())
         vv = kv[:, H * d:]
         if (os.environ.get("REAL_WINDOW_ATTN", "tcgen05") == "tcgen05" and q.dtype in (torch.bfloat16, torch.float16) and dq == dv and dq in (64, 128)
-                and kv.stride(0) % 8 == 0 and (H * d) % 8 == 0 and vv.data_ptr() % 16 == 0):
-            lib().sink_window_attention_tc(qk, vv, out, None, sink, cu_seqlens, max_seqlen, H, H, dq, a.scale, -1, 0, -1.0, False, 1)
+                and kv.stride(0) % 8 == 0 and (H * d) % 8 == 0 and vv.data_ptr() % 16 == 0
+                and (gate is None or a.head_gate or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0))):
+            lib().sink_window_attention_tc(qk, vv, out, None, sink, cu_seqlens, max_seqlen, H, H, dq, a.scale, -1, 0, -1.0, gate, not a.head_gate)
         else:
-            lib().sink_window_attention(qk, vv, out, None, sink, cu_seqlens, max_seqlen, H, H, dq, dv, a.scale, -1, 0, -1.0, False, 1)
+            lib().sink_window_attention(qk, vv, out, None, sink, cu_seqlens, max_seqlen, H, H, dq, dv, a.scale, -1, 0, -1.0, gate, not a.head_gate)
         return out
     qh = q.float().view(T, H, dq)
     if rot:
-        qh = torch.cat([qh[..., :d], _rotate_ref(qh[..., d:], pos, inv_freq, ms).to(q.dtype).float()], -1)
+        qh = torch.cat([qh[..., :d], _rotate_ref(qh[..., d:], pos, inv_freq, ms, _latent_inter(a)).to(q.dtype).float()], -1)
     kh = torch.cat([kv[:, : H * d].float().view(T, H, d), lat[:, r:].float().unsqueeze(1).expand(T, H, rot)], -1)
     vh = kv[:, H * d:].float().view(T, H, dv)
     out = torch.zeros(T, H, dv, dtype=torch.float32, device=q.device)
@@ -768,13 +886,13 @@ def latent_rope_attention(q, kv, lat, a, sink, pos, cu_seqlens, max_seqlen=None)
         for h in range(H):
             sc = (qh[s0:e0, h] @ kh[s0:e0, h].T) * a.scale
             out[s0:e0, h] = _sink_softmax_pv(sc, ok, sink[h].float() if sink is not None else None, vh[s0:e0, h])
-    return out.reshape(T, H * dv).to(q.dtype)
+    return _apply_gate_ref(out, gate).reshape(T, H * dv).to(q.dtype)
 
 
-def latent_rope_decode_attention(q, a, w_ukv, sink, cache, cache_lens, slots):
+def latent_rope_decode_attention(q, a, w_ukv, sink, cache, cache_lens, slots, gate=None):
     """One new token per row against the cached rows [c | k_rot] of its slot (the row of the new token is already stored).  Keys
     and values are never formed: score_j = scale (q_nope W_uk) . c_j + scale rotate(q_rot) . k_rot_j, the weighted sum of the cached
-    latents comes back through W_uv.  Returns [B, H * dv] in q's dtype."""
+    latents comes back through W_uv, times the sigmoid of `gate` as in the packed form.  Returns [B, H * dv] in q's dtype."""
     B = q.shape[0]
     H, d, rot, dv, r = a.n_heads, a.qk_dim, a.rot_dim, a.v_dim, a.kv_rank
     dq = d + rot
@@ -786,18 +904,20 @@ def latent_rope_decode_attention(q, a, w_ukv, sink, cache, cache_lens, slots):
         qa = torch.empty(H, B, r + rot, dtype=torch.float32, device=q.device)
         qa[:, :, :r] = torch.bmm(q.view(B, H, dq)[:, :, :d].transpose(0, 1).float(), wk)
         if rot:
-            lib().latent_query_rope(q, cache_lens, slots, inv_freq, ms, a.scale, qa, d, rot)
+            lib().latent_query_rope(q, cache_lens, slots, inv_freq, ms, a.scale, qa, d, rot, _latent_inter(a))
         ctas = B * ((H + 15) // 16)
         splits = max(1, min((3 * 148 + ctas - 1) // ctas, R // 64, 32))
         sk = cached_on(sink, "_f32", lambda w: w.float().contiguous()) if sink is not None else None
         o = lib().latent_decode_core(qa, cache, cache_lens, slots, 0, splits, sk)
-        return torch.bmm(o[:, :, :r], wv).transpose(0, 1).reshape(B, H * dv).to(q.dtype)
+        out = torch.empty(B, H * dv, dtype=q.dtype, device=q.device)
+        lib().latent_out(torch.bmm(o[:, :, :r], wv), gate, not a.head_gate, out)
+        return out
     idx = slots.long() if slots is not None else torch.arange(B, device=q.device)
     pos = cache_lens[idx]
     qh = q.float().view(B, H, dq)
     qa = torch.einsum("bhd,hdr->bhr", qh[..., :d], wk)
     if rot:
-        qa = torch.cat([qa, _rotate_ref(qh[..., d:], pos, inv_freq, ms) * a.scale], -1)
+        qa = torch.cat([qa, _rotate_ref(qh[..., d:], pos, inv_freq, ms, _latent_inter(a)) * a.scale], -1)
     out = torch.empty(B, H * dv, dtype=torch.float32, device=q.device)
     for b in range(B):
         p = int(pos[b])
@@ -805,7 +925,7 @@ def latent_rope_decode_attention(q, a, w_ukv, sink, cache, cache_lens, slots):
         sc = qa[b] @ cw.t()
         pr = _sink_softmax_pv(sc, torch.ones_like(sc, dtype=torch.bool), sink.float().unsqueeze(-1) if sink is not None else None, cw[:, :r])
         out[b] = torch.einsum("hr,hrv->hv", pr, wv).reshape(-1)
-    return out.to(q.dtype)
+    return _apply_gate_ref(out.view(B, H, dv), gate).reshape(B, H * dv).to(q.dtype)
 
 
 def sigmoid_gate_(x, gate):

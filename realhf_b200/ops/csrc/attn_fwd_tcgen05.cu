@@ -30,7 +30,10 @@
 // slope_h = 2^(-slope_base (h + 1) / nq) (formed per element in the log2 domain with one extra FMA in each pass), a sliding
 // window that also keeps the first `keep` keys (the key tiles of [0, keep) that lie below the window's first tile are walked
 // first by all three roles), a per-head sink logit that starts the running maximum with denominator 1, and the row's output
-// times sigmoid(gate logit of its head).
+// times sigmoid(gate logit of its head, or of the output element).  `chunk` > 0 replaces the window: a query sees the keys of its own
+// chunk of positions up to itself (the tiles below the first row's chunk are not walked, a later row's chunk start is its lower
+// mask edge).  kCap: score = softcap * tanh(s * scale / softcap); the cap is monotone, so the row maximum is taken before it and
+// capped once, and only the pass that forms the weights evaluates tanh per element.
 #include "gemm_common.cuh"
 
 namespace {
@@ -56,6 +59,9 @@ struct AttnParams {
   int64_t gate_ld;
   float slope_base;       // < 0: no distance term
   int vshare = 1;         // consecutive key heads that read one value head (V has nkv / vshare heads)
+  int gate_mode = 1;      // gate logits: 1 one per head, 2 one per output element (element (t, h, c) at gate[t * gate_ld + h * D + c])
+  int chunk = 0;          // > 0 (window 0): a query sees the keys of its own chunk
+  float softcap = 0.f;    // kCap variant
 };
 
 template <int kD> struct ACfg {
@@ -82,7 +88,11 @@ template <> RB_DEVICE uint32_t pack2<__half>(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
-template <int kD, typename T, int kFmt, bool kSink = false>
+// cap * tanh(t / cap) in the log2 domain (times log2 e), tanh(x) = 1 - 2 / (1 + 2^(2 x log2 e)): c = 2 log2 e / cap, k = cap log2 e.
+// Absolute error a few ulp of k; saturates to +-k.
+RB_DEVICE float soft_cap2(float t, float c, float k) { return k - __fdividef(2.f * k, 1.f + exp2f(fminf(t * c, 80.f))); }
+
+template <int kD, typename T, int kFmt, bool kSink = false, bool kCap = false>
 __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q,
                                                                    const __grid_constant__ CUtensorMap tma_k,
                                                                    const __grid_constant__ CUtensorMap tma_v, AttnParams p) {
@@ -96,7 +106,9 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
   const int hk = head / (p.nq / p.nkv);
   const int kv_len = p.causal ? min(L, q0 + kBQ) : L;
   const int win = (p.causal && p.window > 0) ? p.window : 0;
-  const int tile0 = win > 0 ? max(0, q0 - win + 1) / kBKV : 0;   // first key tile any row of this CTA can see
+  const int chunk = kSink ? p.chunk : 0;
+  // first key tile any row of this CTA can see
+  const int tile0 = (kSink && chunk > 0) ? (q0 / chunk * chunk) / kBKV : win > 0 ? max(0, q0 - win + 1) / kBKV : 0;
   // kSink: the tiles of the kept first keys that lie wholly below tile0 come first in every role's walk
   const int n_keep = (kSink && win > 0) ? min(RB_CEIL_DIV(p.keep, kBKV), tile0) : 0;
   const int n_kv = n_keep + RB_CEIL_DIV(kv_len, kBKV) - tile0;    // >= 1: the diagonal tile is always visible
@@ -214,10 +226,14 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
     const uint32_t p_row = sP + (uint32_t)(row >> 3) * 1024u + (uint32_t)(row & 7) * 128u;
     const uint32_t sw = (uint32_t)(row & 7);
     float m_run = -INFINITY, l_run = 0.f, alpha_prev = 0.f;
+    const int row_lo = (kSink && chunk > 0) ? q_pos / chunk * chunk : win > 0 ? q_pos - win + 1 : 0;   // first visible key of the row
+    const int last_lo = (kSink && chunk > 0) ? (q0 + kBQ - 1) / chunk * chunk : q0 + kBQ - win;      // of the tile's last row
+    const bool bounded = win > 0 || (kSink && chunk > 0);
+    const float cap_c = kCap ? 2.f * 1.4426950408889634f / p.softcap : 0.f, cap_k = kCap ? p.softcap * 1.4426950408889634f : 0.f;
     // kSink: scores live in the log2 domain, t = s * c2 - slope2 * (q_pos - key_pos); the sink starts the maximum
     float c2 = 0.f, slope2 = 0.f;
     if constexpr (kSink) {
-      c2 = sl2 * (p.temp ? rb::to_f(reinterpret_cast<const T*>(p.temp)[head]) : 1.f);
+      c2 = (kCap ? p.scale : sl2) * (p.temp ? rb::to_f(reinterpret_cast<const T*>(p.temp)[head]) : 1.f);   // (kCap: natural units until the cap)
       slope2 = p.slope_base >= 0.f ? exp2f(-p.slope_base * (float)(head + 1) / (float)p.nq) * 1.4426950408889634f : 0.f;
       if (p.sink) { m_run = rb::to_f(reinterpret_cast<const T*>(p.sink)[head]) * 1.4426950408889634f; l_run = 1.f; }
     }
@@ -249,9 +265,9 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
       ptx::tc_fence_after();
       // only the last tile of the sequence, the diagonal tile and the tiles the window's lower edge crosses need per-element
       // masks (uniform over the CTA)
-      const bool need_mask = (kv0 + kBKV > L) || (p.causal && kv0 + kBKV - 1 > q0) || (win > 0 && q0 + kBQ - win > kv0);
+      const bool need_mask = (kv0 + kBKV > L) || (p.causal && kv0 + kBKV - 1 > q0) || (bounded && last_lo > kv0);
       const int lim = (p.causal ? min(L, q_pos + 1) : L) - kv0;  // local key columns [lo, lim) are visible to this row
-      const int lo = win > 0 ? q_pos - win + 1 - kv0 : 0;
+      const int lo = bounded ? row_lo - kv0 : 0;
       const int kept = kSink ? p.keep - kv0 : 0;                 // kSink: local columns below `kept` stay visible under `lo`
       auto hidden = [&](int col) { return col >= lim || (col < lo && (!kSink || col >= kept)); };
       const float base = kSink ? slope2 * (float)(kv0 - q_pos) : 0.f;
@@ -264,11 +280,13 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           float s = __uint_as_float(r[i]);
-          if constexpr (kSink) s = fmaf(s, c2, fmaf(slope2, (float)(c * 32 + i), base));
+          if constexpr (kCap) s *= c2;
+          else if constexpr (kSink) s = fmaf(s, c2, fmaf(slope2, (float)(c * 32 + i), base));
           if (need_mask && hidden(c * 32 + i)) s = -INFINITY;
           mx = fmaxf(mx, s);
         }
       }
+      if constexpr (kCap) { if (mx != -INFINITY) mx = soft_cap2(mx, cap_c, cap_k); }
       const float m_new = fmaxf(m_run, mx);
       const float m_eff = (m_new == -INFINITY) ? 0.f : m_new;  // fully masked so far: keep exp2 arguments finite
       const float alpha = kSink ? exp2f(m_run - m_eff) : exp2f((m_run - m_eff) * sl2);
@@ -284,7 +302,10 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
           float e0, e1;
-          if constexpr (kSink) {
+          if constexpr (kCap) {
+            e0 = exp2f(soft_cap2(__uint_as_float(r[i]) * c2, cap_c, cap_k) + neg_m);
+            e1 = exp2f(soft_cap2(__uint_as_float(r[i + 1]) * c2, cap_c, cap_k) + neg_m);
+          } else if constexpr (kSink) {
             e0 = exp2f(fmaf(__uint_as_float(r[i]), c2, fmaf(slope2, (float)(c * 32 + i), base)) + neg_m);
             e1 = exp2f(fmaf(__uint_as_float(r[i + 1]), c2, fmaf(slope2, (float)(c * 32 + i + 1), base)) + neg_m);
           } else {
@@ -322,7 +343,17 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
     if (q_pos < L) {
       float inv = 1.f / l_run;
       if constexpr (kSink) {
-        if (p.gate) inv *= 1.f / (1.f + __expf(-rb::to_f(reinterpret_cast<const T*>(p.gate)[(int64_t)(tok0 + q_pos) * p.gate_ld + head])));
+        if (p.gate && p.gate_mode == 1)
+          inv *= 1.f / (1.f + __expf(-rb::to_f(reinterpret_cast<const T*>(p.gate)[(int64_t)(tok0 + q_pos) * p.gate_ld + head])));
+        if (p.gate && p.gate_mode == 2) {          // (rows of the gate are 16-byte aligned: checked by the host)
+          const T* gr = reinterpret_cast<const T*>(p.gate) + (int64_t)(tok0 + q_pos) * p.gate_ld + (int64_t)head * kD;
+#pragma unroll
+          for (int i = 0; i < kD; i += 8) {
+            const rb::Pack<T, 8> gv = *reinterpret_cast<const rb::Pack<T, 8>*>(gr + i);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) O[i + j] *= __fdividef(1.f, 1.f + __expf(-rb::to_f(gv.v[j])));
+          }
+        }
       }
       T* dst = reinterpret_cast<T*>(p.out) + (int64_t)(tok0 + q_pos) * p.out_ld + (int64_t)head * kD;
 #pragma unroll
@@ -346,11 +377,11 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
   }
 }
 
-template <int kD, typename T, int kFmt, bool kSink = false>
+template <int kD, typename T, int kFmt, bool kSink = false, bool kCap = false>
 int launch_attn_fwd(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnParams& p, int B,
                     int max_seqlen, cudaStream_t s) {
   using C = ACfg<kD>;
-  auto kern = attn_fwd_kernel<kD, T, kFmt, kSink>;
+  auto kern = attn_fwd_kernel<kD, T, kFmt, kSink, kCap>;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmemBytes) != cudaSuccess) return -30;
@@ -397,28 +428,35 @@ extern "C" int rb_attn_fwd(const void* q, const void* k, const void* v, void* ou
 }
 
 // Window attention with a sink on the tensor cores (see the kSink notes at the top): q / k / v as for rb_attn_fwd (equal query /
-// value head size of 64 or 128), temp / sink [nq] in the operand type or null, gate logits at gate[t * gate_ld + h] or null,
-// window <= 0 = every earlier key, keep = first keys that stay visible, slope_base < 0 = no distance term.
+// value head size of 64 or 128), temp / sink [nq] in the operand type or null, gate logits at gate[t * gate_ld + h] (gate_mode 1) or
+// gate[t * gate_ld + h * hd + c] (gate_mode 2) or null, window <= 0 = every earlier key, keep = first keys that stay visible,
+// chunk > 0 = chunked instead of windowed, softcap > 0 = capped scores (no distance term then), slope_base < 0 = no distance term.
 extern "C" int rb_attn_fwd_sink(const void* q, const void* k, const void* v, void* out, const int* cu_seqlens, int64_t q_ld, int64_t k_ld,
                                 int64_t v_ld, int64_t out_ld, int T, int B, int nq, int nkv, int hd, int max_seqlen, float scale, int window,
-                                int keep, const void* temp, const void* sink, const void* gate, int64_t gate_ld, float slope_base, int dt,
-                                int vshare, cudaStream_t s) {
+                                int keep, const void* temp, const void* sink, const void* gate, int64_t gate_ld, int gate_mode, int chunk,
+                                float softcap, float slope_base, int dt, int vshare, cudaStream_t s) {
   if (hd != 128 && hd != 64) return -1;
   if (dt != 1 && dt != 2) return -2;
   if (nq % nkv != 0 || T <= 0 || B <= 0 || max_seqlen <= 0 || vshare < 1 || nkv % vshare) return -3;
   if ((q_ld | k_ld | v_ld | out_ld) % 8 != 0) return -4;
   if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)out) & 15) return -5;
+  if (gate != nullptr && gate_mode == 2 && (gate_ld % 8 != 0 || ((uintptr_t)gate & 15))) return -6;
+  if (softcap > 0.f && slope_base >= 0.f) return -7;
+  if (chunk > 0 && window > 0) return -8;
   CUtensorMap mq, mk, mv;
   const int bf = dt == 1;
   if (!make_tmap(&mq, q, bf, T, (uint64_t)nq * hd, q_ld, 64, kBQ)) return -10;
   if (!make_tmap(&mk, k, bf, T, (uint64_t)nkv * hd, k_ld, 64, kBKV)) return -11;
   if (!make_tmap(&mv, v, bf, T, (uint64_t)(nkv / vshare) * hd, v_ld, 64, 64)) return -12;
   AttnParams p{cu_seqlens, out, nullptr, out_ld, T, nq, nkv, scale, 1, window > 0 ? window : 0, window > 0 ? keep : 0, temp, sink, gate, gate_ld,
-               slope_base, vshare};
-  if (hd == 128) {
-    return bf ? launch_attn_fwd<128, __nv_bfloat16, 1, true>(mq, mk, mv, p, B, max_seqlen, s)
-              : launch_attn_fwd<128, __half, 0, true>(mq, mk, mv, p, B, max_seqlen, s);
-  }
-  return bf ? launch_attn_fwd<64, __nv_bfloat16, 1, true>(mq, mk, mv, p, B, max_seqlen, s)
-            : launch_attn_fwd<64, __half, 0, true>(mq, mk, mv, p, B, max_seqlen, s);
+               slope_base, vshare, gate_mode, chunk, softcap};
+#define RB_GO(CAP)                                                                                                \
+  if (hd == 128)                                                                                                  \
+    return bf ? launch_attn_fwd<128, __nv_bfloat16, 1, true, CAP>(mq, mk, mv, p, B, max_seqlen, s)               \
+              : launch_attn_fwd<128, __half, 0, true, CAP>(mq, mk, mv, p, B, max_seqlen, s);                      \
+  return bf ? launch_attn_fwd<64, __nv_bfloat16, 1, true, CAP>(mq, mk, mv, p, B, max_seqlen, s)                  \
+            : launch_attn_fwd<64, __half, 0, true, CAP>(mq, mk, mv, p, B, max_seqlen, s)
+  if (softcap > 0.f) { RB_GO(true); }
+  RB_GO(false);
+#undef RB_GO
 }

@@ -36,10 +36,11 @@ int rb_mlstm_scan(const void*, int64_t, int, const void*, float*, float*, const 
                   float, int, cudaStream_t);
 int rb_mlstm_out(const float*, const float*, const void*, int, const void*, int64_t, int, void*, int, int64_t, int, int, float, cudaStream_t);
 int rb_latent_rope_prepare(const void*, int64_t, int, const void*, const void*, const float*, float, const int*, const int*, const int*, const int*,
-                           const int*, void*, void*, void*, int64_t, int, int, int, int, float, cudaStream_t);
+                           const int*, void*, void*, void*, int64_t, int, int, int, int, int, float, cudaStream_t);
 int rb_latent_rope_assemble(const void*, int64_t, const void*, int64_t, const void*, int64_t, int, const int*, const float*, float, void*, int, int64_t,
-                            int, int, int, cudaStream_t);
-int rb_latent_query_rope(const void*, int64_t, int, const int*, const int*, const float*, float, float, float*, int, int, int, int, int, cudaStream_t);
+                            int, int, int, int, cudaStream_t);
+int rb_latent_query_rope(const void*, int64_t, int, const int*, const int*, const float*, float, float, float*, int, int, int, int, int, int, cudaStream_t);
+int rb_latent_out(const float*, const void*, int64_t, int, int, void*, int, int, int, cudaStream_t);
 int rb_sigmoid_gate(void*, int, const void*, int64_t, int, int64_t, int, cudaStream_t);
 int rb_softmax_router(const void*, int64_t, int, const void*, int, const void*, int, const void*, int, float*, int64_t*, float*, int64_t, int, int, int,
                       int, int, cudaStream_t);
@@ -48,7 +49,7 @@ int rb_moe_combine(const void*, int, const void*, int64_t, int, const int64_t*, 
 int rb_moe_dispatch(const int64_t*, int64_t*, int*, int, int, int, cudaStream_t);
 int rb_moe_gather(const void*, int64_t, int, const int64_t*, const float*, void*, int64_t, int, int, cudaStream_t);
 int rb_centred_norm(void*, int, const void*, int64_t, const void*, int64_t, int, float, float, const void*, const void*, const void*, int, float, void*,
-                    int, int64_t, int, float, cudaStream_t);
+                    int, int64_t, int, float, int, int, const void*, int64_t, int, cudaStream_t);
 int rb_rotate_heads(void*, int64_t, int, const int*, const int*, const int*, const float*, int64_t, int, int, int, int, cudaStream_t);
 int rb_decay_prepare(const void*, int64_t, int, float*, const int*, const int*, const int*, const float*, int64_t, int, int, int, int, int, int, float,
                      cudaStream_t);
@@ -106,7 +107,7 @@ void mlstm_out(const Tensor& o, const Tensor& m, const Tensor& w, const Tensor& 
 // pos given: packed form (cache / tok_slot / remain optional); pos absent: step form (position lens[slot], the cache row is written)
 void latent_rope_prepare(const Tensor& proj, const OptT& wq, const Tensor& wc, const Tensor& inv_freq, double mscale, const OptT& pos, const OptT& lens,
                          const OptT& slots, const OptT& tok_slot, const OptT& remain, const OptT& cq, const OptT& lat, const OptT& cache, int64_t q_rank,
-                         int64_t r, int64_t rot, double eps) {
+                         int64_t r, int64_t rot, double eps, bool inter) {
   CHECK_ROWS(proj); CHECK_IN(wc); CHECK_IN(inv_freq);
   const int64_t T = proj.size(0);
   TORCH_CHECK(proj.size(1) >= q_rank + r + rot && wc.numel() == r && wc.scalar_type() == proj.scalar_type());
@@ -139,12 +140,12 @@ void latent_rope_prepare(const Tensor& proj, const OptT& wq, const Tensor& wc, c
                                         pos.has_value() ? nullptr : int_ptr(slots, T, "slots"),
                                         cachep && pos.has_value() ? int_ptr(tok_slot, T, "tok_slot") : nullptr,
                                         cachep && pos.has_value() ? int_ptr(remain, T, "remain") : nullptr, cqp, latp, cachep, T, (int)q_rank, (int)r,
-                                        (int)rot, R, (float)eps, cur_stream());
+                                        (int)rot, R, inter ? 1 : 0, (float)eps, cur_stream());
   TORCH_CHECK(rc == 0, "latent_rope_prepare: unsupported shape (rc ", rc, ")");
 }
 
 void latent_rope_assemble(const Tensor& q, const Tensor& kn, const Tensor& lat, const Tensor& pos, const Tensor& inv_freq, double mscale, Tensor out,
-                          int64_t H, int64_t d, int64_t rot, int64_t r) {
+                          int64_t H, int64_t d, int64_t rot, int64_t r, bool inter) {
   CHECK_ROWS(q); CHECK_ROWS(kn); CHECK_ROWS(lat); CHECK_IN(pos); CHECK_IN(inv_freq); CHECK_IN(out);
   const int64_t T = q.size(0);
   TORCH_CHECK(q.size(1) >= H * (d + rot) && kn.size(1) >= H * d && lat.size(1) >= r + rot && out.numel() == T * 2 * H * (d + rot));
@@ -153,12 +154,12 @@ void latent_rope_assemble(const Tensor& q, const Tensor& kn, const Tensor& lat, 
   c10::cuda::CUDAGuard g(q.device());
   TORCH_CHECK(rb_latent_rope_assemble(q.data_ptr(), q.stride(0), kn.data_ptr(), kn.stride(0), lat.data_ptr(), lat.stride(0), (int)r,
                                       int_ptr(pos, T, "pos"), inv_freq.data_ptr<float>(), (float)mscale, out.data_ptr(), dt_code(q), T, (int)H, (int)d,
-                                      (int)rot, cur_stream()) == 0);
+                                      (int)rot, inter ? 1 : 0, cur_stream()) == 0);
 }
 
 // qa [H, B, r + rot] fp32: columns [r, r + rot) <- scale * rotate(q[b, h, d:])
 void latent_query_rope(const Tensor& q, const Tensor& lens, const OptT& slots, const Tensor& inv_freq, double mscale, double scale, Tensor qa,
-                       int64_t d, int64_t rot) {
+                       int64_t d, int64_t rot, bool inter) {
   CHECK_ROWS(q); CHECK_IN(lens); CHECK_IN(inv_freq); CHECK_IN(qa);
   TORCH_CHECK(qa.dim() == 3 && qa.scalar_type() == at::kFloat && qa.size(1) == q.size(0) && qa.size(2) > rot);
   const int64_t H = qa.size(0), B = qa.size(1), r = qa.size(2) - rot;
@@ -166,7 +167,21 @@ void latent_query_rope(const Tensor& q, const Tensor& lens, const OptT& slots, c
   c10::cuda::CUDAGuard g(q.device());
   TORCH_CHECK(rb_latent_query_rope(q.data_ptr(), q.stride(0), dt_code(q), int_ptr(lens, 1, "lens"), int_ptr(slots, B, "slots"),
                                    inv_freq.data_ptr<float>(), (float)mscale, (float)scale, qa.data_ptr<float>(), (int)B, (int)H, (int)d, (int)rot, (int)r,
-                                   cur_stream()) == 0);
+                                   inter ? 1 : 0, cur_stream()) == 0);
+}
+
+// o [H, B, dv] fp32 -> out [B, H * dv], times sigmoid of gate logits per head ([B, >= H]) or per element ([B, >= H * dv]) when given
+void latent_out(const Tensor& o, const OptT& gate, bool element, Tensor out) {
+  CHECK_IN(o); CHECK_IN(out);
+  TORCH_CHECK(o.dim() == 3 && o.scalar_type() == at::kFloat && out.numel() == o.numel() && out.size(0) == o.size(1));
+  const int64_t H = o.size(0), B = o.size(1), dv = o.size(2);
+  if (gate.has_value()) {
+    CHECK_ROWS((*gate));
+    TORCH_CHECK(gate->size(0) == B && gate->size(1) >= (element ? H * dv : H) && gate->scalar_type() == out.scalar_type());
+  }
+  c10::cuda::CUDAGuard g(o.device());
+  TORCH_CHECK(rb_latent_out(o.data_ptr<float>(), gate.has_value() ? gate->data_ptr() : nullptr, gate.has_value() ? gate->stride(0) : 0,
+                            gate.has_value() ? (element ? 2 : 1) : 0, dt_code(out), out.data_ptr(), (int)B, (int)H, (int)dv, cur_stream()) == 0);
 }
 
 void sigmoid_gate_(Tensor x, const Tensor& gate) {
@@ -256,15 +271,18 @@ Tensor moe_gather(const Tensor& x, const Tensor& row, int64_t k, const OptT& sca
   return xs;
 }
 
-// "layer" stacks (centred_norm.cu): res += mult * scale * LN(a y + b y2) * w_post, out = LN(res or the branch) * w_next
+// wrapped stacks (centred_norm.cu): res += mult * scale * N((a y + b y2) * sigmoid(gate)) * w_post, out = N(res or the branch) * w_next; N is
+// LayerNorm, or with `rms` RMSNorm; w_post / w_next are vectors or have one element
 void centred_norm(const OptT& res, const Tensor& y, const OptT& y2, double a, double b, const OptT& w_post, const OptT& scale, double mult,
-                  const OptT& w_next, const OptT& out, double eps) {
+                  const OptT& w_next, const OptT& out, double eps, bool rms, const OptT& gate) {
   CHECK_ROWS(y);
   const int64_t T = y.size(0), W = y.size(1);
   const Tensor* wv = w_post.has_value() ? &*w_post : (w_next.has_value() ? &*w_next : nullptr);
   TORCH_CHECK(wv != nullptr && w_next.has_value() == out.has_value() && (res.has_value() || out.has_value()), "centred_norm: arguments");
+  const bool w_one = wv->numel() == 1;
   for (const OptT* o : {&w_post, &scale, &w_next})
-    if (o->has_value()) { CHECK_IN((**o)); TORCH_CHECK((*o)->numel() == W && (*o)->scalar_type() == wv->scalar_type()); }
+    if (o->has_value()) { CHECK_IN((**o)); TORCH_CHECK((*o)->numel() == (w_one && o != &scale ? 1 : W) && (*o)->scalar_type() == wv->scalar_type()); }
+  if (gate.has_value()) { CHECK_ROWS((*gate)); TORCH_CHECK(gate->size(0) == T && gate->size(1) == W); }
   if (res.has_value()) { CHECK_IN((*res)); TORCH_CHECK(res->numel() == T * W && w_post.has_value()); }
   if (y2.has_value()) { CHECK_ROWS((*y2)); TORCH_CHECK(y2->size(0) == T && y2->size(1) == W && y2->scalar_type() == y.scalar_type()); }
   if (out.has_value()) { CHECK_IN((*out)); TORCH_CHECK(out->numel() == T * W); }
@@ -274,7 +292,8 @@ void centred_norm(const OptT& res, const Tensor& y, const OptT& y2, double a, do
                               w_post.has_value() ? w_post->data_ptr() : nullptr, scale.has_value() ? scale->data_ptr() : nullptr,
                               w_next.has_value() ? w_next->data_ptr() : nullptr, dt_code(*wv), (float)mult,
                               out.has_value() ? out->data_ptr() : nullptr, out.has_value() ? dt_code(*out) : 0, T, (int)W, (float)eps,
-                              cur_stream()) == 0);
+                              rms ? 1 : 0, w_one ? 1 : 0, gate.has_value() ? gate->data_ptr() : nullptr, gate.has_value() ? gate->stride(0) : 0,
+                              gate.has_value() ? dt_code(*gate) : 0, cur_stream()) == 0);
 }
 
 // in place: the n_h heads of size d at the start of every row of x turn by the row's position (decay.cu)
@@ -352,15 +371,16 @@ void decay_out(const Tensor& o, const OptT& w, const Tensor& gate, Tensor out, d
 void register_mix_ops(torch::Library& m) {
   m.def("mlstm_scan(Tensor proj, Tensor gate_bias, Tensor(a!) o, Tensor(b!) m_out, Tensor? cu, Tensor(c!)? state, Tensor(d!)? m_state, Tensor? slots, int H, int d, int dv, float cap, bool load_state) -> ()", &mlstm_scan);
   m.def("mlstm_out(Tensor o, Tensor m, Tensor w, Tensor gate, Tensor(a!) out, float eps) -> ()", &mlstm_out);
-  m.def("latent_rope_prepare(Tensor proj, Tensor? wq, Tensor wc, Tensor inv_freq, float mscale, Tensor? pos, Tensor? lens, Tensor? slots, Tensor? tok_slot, Tensor? remain, Tensor(a!)? cq, Tensor(b!)? lat, Tensor(c!)? cache, int q_rank, int r, int rot, float eps) -> ()", &latent_rope_prepare);
-  m.def("latent_rope_assemble(Tensor q, Tensor kn, Tensor lat, Tensor pos, Tensor inv_freq, float mscale, Tensor(a!) out, int H, int d, int rot, int r) -> ()", &latent_rope_assemble);
-  m.def("latent_query_rope(Tensor q, Tensor lens, Tensor? slots, Tensor inv_freq, float mscale, float scale, Tensor(a!) qa, int d, int rot) -> ()", &latent_query_rope);
+  m.def("latent_rope_prepare(Tensor proj, Tensor? wq, Tensor wc, Tensor inv_freq, float mscale, Tensor? pos, Tensor? lens, Tensor? slots, Tensor? tok_slot, Tensor? remain, Tensor(a!)? cq, Tensor(b!)? lat, Tensor(c!)? cache, int q_rank, int r, int rot, float eps, bool inter=True) -> ()", &latent_rope_prepare);
+  m.def("latent_rope_assemble(Tensor q, Tensor kn, Tensor lat, Tensor pos, Tensor inv_freq, float mscale, Tensor(a!) out, int H, int d, int rot, int r, bool inter=True) -> ()", &latent_rope_assemble);
+  m.def("latent_query_rope(Tensor q, Tensor lens, Tensor? slots, Tensor inv_freq, float mscale, float scale, Tensor(a!) qa, int d, int rot, bool inter=True) -> ()", &latent_query_rope);
+  m.def("latent_out(Tensor o, Tensor? gate, bool element, Tensor(a!) out) -> ()", &latent_out);
   m.def("sigmoid_gate_(Tensor(a!) x, Tensor gate) -> ()", &sigmoid_gate_);
   m.def("moe_dispatch(Tensor idx, int E, int R) -> Tensor[]", &moe_dispatch);
   m.def("moe_gather(Tensor x, Tensor row, int k, Tensor? scale=None) -> Tensor", &moe_gather);
   m.def("softmax_router(Tensor x, Tensor w, Tensor? corr, Tensor? u, int k, bool renorm, bool sigmoid=False) -> Tensor[]", &softmax_router);
   m.def("moe_combine(Tensor y, Tensor x, Tensor row, Tensor probs, Tensor idx, Tensor? y_shared, Tensor? gate, Tensor(a!) out, int E, bool unit=False) -> ()", &moe_combine);
-  m.def("centred_norm(Tensor(a!)? res, Tensor y, Tensor? y2, float a, float b, Tensor? w_post, Tensor? scale, float mult, Tensor? w_next, Tensor(b!)? out, float eps) -> ()", &centred_norm);
+  m.def("centred_norm(Tensor(a!)? res, Tensor y, Tensor? y2, float a, float b, Tensor? w_post, Tensor? scale, float mult, Tensor? w_next, Tensor(b!)? out, float eps, bool rms=False, Tensor? gate=None) -> ()", &centred_norm);
   m.def("rotate_heads_(Tensor(a!) x, Tensor? pos, Tensor? lens, Tensor? slots, Tensor inv_freq, int n_h, int d, int dims, bool interleaved) -> ()", &rotate_heads_);
   m.def("decay_prepare(Tensor proj, Tensor(a!) u, Tensor? pos, Tensor? lens, Tensor? slots, Tensor? inv_freq, int H, int d, int dv, int dims, bool interleaved, bool silu, float k_scale) -> ()", &decay_prepare);
   m.def("decay_scan(Tensor u, Tensor decay, Tensor(a!) o, Tensor? cu, Tensor(b!)? state, Tensor? slots, int H, int d, int dv, bool load_state) -> ()", &decay_scan);

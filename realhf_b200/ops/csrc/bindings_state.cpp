@@ -40,17 +40,22 @@ extern "C" {
 int rb_embed_sinusoid(const int64_t*, const void*, int, const int*, const int*, const float*, float*, int64_t, int, int, cudaStream_t);
 int rb_concat_cast(const void*, int, int, const void*, int, int, void*, int, int64_t, cudaStream_t);
 int rb_relu2(const void*, void*, int, int64_t, cudaStream_t);
+int rb_relu2_cols(void*, int, int64_t, int, int64_t, cudaStream_t);
 int rb_rms_norm_rows(void*, int, const void*, int, const void*, int, void*, int, int64_t, int, float, float, cudaStream_t);
 int rb_value_norm_store(const void*, int64_t, int, void*, void*, void*, const int*, const int*, const int*, int64_t, int, int, int, int, int, int, int,
                         float, int, cudaStream_t);
 int rb_sink_window_prefill(const void*, int64_t, const void*, void*, const void*, const void*, const int*, int, int, int, int, int, int, float, int,
-                           int, float, int, int, int, int64_t, int, cudaStream_t);
+                           int, float, const void*, int64_t, int, int, float, int, int, int64_t, int, cudaStream_t);
 int rb_sink_window_decode(const void*, int64_t, void*, const void*, const void*, void*, void*, const int*, const int*, int, int, int, int, int, int,
-                          float, int, int, float, int, int, float, int, int, int, cudaStream_t);
+                          float, int, int, float, const void*, int64_t, int, int, float, const float*, int, int, int, float, int, int, int, cudaStream_t);
 int rb_sink_window_decode_fast(const void*, int64_t, void*, const void*, const void*, void*, void*, const int*, const int*, float*, float*, int, int,
-                               int, int, int, int, float, int, int, float, int, int, float, int, int, cudaStream_t);
+                               int, int, int, int, float, int, int, float, const void*, int64_t, int, int, float, const float*, int, int, int, float, int,
+                               int, cudaStream_t);
 int rb_attn_fwd_sink(const void*, const void*, const void*, void*, const int*, int64_t, int64_t, int64_t, int64_t, int, int, int, int, int, int, float,
-                     int, int, const void*, const void*, const void*, int64_t, float, int, int, cudaStream_t);
+                     int, int, const void*, const void*, const void*, int64_t, int, int, float, float, int, int, cudaStream_t);
+int rb_window_prepare(void*, int64_t, int, const void*, const void*, const float*, const float*, const int*, const int*, const int*, const int*,
+                      const int*, void*, void*, int64_t, int, int, int, int, int, int, int, int, int, int, float, cudaStream_t);
+int rb_turn_gate(void*, int, const void*, int64_t, int, const float*, const int*, const int*, const int*, int64_t, int, int, int, int, cudaStream_t);
 int rb_delta_prepare(const void*, int64_t, int, const void*, const void*, const void*, float*, const int*, float*, const int*, const int*, const int*,
                      int64_t, int, int, int, int, int, float, cudaStream_t);
 int rb_delta_rule(const float*, float*, const int*, float*, const int*, int, int, int, int, int, int, cudaStream_t);
@@ -76,6 +81,13 @@ void concat_cast(const Tensor& a, const Tensor& b, Tensor out) {
   c10::cuda::CUDAGuard g(a.device());
   TORCH_CHECK(rb_concat_cast(a.data_ptr(), dt_code(a), (int)a.size(1), b.data_ptr(), dt_code(b), (int)b.size(1), out.data_ptr(), dt_code(out),
                              a.size(0), cur_stream()) == 0);
+}
+
+void relu2_cols_(Tensor x, int64_t n_cols) {
+  CHECK_ROWS(x);
+  TORCH_CHECK(n_cols >= 0 && n_cols <= x.size(1));
+  c10::cuda::CUDAGuard g(x.device());
+  TORCH_CHECK(rb_relu2_cols(x.data_ptr(), dt_code(x), x.stride(0), (int)n_cols, x.size(0), cur_stream()) == 0);
 }
 
 Tensor relu2(const Tensor& x) {
@@ -119,59 +131,79 @@ void value_norm_store(const Tensor& qkvg, Tensor vout, const OptT& kc, const Opt
                                   do_norm ? 1 : 0, (float)eps, (int)vshare, cur_stream()) == 0);
 }
 
+// Gate logits of an attention block: a view whose row t holds one number per head ([T, >= H], `element` false) or per output element.
+struct Gate { const void* p; int64_t ld; int mode; };
+static Gate gate_arg(const OptT& gate, bool element, const Tensor& like, int64_t T, int64_t H, int64_t dv) {
+  if (!gate.has_value()) return Gate{nullptr, 0, 0};
+  CHECK_ROWS((*gate));
+  TORCH_CHECK(gate->size(0) == T && gate->size(1) >= (element ? H * dv : H) && gate->scalar_type() == like.scalar_type(), "gate: [T, H] or [T, H * dv]");
+  return Gate{gate->data_ptr(), gate->stride(0), element ? 2 : 1};
+}
+
 void sink_window_attention(const Tensor& qkvg, const Tensor& vn, Tensor out, const OptT& temp, const OptT& sink, const Tensor& cu, int64_t max_seqlen,
-                           int64_t H, int64_t G, int64_t d, int64_t dv, double scale, int64_t window, int64_t keep, double slope_base, bool gate,
-                           int64_t vshare) {
+                           int64_t H, int64_t G, int64_t d, int64_t dv, double scale, int64_t window, int64_t keep, double slope_base,
+                           const OptT& gate, bool element_gate, int64_t chunk, double softcap, int64_t vshare) {
   // vn: rows of G / vshare value heads (any row stride); out in its own type (fp32 keeps the weighted sums unrounded)
   CHECK_ROWS(qkvg); CHECK_ROWS(vn); CHECK_IN(out); CHECK_IN(cu);
   const int64_t T = qkvg.size(0);
   TORCH_CHECK(vshare >= 1 && G % vshare == 0);
-  TORCH_CHECK(qkvg.size(1) >= H * d + G * d + (gate ? G / vshare * dv + H : 0) && vn.size(0) == T && vn.size(1) >= G / vshare * dv && out.numel() == T * H * dv);
+  TORCH_CHECK(qkvg.size(1) >= H * d + G * d && vn.size(0) == T && vn.size(1) >= G / vshare * dv && out.numel() == T * H * dv);
   TORCH_CHECK(vn.scalar_type() == qkvg.scalar_type() && cu.scalar_type() == at::kInt);
+  const Gate ga = gate_arg(gate, element_gate, qkvg, T, H, dv);
   c10::cuda::CUDAGuard g(qkvg.device());
   const int rc = rb_sink_window_prefill(qkvg.data_ptr(), qkvg.stride(0), vn.data_ptr(), out.data_ptr(), same_type_ptr(temp, qkvg, H, "temp"),
                                         same_type_ptr(sink, qkvg, H, "sink"), cu.data_ptr<int>(), (int)cu.numel() - 1, (int)max_seqlen, (int)H, (int)G,
-                                        (int)d, (int)dv, (float)scale, (int)window, (int)keep, (float)slope_base, gate ? 1 : 0, dt_code(qkvg), (int)vshare,
-                                        vn.stride(0), dt_code(out), cur_stream());
+                                        (int)d, (int)dv, (float)scale, (int)window, (int)keep, (float)slope_base, ga.p, ga.ld, ga.mode, (int)chunk,
+                                        (float)softcap, dt_code(qkvg), (int)vshare, vn.stride(0), dt_code(out), cur_stream());
   TORCH_CHECK(rc == 0, "sink_window_attention: unsupported shape (rc ", rc, ")");
 }
 
 // tensor-core form: 16-bit operands, equal query / value head size of 64 or 128
 void sink_window_attention_tc(const Tensor& qkvg, const Tensor& vn, Tensor out, const OptT& temp, const OptT& sink, const Tensor& cu, int64_t max_seqlen,
-                              int64_t H, int64_t G, int64_t d, double scale, int64_t window, int64_t keep, double slope_base, bool gate,
-                              int64_t vshare) {
+                              int64_t H, int64_t G, int64_t d, double scale, int64_t window, int64_t keep, double slope_base, const OptT& gate,
+                              bool element_gate, int64_t chunk, double softcap, int64_t vshare) {
   CHECK_ROWS(qkvg); CHECK_ROWS(vn); CHECK_IN(out); CHECK_IN(cu);
   const int64_t T = qkvg.size(0);
   TORCH_CHECK(vshare >= 1 && G % vshare == 0);
-  TORCH_CHECK(qkvg.size(1) >= H * d + G * d + (gate ? G / vshare * d + H : 0) && vn.size(0) == T && vn.size(1) >= G / vshare * d && out.numel() == T * H * d);
+  TORCH_CHECK(qkvg.size(1) >= H * d + G * d && vn.size(0) == T && vn.size(1) >= G / vshare * d && out.numel() == T * H * d);
   TORCH_CHECK(vn.scalar_type() == qkvg.scalar_type() && out.scalar_type() == qkvg.scalar_type() && cu.scalar_type() == at::kInt);
+  const Gate ga = gate_arg(gate, element_gate, qkvg, T, H, d);
   c10::cuda::CUDAGuard g(qkvg.device());
   const char* base = static_cast<const char*>(qkvg.data_ptr());
   const int es = (int)qkvg.element_size();
   const int rc = rb_attn_fwd_sink(base, base + H * d * es, vn.data_ptr(), out.data_ptr(), cu.data_ptr<int>(), qkvg.stride(0), qkvg.stride(0), vn.stride(0),
                                   H * d, (int)T, (int)cu.numel() - 1, (int)H, (int)G, (int)d, (int)max_seqlen, (float)scale, (int)window, (int)keep,
-                                  same_type_ptr(temp, qkvg, H, "temp"), same_type_ptr(sink, qkvg, H, "sink"),
-                                  gate ? base + (H * d + G * d + G / vshare * d) * es : nullptr, qkvg.stride(0), (float)slope_base, dt_code(qkvg),
-                                  (int)vshare, cur_stream());
+                                  same_type_ptr(temp, qkvg, H, "temp"), same_type_ptr(sink, qkvg, H, "sink"), ga.p, ga.ld, ga.mode, (int)chunk,
+                                  (float)softcap, (float)slope_base, dt_code(qkvg), (int)vshare, cur_stream());
   TORCH_CHECK(rc == 0, "sink_window_attention_tc: unsupported shape (rc ", rc, ")");
 }
 
+// turn_freq [turn_dims / 2] fp32: every head's output is turned back by the row's position over its first turn_dims columns (before the gate)
 void sink_window_decode_attention(const Tensor& qkvg, Tensor out, const OptT& temp, const OptT& sink, Tensor kc, Tensor vc, const Tensor& lens,
                                   const OptT& slots, int64_t H, int64_t G, int64_t d, int64_t dv, double scale, int64_t window, int64_t keep,
-                                  double slope_base, bool gate, bool do_norm, double eps, int64_t vshare) {
+                                  double slope_base, const OptT& gate, bool element_gate, int64_t chunk, double softcap, const OptT& turn_freq,
+                                  int64_t turn_dims, bool turn_inter, bool do_norm, double eps, int64_t vshare) {
   CHECK_ROWS(qkvg); CHECK_IN(out); CHECK_IN(kc); CHECK_IN(vc); CHECK_IN(lens);
   const int64_t B = qkvg.size(0);
   TORCH_CHECK(vshare >= 1 && G % vshare == 0);
   const int64_t Gv = G / vshare;
-  TORCH_CHECK(qkvg.size(1) >= H * d + G * d + Gv * dv + (gate ? H : 0) && out.numel() == B * H * dv && lens.scalar_type() == at::kInt);
+  TORCH_CHECK(qkvg.size(1) >= H * d + G * d + Gv * dv && out.numel() == B * H * dv && lens.scalar_type() == at::kInt);
   TORCH_CHECK(kc.dim() == 4 && kc.size(1) == G && kc.size(3) == d && vc.size(1) == Gv && vc.size(3) == dv && vc.size(2) == kc.size(2));
   TORCH_CHECK(kc.scalar_type() == qkvg.scalar_type() && vc.scalar_type() == qkvg.scalar_type());
   TORCH_CHECK(out.scalar_type() == qkvg.scalar_type() || out.scalar_type() == at::kFloat);
   TORCH_CHECK(slots.has_value() || kc.size(0) >= B);
+  const Gate ga = gate_arg(gate, element_gate, qkvg, B, H, dv);
+  const float* tf = nullptr;
+  if (turn_dims > 0) {
+    TORCH_CHECK(turn_freq.has_value() && turn_freq->is_cuda() && turn_freq->is_contiguous() && turn_freq->scalar_type() == at::kFloat &&
+                turn_freq->numel() >= turn_dims / 2 && turn_dims % 2 == 0 && turn_dims <= dv, "turn_freq: [turn_dims / 2] fp32");
+    tf = turn_freq->data_ptr<float>();
+  }
   c10::cuda::CUDAGuard g(qkvg.device());
   const int rep = (int)(H / G);
-  if (qkvg.scalar_type() != at::kFloat && out.scalar_type() == qkvg.scalar_type() && d == dv && (d == 64 || d == 128) && (rep == 1 || rep == 2 || rep == 4 || rep == 8) &&
-      qkvg.stride(0) % 8 == 0 && (H * d) % 8 == 0 && reinterpret_cast<uintptr_t>(qkvg.data_ptr()) % 16 == 0) {
+  if (qkvg.scalar_type() != at::kFloat && out.scalar_type() == qkvg.scalar_type() && d == dv && (d == 64 || d == 128) &&
+      (rep == 1 || rep == 2 || rep == 3 || rep == 4 || rep == 6 || rep == 8) && qkvg.stride(0) % 8 == 0 && (H * d) % 8 == 0 &&
+      reinterpret_cast<uintptr_t>(qkvg.data_ptr()) % 16 == 0) {
     // enough CTAs for two per SM, at least 128 keys per split (the cache's row count bounds the visible keys).  Measured at 32 rows x
     // 4 kv heads x 576 keys with a cold L2: 65 us with 3 splits + merge, 74 us as one split
     const int64_t rows = kc.size(2);
@@ -186,15 +218,63 @@ void sink_window_decode_attention(const Tensor& qkvg, Tensor out, const OptT& te
                                                same_type_ptr(sink, qkvg, H, "sink"), kc.data_ptr(), vc.data_ptr(), lens.data_ptr<int>(),
                                                int_ptr(slots, B, "slots"), splits > 1 ? pa.data_ptr<float>() : nullptr,
                                                splits > 1 ? pm.data_ptr<float>() : nullptr, splits, (int)B, (int)H, (int)G, (int)d, (int)rows, (float)scale,
-                                               (int)window, (int)keep, (float)slope_base, gate ? 1 : 0, do_norm ? 1 : 0, (float)eps, dt_code(qkvg),
-                                               (int)vshare, cur_stream());
+                                               (int)window, (int)keep, (float)slope_base, ga.p, ga.ld, ga.mode, (int)chunk, (float)softcap, tf,
+                                               (int)turn_dims, turn_inter ? 1 : 0, do_norm ? 1 : 0, (float)eps, dt_code(qkvg), (int)vshare, cur_stream());
     if (rcf == 0) return;
   }
   const int rc = rb_sink_window_decode(qkvg.data_ptr(), qkvg.stride(0), out.data_ptr(), same_type_ptr(temp, qkvg, H, "temp"),
                                        same_type_ptr(sink, qkvg, H, "sink"), kc.data_ptr(), vc.data_ptr(), lens.data_ptr<int>(), int_ptr(slots, B, "slots"),
                                        (int)B, (int)H, (int)G, (int)d, (int)dv, (int)kc.size(2), (float)scale, (int)window, (int)keep, (float)slope_base,
-                                       gate ? 1 : 0, do_norm ? 1 : 0, (float)eps, dt_code(qkvg), (int)vshare, dt_code(out), cur_stream());
+                                       ga.p, ga.ld, ga.mode, (int)chunk, (float)softcap, tf, (int)turn_dims, turn_inter ? 1 : 0, do_norm ? 1 : 0,
+                                       (float)eps, dt_code(qkvg), (int)vshare, dt_code(out), cur_stream());
   TORCH_CHECK(rc == 0, "sink_window_decode_attention: unsupported shape (rc ", rc, ")");
+}
+
+// window_prepare.cu: query / key norm over all heads (wq, wk optional), rotation of q and k (q_freq, dims) and of v (v_freq, vdims) in
+// place; with caches (packed form) the rows a later decode step can still see are stored
+void window_prepare_(Tensor qkv, const OptT& wq, const OptT& wk, const OptT& q_freq, const OptT& v_freq, const OptT& pos, const OptT& lens,
+                     const OptT& slots, const OptT& kc, const OptT& vc, const OptT& tok_slot, const OptT& remain, int64_t H, int64_t G, int64_t d,
+                     int64_t dv, int64_t dims, bool inter, int64_t vdims, bool vinter, int64_t keep, double eps) {
+  CHECK_ROWS(qkv);
+  const int64_t T = qkv.size(0);
+  TORCH_CHECK(qkv.size(1) >= (H + G) * d + G * dv && (pos.has_value() || lens.has_value()) && wq.has_value() == wk.has_value());
+  auto freq = [](const OptT& t, int64_t n) -> const float* {
+    if (n == 0) return nullptr;
+    TORCH_CHECK(t.has_value() && t->is_cuda() && t->is_contiguous() && t->scalar_type() == at::kFloat && t->numel() >= n / 2 && n % 2 == 0, "frequencies");
+    return t->data_ptr<float>();
+  };
+  int rows = 1;
+  void *kp = nullptr, *vp = nullptr;
+  if (kc.has_value()) {
+    CHECK_IN((*kc)); CHECK_IN((*vc));
+    TORCH_CHECK(kc->dim() == 4 && kc->size(1) == G && kc->size(3) == d && vc->size(1) == G && vc->size(3) == dv && vc->size(2) == kc->size(2));
+    TORCH_CHECK(kc->scalar_type() == qkv.scalar_type() && vc->scalar_type() == qkv.scalar_type() && pos.has_value() && tok_slot.has_value() && remain.has_value());
+    rows = kc->size(2); kp = kc->data_ptr(); vp = vc->data_ptr();
+  }
+  c10::cuda::CUDAGuard g(qkv.device());
+  const int rc = rb_window_prepare(qkv.data_ptr(), qkv.stride(0), dt_code(qkv), same_type_ptr(wq, qkv, H * d, "wq"), same_type_ptr(wk, qkv, G * d, "wk"),
+                                   freq(q_freq, dims), freq(v_freq, vdims), int_ptr(pos, T, "pos"), pos.has_value() ? nullptr : int_ptr(lens, 1, "lens"),
+                                   pos.has_value() ? nullptr : int_ptr(slots, T, "slots"), kp ? int_ptr(tok_slot, T, "tok_slot") : nullptr,
+                                   kp ? int_ptr(remain, T, "remain") : nullptr, kp, vp, T, (int)H, (int)G, (int)d, (int)dv, (int)dims, inter ? 1 : 0,
+                                   (int)vdims, vinter ? 1 : 0, (int)keep, rows, (float)eps, cur_stream());
+  TORCH_CHECK(rc == 0, "window_prepare_: unsupported shape (rc ", rc, ")");
+}
+
+// x [T, H * dv] in place: every head turned back by the row's position over its first `dims` columns, then times sigmoid(gate)
+void turn_gate_(Tensor x, const OptT& gate, bool element_gate, const OptT& v_freq, const OptT& pos, const OptT& lens, const OptT& slots, int64_t H,
+                int64_t dv, int64_t dims, bool inter) {
+  CHECK_IN(x);
+  const int64_t T = x.size(0);
+  TORCH_CHECK(x.numel() == T * H * dv && dims % 2 == 0 && dims <= dv && (pos.has_value() || lens.has_value()));
+  const Gate ga = gate_arg(gate, element_gate, x, T, H, dv);
+  const float* tf = nullptr;
+  if (dims > 0) {
+    TORCH_CHECK(v_freq.has_value() && v_freq->is_cuda() && v_freq->is_contiguous() && v_freq->scalar_type() == at::kFloat && v_freq->numel() >= dims / 2);
+    tf = v_freq->data_ptr<float>();
+  }
+  c10::cuda::CUDAGuard g(x.device());
+  TORCH_CHECK(rb_turn_gate(x.data_ptr(), dt_code(x), ga.p, ga.ld, ga.mode, tf, int_ptr(pos, T, "pos"), pos.has_value() ? nullptr : int_ptr(lens, 1, "lens"),
+                           pos.has_value() ? nullptr : int_ptr(slots, T, "slots"), T, (int)H, (int)dv, (int)dims, inter ? 1 : 0, cur_stream()) == 0);
 }
 
 // pos given: packed form (conv_state / tok_slot / remain optional); pos absent: step form (conv_state indexed by slots or row)
@@ -266,11 +346,14 @@ void register_state_ops(torch::Library& m) {
   m.def("embed_sinusoid(Tensor ids, Tensor wte, Tensor pos, Tensor? slots, Tensor inv_freq, Tensor(a!) out) -> ()", &embed_sinusoid);
   m.def("concat_cast(Tensor a, Tensor b, Tensor(a!) out) -> ()", &concat_cast);
   m.def("relu2(Tensor x) -> Tensor", &relu2);
+  m.def("relu2_cols_(Tensor(a!) x, int n_cols) -> ()", &relu2_cols_);
   m.def("rms_norm_rows(Tensor(a!) x, Tensor? y, Tensor w, Tensor(b!) out, float eps, float w_offset=0.0) -> ()", &rms_norm_rows);
   m.def("value_norm_store(Tensor qkvg, Tensor(a!) vout, Tensor(b!)? kc, Tensor(c!)? vc, Tensor? tok_slot, Tensor pos, Tensor? remain, int H, int G, int d, int dv, int keep, bool do_norm, float eps, int vshare=1) -> ()", &value_norm_store);
-  m.def("sink_window_attention(Tensor qkvg, Tensor vn, Tensor(a!) out, Tensor? temp, Tensor? sink, Tensor cu, int max_seqlen, int H, int G, int d, int dv, float scale, int window, int keep, float slope_base, bool gate, int vshare=1) -> ()", &sink_window_attention);
-  m.def("sink_window_attention_tc(Tensor qkvg, Tensor vn, Tensor(a!) out, Tensor? temp, Tensor? sink, Tensor cu, int max_seqlen, int H, int G, int d, float scale, int window, int keep, float slope_base, bool gate, int vshare=1) -> ()", &sink_window_attention_tc);
-  m.def("sink_window_decode_attention(Tensor qkvg, Tensor(a!) out, Tensor? temp, Tensor? sink, Tensor(b!) kc, Tensor(c!) vc, Tensor lens, Tensor? slots, int H, int G, int d, int dv, float scale, int window, int keep, float slope_base, bool gate, bool do_norm, float eps, int vshare=1) -> ()", &sink_window_decode_attention);
+  m.def("sink_window_attention(Tensor qkvg, Tensor vn, Tensor(a!) out, Tensor? temp, Tensor? sink, Tensor cu, int max_seqlen, int H, int G, int d, int dv, float scale, int window, int keep, float slope_base, Tensor? gate=None, bool element_gate=False, int chunk=0, float softcap=0.0, int vshare=1) -> ()", &sink_window_attention);
+  m.def("sink_window_attention_tc(Tensor qkvg, Tensor vn, Tensor(a!) out, Tensor? temp, Tensor? sink, Tensor cu, int max_seqlen, int H, int G, int d, float scale, int window, int keep, float slope_base, Tensor? gate=None, bool element_gate=False, int chunk=0, float softcap=0.0, int vshare=1) -> ()", &sink_window_attention_tc);
+  m.def("sink_window_decode_attention(Tensor qkvg, Tensor(a!) out, Tensor? temp, Tensor? sink, Tensor(b!) kc, Tensor(c!) vc, Tensor lens, Tensor? slots, int H, int G, int d, int dv, float scale, int window, int keep, float slope_base, Tensor? gate, bool element_gate, int chunk, float softcap, Tensor? turn_freq, int turn_dims, bool turn_inter, bool do_norm, float eps, int vshare=1) -> ()", &sink_window_decode_attention);
+  m.def("window_prepare_(Tensor(a!) qkv, Tensor? wq, Tensor? wk, Tensor? q_freq, Tensor? v_freq, Tensor? pos, Tensor? lens, Tensor? slots, Tensor(b!)? kc, Tensor(c!)? vc, Tensor? tok_slot, Tensor? remain, int H, int G, int d, int dv, int dims, bool inter, int vdims, bool vinter, int keep, float eps) -> ()", &window_prepare_);
+  m.def("turn_gate_(Tensor(a!) x, Tensor? gate, bool element_gate, Tensor? v_freq, Tensor? pos, Tensor? lens, Tensor? slots, int H, int dv, int dims, bool inter) -> ()", &turn_gate_);
   m.def("delta_prepare(Tensor proj, Tensor conv_w, Tensor A_log, Tensor dt_bias, Tensor(a!) u, Tensor? pos, Tensor(b!)? conv_state, Tensor? tok_slot, Tensor? remain, Tensor? slots, int H, int G, int d, int dv, int taps, float unit_eps) -> ()", &delta_prepare);
   m.def("delta_rule_scan(Tensor u, Tensor(a!) o, Tensor cu, Tensor(b!)? s_state, Tensor? slots, int H, int G, int d, int dv) -> ()", &delta_rule_scan);
   m.def("delta_rule_step(Tensor u, Tensor(a!) o, Tensor(b!) s_state, Tensor? slots, int H, int G, int d, int dv) -> ()", &delta_rule_step);

@@ -38,6 +38,7 @@ struct Params {
   float glu_alpha;
   // optional unary activation on the plain (non-GLU) epilogue of the 2-CTA kernel, after the bias: 0 none, 1 relu(x)^2
   int unary_act;
+  int act_cols;            // unary_act applies to output columns below this
 };
 
 template <typename T> RB_DEVICE void store_chunk(T* dst, const float* v, int n_valid, bool vec_ok);

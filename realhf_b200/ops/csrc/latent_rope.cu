@@ -1,7 +1,7 @@
 // Latent attention with a rotated key part (`LatentAttentionConfig` with `rot_dim` > 0): the row a token leaves in the cache is
 // [c | k_rot], c = RMSNorm(latent) * w of rank r and k_rot the rotated `rot` last outputs of the down-projection, shared by all
-// heads.  Queries may pass a normalised latent of their own (q_rank > 0).  Rotation: pair (2i, 2i + 1) turns by the angle
-// pos * f_i (fp32 product, sincosf), cos and sin times `mscale`; the frequency table f (with any rescaling of long contexts already
+// heads.  Queries may pass a normalised latent of their own (q_rank > 0).  Rotation: pair (2i, 2i + 1), or (i, i + rot / 2) in the half
+// layout (inter 0), turns by the angle pos * f_i (fp32 product, sincosf), cos and sin times `mscale`; the frequency table f (with any rescaling of long contexts already
 // applied) comes from the host.  All arithmetic is fp32; storage types by run-time code (anytype.cuh).
 //
 //   latent_rope_prepare    one CTA per token: cq = RMSNorm(proj[:, :q_rank]) * w_q -> [T, q_rank]; [c | k_rot] -> packed
@@ -10,6 +10,7 @@
 //   latent_rope_assemble   one CTA per token: q [T, H (d + rot)] with its rotated part turned, and per head the key
 //                          [k_nope_h | k_rot] -> one tensor [T, 2 H (d + rot)] = [queries | keys] for the packed attention kernel.
 //   latent_query_rope      decode: scale * rotate(q_rot) -> columns [r, r + rot) of the absorbed query [H, B, r + rot] fp32.
+//   latent_out             decode: per-head results [H, B, dv] fp32 -> [B, H dv] in the storage type, times a sigmoid gate per head or element.
 //   sigmoid_gate_          out[t, c] *= sigmoid(g[t, c]).
 #include "anytype.cuh"
 
@@ -28,9 +29,13 @@ struct PrepParams {
   void* cq;                                // [T, q_rank] or null
   void* lat;                               // [T, r + rot] or null
   void* cache;                             // [n_slots, R, r + rot] or null
-  int q_rank, r, rot, R;
+  int q_rank, r, rot, R, inter;
   float eps;
 };
+
+// the two elements of pair i of a rotated part of `rot` dimensions
+RB_DEVICE int pair_first(int i, int inter) { return inter ? 2 * i : i; }
+RB_DEVICE int pair_second(int i, int rot, int inter) { return inter ? 2 * i + 1 : i + rot / 2; }
 
 __global__ void __launch_bounds__(128) latent_rope_prepare_kernel(PrepParams p) {
   __shared__ float red[32];
@@ -73,17 +78,18 @@ __global__ void __launch_bounds__(128) latent_rope_prepare_kernel(PrepParams p) 
     float sn, cs;
     sincosf(fp * p.inv_freq[i], &sn, &cs);
     sn *= p.mscale; cs *= p.mscale;
-    const float u = ld_any(p.proj, dt, cb + p.r + 2 * i), v = ld_any(p.proj, dt, cb + p.r + 2 * i + 1);
+    const int e0 = p.r + pair_first(i, p.inter), e1 = p.r + pair_second(i, p.rot, p.inter);
+    const float u = ld_any(p.proj, dt, cb + e0), v = ld_any(p.proj, dt, cb + e1);
     const float a = u * cs - v * sn, b = v * cs + u * sn;
-    if (p.lat) { st_any(p.lat, dt, t * w + p.r + 2 * i, a); st_any(p.lat, dt, t * w + p.r + 2 * i + 1, b); }
-    if (crow >= 0) { st_any(p.cache, dt, crow * w + p.r + 2 * i, a); st_any(p.cache, dt, crow * w + p.r + 2 * i + 1, b); }
+    if (p.lat) { st_any(p.lat, dt, t * w + e0, a); st_any(p.lat, dt, t * w + e1, b); }
+    if (crow >= 0) { st_any(p.cache, dt, crow * w + e0, a); st_any(p.cache, dt, crow * w + e1, b); }
   }
 }
 
 __global__ void __launch_bounds__(256) latent_rope_assemble_kernel(const void* __restrict__ q, int64_t ldq, const void* __restrict__ kn, int64_t ldk,
                                                                     const void* __restrict__ lat, int64_t ldl, int r, const int* __restrict__ pos,
                                                                     const float* __restrict__ inv_freq, float mscale, void* __restrict__ out, int dt,
-                                                                    int H, int d, int rot) {
+                                                                    int H, int d, int rot, int inter) {
   const int64_t t = blockIdx.x;
   const int dq = d + rot;
   rb::pdl_trigger();
@@ -96,15 +102,16 @@ __global__ void __launch_bounds__(256) latent_rope_assemble_kernel(const void* _
       st_any(out, dt, ob + idx, ld_any(q, dt, t * ldq + idx));
       st_any(out, dt, ob + H * dq + idx, ld_any(kn, dt, t * ldk + h * d + e));
     } else {
-      const int j = e - d, i = j >> 1;
+      const int j = e - d;
       st_any(out, dt, ob + H * dq + idx, ld_any(lat, dt, t * ldl + r + j));
-      if ((j & 1) == 0) {
+      if (inter ? (j & 1) == 0 : j < rot / 2) {         // the pair's first element does both
+        const int i = inter ? j >> 1 : j, step = inter ? 1 : rot / 2;
         float sn, cs;
         sincosf(fp * inv_freq[i], &sn, &cs);
         sn *= mscale; cs *= mscale;
-        const float u = ld_any(q, dt, t * ldq + idx), v = ld_any(q, dt, t * ldq + idx + 1);
+        const float u = ld_any(q, dt, t * ldq + idx), v = ld_any(q, dt, t * ldq + idx + step);
         st_any(out, dt, ob + idx, u * cs - v * sn);
-        st_any(out, dt, ob + idx + 1, v * cs + u * sn);
+        st_any(out, dt, ob + idx + step, v * cs + u * sn);
       }
     }
   }
@@ -112,7 +119,7 @@ __global__ void __launch_bounds__(256) latent_rope_assemble_kernel(const void* _
 
 __global__ void __launch_bounds__(128) latent_query_rope_kernel(const void* __restrict__ q, int64_t ldq, int dt, const int* __restrict__ lens,
                                                                  const int* __restrict__ slots, const float* __restrict__ inv_freq, float mscale,
-                                                                 float scale, float* __restrict__ qa, int B, int H, int d, int rot, int r) {
+                                                                 float scale, float* __restrict__ qa, int B, int H, int d, int rot, int r, int inter) {
   const int b = blockIdx.x;
   rb::pdl_trigger();
   rb::pdl_wait();
@@ -123,12 +130,28 @@ __global__ void __launch_bounds__(128) latent_query_rope_kernel(const void* __re
     float sn, cs;
     sincosf(fp * inv_freq[i], &sn, &cs);
     sn *= mscale; cs *= mscale;
-    const int64_t src = (int64_t)b * ldq + h * dq + d + 2 * i;
-    const float u = ld_any(q, dt, src), v = ld_any(q, dt, src + 1);
-    float* dst = qa + ((int64_t)h * B + b) * w + r + 2 * i;
+    const int step = inter ? 1 : rot / 2;
+    const int64_t src = (int64_t)b * ldq + h * dq + d + pair_first(i, inter);
+    const float u = ld_any(q, dt, src), v = ld_any(q, dt, src + step);
+    float* dst = qa + ((int64_t)h * B + b) * w + r + pair_first(i, inter);
     dst[0] = (u * cs - v * sn) * scale;
-    dst[1] = (v * cs + u * sn) * scale;
+    dst[step] = (v * cs + u * sn) * scale;
   }
+}
+
+__global__ void __launch_bounds__(256) latent_out_kernel(const float* __restrict__ o, const void* __restrict__ gate, int64_t ldg, int gmode, int dt,
+                                                         void* __restrict__ out, int B, int H, int dv) {
+  const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  rb::pdl_trigger();
+  rb::pdl_wait();
+  if (idx >= (int64_t)B * H * dv) return;
+  const int c = (int)(idx % dv);
+  const int64_t bh = idx / dv;
+  const int h = (int)(bh % H);
+  const int64_t b = bh / H;
+  float v = o[((int64_t)h * B + b) * dv + c];
+  if (gmode != 0) v /= 1.f + expf(-ld_any(gate, dt, b * ldg + (gmode == 1 ? h : h * dv + c)));
+  st_any(out, dt, idx, v);
 }
 
 __global__ void sigmoid_gate_kernel(void* __restrict__ x, int dtx, const void* __restrict__ g, int64_t ldg, int dtg, int64_t n, int W, int vec4) {
@@ -155,27 +178,34 @@ __global__ void sigmoid_gate_kernel(void* __restrict__ x, int dtx, const void* _
 
 extern "C" int rb_latent_rope_prepare(const void* proj, int64_t ld, int dt, const void* wq, const void* wc, const float* inv_freq, float mscale,
                                       const int* pos, const int* lens, const int* slots, const int* tok_slot, const int* remain, void* cq, void* lat,
-                                      void* cache, int64_t T, int q_rank, int r, int rot, int R, float eps, cudaStream_t s) {
+                                      void* cache, int64_t T, int q_rank, int r, int rot, int R, int inter, float eps, cudaStream_t s) {
   if (T == 0) return 0;
   if (rot & 1) return -1;
-  PrepParams p{proj, ld, dt, wq, wc, inv_freq, mscale, pos, lens, slots, tok_slot, remain, cq, lat, cache, q_rank, r, rot, R, eps};
+  PrepParams p{proj, ld, dt, wq, wc, inv_freq, mscale, pos, lens, slots, tok_slot, remain, cq, lat, cache, q_rank, r, rot, R, inter, eps};
   return rb::launch_pdl(latent_rope_prepare_kernel, dim3((unsigned)T), dim3(128), 0, s, p) == cudaSuccess ? 0 : 2;
 }
 
 extern "C" int rb_latent_rope_assemble(const void* q, int64_t ldq, const void* kn, int64_t ldk, const void* lat, int64_t ldl, int r, const int* pos,
-                                       const float* inv_freq, float mscale, void* out, int dt, int64_t T, int H, int d, int rot, cudaStream_t s) {
+                                       const float* inv_freq, float mscale, void* out, int dt, int64_t T, int H, int d, int rot, int inter,
+                                       cudaStream_t s) {
   if (T == 0) return 0;
   if (rot & 1) return -1;
   return rb::launch_pdl(latent_rope_assemble_kernel, dim3((unsigned)T), dim3(256), 0, s, q, ldq, kn, ldk, lat, ldl, r, pos, inv_freq, mscale, out, dt,
-                        H, d, rot) == cudaSuccess ? 0 : 2;
+                        H, d, rot, inter) == cudaSuccess ? 0 : 2;
 }
 
 extern "C" int rb_latent_query_rope(const void* q, int64_t ldq, int dt, const int* lens, const int* slots, const float* inv_freq, float mscale,
-                                    float scale, float* qa, int B, int H, int d, int rot, int r, cudaStream_t s) {
+                                    float scale, float* qa, int B, int H, int d, int rot, int r, int inter, cudaStream_t s) {
   if (B == 0 || rot == 0) return 0;
   if (rot & 1) return -1;
   return rb::launch_pdl(latent_query_rope_kernel, dim3((unsigned)B), dim3(128), 0, s, q, ldq, dt, lens, slots, inv_freq, mscale, scale, qa, B, H, d, rot,
-                        r) == cudaSuccess ? 0 : 2;
+                        r, inter) == cudaSuccess ? 0 : 2;
+}
+
+extern "C" int rb_latent_out(const float* o, const void* gate, int64_t ldg, int gmode, int dt, void* out, int B, int H, int dv, cudaStream_t s) {
+  const int64_t n = (int64_t)B * H * dv;
+  if (n == 0) return 0;
+  return rb::launch_pdl(latent_out_kernel, dim3((unsigned)RB_CEIL_DIV(n, (int64_t)256)), dim3(256), 0, s, o, gate, ldg, gmode, dt, out, B, H, dv) == cudaSuccess ? 0 : 2;
 }
 
 extern "C" int rb_sigmoid_gate(void* x, int dtx, const void* g, int64_t ldg, int dtg, int64_t T, int W, cudaStream_t s) {

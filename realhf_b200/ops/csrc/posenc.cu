@@ -55,6 +55,23 @@ __global__ void relu2_kernel(const void* __restrict__ x, void* __restrict__ out,
   }
 }
 
+// in place on the first n_cols columns of every row (row stride ld); vec: four columns per thread
+__global__ void relu2_cols_kernel(void* __restrict__ x, int dt, int64_t ld, int n_cols, int64_t n, int vec) {
+  const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * (vec ? 4 : 1);
+  rb::pdl_trigger();
+  rb::pdl_wait();
+  if (i >= n) return;
+  const int64_t at = i / n_cols * ld + i % n_cols;
+  if (vec) {
+    float4 v = rb::ld4_any(x, dt, at);
+    v.x = fmaxf(v.x, 0.f); v.y = fmaxf(v.y, 0.f); v.z = fmaxf(v.z, 0.f); v.w = fmaxf(v.w, 0.f);
+    rb::st4_any(x, dt, at, make_float4(v.x * v.x, v.y * v.y, v.z * v.z, v.w * v.w));
+  } else {
+    const float v = fmaxf(rb::ld_any(x, dt, at), 0.f);
+    rb::st_any(x, dt, at, v * v);
+  }
+}
+
 // one CTA per row; the row is read once from DRAM (second pass from L1 / L2)
 __global__ void __launch_bounds__(256) rms_norm_rows_kernel(void* __restrict__ x, int dtx, const void* __restrict__ y, int dty,
                                                             const void* __restrict__ w, int dtw, void* __restrict__ out, int dto, int W, float eps,
@@ -113,6 +130,14 @@ extern "C" int rb_embed_sinusoid(const int64_t* ids, const void* wte, int dtw, c
 extern "C" int rb_concat_cast(const void* a, int dta, int Wa, const void* b, int dtb, int Wb, void* out, int dto, int64_t T, cudaStream_t s) {
   if (T == 0) return 0;
   return rb::launch_pdl(concat_cast_kernel, dim3((unsigned)T), dim3(256), 0, s, a, dta, Wa, b, dtb, Wb, out, dto) == cudaSuccess ? 0 : -3;
+}
+
+extern "C" int rb_relu2_cols(void* x, int dt, int64_t ld, int n_cols, int64_t T, cudaStream_t s) {
+  const int64_t n = T * n_cols;
+  if (n == 0) return 0;
+  const int vec = n_cols % 4 == 0 && ld % 4 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0;
+  const int64_t work = vec ? n / 4 : n;
+  return rb::launch_pdl(relu2_cols_kernel, dim3((unsigned)((work + 255) / 256)), dim3(256), 0, s, x, dt, ld, n_cols, n, vec) == cudaSuccess ? 0 : -3;
 }
 
 extern "C" int rb_relu2(const void* x, void* out, int dt, int64_t n, cudaStream_t s) {

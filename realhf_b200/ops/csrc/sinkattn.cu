@@ -1,9 +1,14 @@
-// Window attention with a sink (`WindowAttentionConfig`): grouped key / value heads, no rotation.
+// Window attention with a sink (`WindowAttentionConfig`): grouped key / value heads; rotated heads arrive rotated
+// (window_prepare.cu).
 //
 //   score(i, j) = q_i . k_j * scale * temp_h - slope_h * (i - j),   slope_h = 2^(-slope_base (h + 1) / H)
+//                 softcap > 0: softcap * tanh(q_i . k_j * scale * temp_h / softcap) instead
 //   visible:      j <= i and (i - j < window or j < keep_first)                (window < 0: every j <= i)
+//                 chunk > 0: j <= i and floor(j / chunk) = floor(i / chunk) instead
 //   weights:      exp(score - m) / (sum_visible exp(score - m) + exp(sink_h - m))   (the sink is a bare logit: key-less, value-less)
-//   output:       sum_j w_ij vhat_j * sigmoid(gate_h),   vhat = v / sqrt(mean(v^2) + eps) per head (cached so)
+//   output:       sum_j w_ij vhat_j * sigmoid(gate),   vhat = v / sqrt(mean(v^2) + eps) per head (cached so; do_norm);
+//                 the gate is one number per head or one per output element.  Decode forms with turn_dims > 0 first turn the head's
+//                 output back by the query's position (pair m by -n f_m), as needed when the values are cached rotated
 //
 // Everything is fp32 arithmetic whatever the storage type (a type code per launch: 0 fp32, 1 bf16, 2 fp16); exact expf (compiled
 // without fast-math).  The projection output `qkvg` [T, ld] holds [q (H x d) | k (G x d) | v (G x dv) | gate logits] per row.
@@ -29,6 +34,28 @@ using rb::st_any;
 RB_DEVICE int cache_row(int p, int keep, int rows) {
   const int ring = max(rows - keep, 1);
   return p < keep ? p : keep + (p - keep) % ring;
+}
+
+// first position of the window / chunk part that query i sees (the kept first keys come on top)
+RB_DEVICE int first_visible(int i, int window, int chunk) {
+  if (chunk > 0) return i / chunk * chunk;
+  return window < 0 ? 0 : max(0, i - window + 1);
+}
+
+// gate factor of output column col of head h: gate logits at g[row + h] (mode 1) or g[row + h * dv + col] (mode 2)
+RB_DEVICE float gate_factor(const void* g, int dt, int64_t row, int mode, int h, int dv, int col) {
+  if (mode == 0) return 1.f;
+  return 1.f / (1.f + expf(-ld_any(g, dt, row + (mode == 1 ? h : h * dv + col))));
+}
+
+// a head's output turned back by position n: the pair of column c is (c, partner); o = the column's own value, po its partner's
+RB_DEVICE int turn_partner(int c, int dims, int interleaved) { return interleaved ? c ^ 1 : (c < dims / 2 ? c + dims / 2 : c - dims / 2); }
+RB_DEVICE float turn_back(float o, float po, int c, float n, const float* inv_freq, int dims, int interleaved) {
+  const int half = dims / 2, m = interleaved ? c >> 1 : (c < half ? c : c - half);
+  const bool first = interleaved ? (c & 1) == 0 : c < half;
+  float sn, cs;
+  sincosf(n * inv_freq[m], &sn, &cs);
+  return first ? o * cs + po * sn : o * cs - po * sn;
 }
 
 // ------------------------------------------------------------------------------------------------ value norm + cache fill
@@ -77,9 +104,11 @@ struct PrefillParams {
   void* out;                 // [T, H * dv] in type dto
   const void* temp; const void* sink;   // [H] in the model type, or null
   const int* cu;             // [n_seqs + 1]
-  int H, G, d, dv, window, keep, gate, dt;
+  int H, G, d, dv, window, keep, dt;
   float scale, slope_base;
   int vshare, dto; int64_t vld;
+  const void* gate; int64_t gld; int gmode;   // gate logits (type dt): row t at gate + t * gld; mode 0 none, 1 per head, 2 per element
+  int chunk; float softcap;
 };
 
 // NJ = ceil(dv / 32): a thread owns 2 query rows x NJ float4 column groups of the output tile
@@ -118,7 +147,7 @@ __global__ void __launch_bounds__(kPfThreads) sink_window_prefill_kernel(Prefill
   }
   // key ranges of this query tile: the kept first tokens [0, ka) and the window part [lo, q_last]
   const int q_last = q0 + nq - 1;
-  const int lo = p.window < 0 ? 0 : max(0, q0 - p.window + 1);
+  const int lo = first_visible(q0, p.window, p.chunk);
   const int ka = p.window < 0 ? 0 : min(p.keep, lo);
   const int lo_al = lo / BK * BK;                       // window tiles start on a tile border
   const int n_keep_tiles = RB_CEIL_DIV(min(ka, lo_al), BK);   // keys of [0, ka) below lo_al (the rest falls into window tiles)
@@ -152,17 +181,20 @@ __global__ void __launch_bounds__(kPfThreads) sink_window_prefill_kernel(Prefill
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       const int i = q0 + ty * 2 + r;
+      const int c_lo = p.chunk > 0 ? i / p.chunk * p.chunk : 0;
       float mx = -INFINITY;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const int j = k0 + tx + 8 * c;
-        const bool vis = j < kend && j <= i && i <= q_last && (p.window < 0 || i - j < p.window || j < p.keep);
-        s[r][c] = vis ? s[r][c] * qmul - slope * (float)(i - j) : -INFINITY;
+        const bool vis = j < kend && j <= i && i <= q_last && j >= c_lo && (p.window < 0 || i - j < p.window || j < p.keep);
+        float sc = s[r][c] * qmul;
+        if (p.softcap > 0.f) sc = p.softcap * tanhf(sc / p.softcap);
+        s[r][c] = vis ? sc - slope * (float)(i - j) : -INFINITY;
         mx = fmaxf(mx, s[r][c]);
       }
 #pragma unroll
       for (int off = 1; off < 8; off <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-      const float mn = fmaxf(m[r], mx);
+      const float mn = fmaxf(m[r], mx);                    // (-inf: no visible key so far, every weight below is 0)
       const float corr = (m[r] == -INFINITY) ? 0.f : expf(m[r] - mn);
       float ps = 0.f;
 #pragma unroll
@@ -194,20 +226,22 @@ __global__ void __launch_bounds__(kPfThreads) sink_window_prefill_kernel(Prefill
       }
     }
   }
-  const int og = p.H * d + p.G * d + p.G / p.vshare * dv;
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int i = q0 + ty * 2 + r;
     if (i > q_last) continue;
     const int64_t t = s0 + i;
     float f = l[r] > 0.f ? 1.f / l[r] : 0.f;
-    if (p.gate) f *= 1.f / (1.f + expf(-ld_any(p.qkvg, dt, t * p.ld + og + h)));
+    if (p.gmode == 1) f *= gate_factor(p.gate, dt, t * p.gld, 1, h, dv, 0);
 #pragma unroll
     for (int j = 0; j < NJ; ++j)
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const int col = j * 32 + tx * 4 + c;
-        if (col < dv) st_any(p.out, p.dto, t * (int64_t)(p.H * dv) + h * dv + col, o[r][j][c] * f);
+        if (col < dv) {
+          const float ge = p.gmode == 2 ? gate_factor(p.gate, dt, t * p.gld, 2, h, dv, col) : 1.f;
+          st_any(p.out, p.dto, t * (int64_t)(p.H * dv) + h * dv + col, o[r][j][c] * f * ge);
+        }
       }
   }
 }
@@ -283,9 +317,12 @@ struct DecodeParams {
   void* out; const void* temp; const void* sink;
   void* kc; void* vc;
   const int* lens; const int* slots;
-  int H, G, d, dv, rows, window, keep, gate, do_norm, dt;
+  int H, G, d, dv, rows, window, keep, do_norm, dt;
   float scale, slope_base, eps;
   int vshare, dto;
+  const void* gate; int64_t gld; int gmode;   // as in PrefillParams
+  int chunk; float softcap;
+  const float* turn_freq; int turn_dims, turn_inter;   // turn_dims > 0: the output is turned back by the position (frequencies [dims / 2])
 };
 
 __global__ void __launch_bounds__(kDecThreads) sink_window_decode_kernel(DecodeParams p) {
@@ -303,7 +340,7 @@ __global__ void __launch_bounds__(kDecThreads) sink_window_decode_kernel(DecodeP
   const int n = p.lens[slot];               // the new token's position
   const int64_t base = (int64_t)b * p.ld;
   const int gv = g / p.vshare, Gv = p.G / p.vshare;
-  const int ok = p.H * d, ov = ok + p.G * d, og = ov + Gv * dv;
+  const int ok = p.H * d, ov = ok + p.G * d;
   const int64_t cbase = ((int64_t)slot * p.G + g) * p.rows, vbase = ((int64_t)slot * Gv + gv) * p.rows;
 
   for (int idx = tid; idx < rep * d; idx += kDecThreads) {
@@ -323,7 +360,7 @@ __global__ void __launch_bounds__(kDecThreads) sink_window_decode_kernel(DecodeP
   }
   __syncthreads();   // the CTA's own global writes are visible to its threads from here on
 
-  const int lo = p.window < 0 ? 0 : max(0, n - p.window + 1);
+  const int lo = first_visible(n, p.window, p.chunk);
   const int ka = p.window < 0 ? 0 : min(p.keep, lo);
   const int nk = ka + (n - lo + 1);         // visible keys: positions [0, ka) and [lo, n]
   float m[kMaxRep], l[kMaxRep], acc[kMaxRep][kMaxColsPerThread];
@@ -369,6 +406,7 @@ __global__ void __launch_bounds__(kDecThreads) sink_window_decode_kernel(DecodeP
     for (int r = 0; r < kMaxRep; ++r)
       if (r < rep) {
         const float slope = p.slope_base >= 0.f ? exp2f(-p.slope_base * (float)(h0 + r + 1) / (float)p.H) : 0.f;
+        if (p.softcap > 0.f) s[r] = p.softcap * tanhf(s[r] / p.softcap);
         s[r] = have ? s[r] - slope * (float)(n - j) : -INFINITY;
         const float wm = rb::warp_max(s[r]);
         if (lane == 0) red[r * 4 + warp] = wm;
@@ -412,16 +450,29 @@ __global__ void __launch_bounds__(kDecThreads) sink_window_decode_kernel(DecodeP
     }
     __syncthreads();
   }
+  if (p.turn_dims > 0) {                    // neighbours' columns are needed: through shared memory (qs and ps are done with)
+#pragma unroll
+    for (int r = 0; r < kMaxRep; ++r)
+#pragma unroll
+      for (int c = 0; c < kMaxColsPerThread; ++c)
+        if (r < rep && tid + c * kDecThreads < dv) smem[r * dv + tid + c * kDecThreads] = acc[r][c];
+    __syncthreads();
+  }
 #pragma unroll
   for (int r = 0; r < kMaxRep; ++r)
     if (r < rep) {
       const int h = h0 + r;
       float f = l[r] > 0.f ? 1.f / l[r] : 0.f;
-      if (p.gate) f *= 1.f / (1.f + expf(-ld_any(p.qkvg, dt, base + og + h)));
+      if (p.gmode == 1) f *= gate_factor(p.gate, dt, (int64_t)b * p.gld, 1, h, dv, 0);
 #pragma unroll
       for (int c = 0; c < kMaxColsPerThread; ++c) {
         const int col = tid + c * kDecThreads;
-        if (col < dv) st_any(p.out, p.dto, (int64_t)b * (p.H * dv) + h * dv + col, acc[r][c] * f);
+        if (col >= dv) continue;
+        float o = acc[r][c];
+        if (col < p.turn_dims)
+          o = turn_back(o, smem[r * dv + turn_partner(col, p.turn_dims, p.turn_inter)], col, (float)n, p.turn_freq, p.turn_dims, p.turn_inter);
+        if (p.gmode == 2) o *= gate_factor(p.gate, dt, (int64_t)b * p.gld, 2, h, dv, col);
+        st_any(p.out, p.dto, (int64_t)b * (p.H * dv) + h * dv + col, o * f);
       }
     }
 }
@@ -467,7 +518,7 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
   const int n = p.lens[slot];
   const T* row_in = reinterpret_cast<const T*>(p.qkvg) + (int64_t)b * p.ld;
   const int Gv = p.G / p.vshare, gv = g / p.vshare;
-  const int ok = p.H * HD, ov = ok + p.G * HD, og = ov + Gv * HD;
+  const int ok = p.H * HD, ov = ok + p.G * HD;
   T* kc = reinterpret_cast<T*>(p.kc) + ((int64_t)slot * p.G + g) * p.rows * HD;
   T* vc = reinterpret_cast<T*>(p.vc) + ((int64_t)slot * Gv + gv) * p.rows * HD;   // (CTAs that share a value head append the same values)
 
@@ -494,7 +545,7 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
     for (int i = 0; i < 8; ++i) vn[i] = rb::to_f(rb::from_f<T>(vn[i] * rs));     // as later steps will read it from the cache
   }
   const int ring = max(p.rows - p.keep, 1);
-  const int lo = p.window < 0 ? 0 : max(0, n - p.window + 1);
+  const int lo = first_visible(n, p.window, p.chunk);
   const int ka = p.window < 0 ? 0 : min(p.keep, lo);
   const bool flat = lo < p.keep;                       // every visible position still lives in row = position
   const int r_lo = flat ? 0 : (lo - p.keep) % ring;
@@ -534,6 +585,7 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
       for (int i = 0; i < 8; ++i) s = fmaf(q[r][i], kf[i], s);
 #pragma unroll
       for (int o = LPR / 2; o > 0; o >>= 1) s += __shfl_xor_sync(gmask, s, o, LPR);
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
       s -= slope[r] * dist;
       const float mn = fmaxf(m[r], s);
       const float corr = (m[r] == -INFINITY) ? 0.f : __expf(m[r] - mn), pr = __expf(s - mn);
@@ -599,17 +651,20 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
     float mg = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kFastWarps; ++w) mg = fmaxf(mg, sm_m[w][r]);
-    float lg = 0.f, ag = 0.f;
+    const bool turn = fp.splits == 1 && c < p.turn_dims;
+    const int pc = turn ? turn_partner(c, p.turn_dims, p.turn_inter) : c;
+    float lg = 0.f, ag = 0.f, pg = 0.f;
 #pragma unroll
     for (int w = 0; w < kFastWarps; ++w) {
       const float cf = (sm_m[w][r] == -INFINITY) ? 0.f : __expf(sm_m[w][r] - mg);
       lg += sm_l[w][r] * cf;
       ag += sm_acc[w][r][c] * cf;
+      pg += sm_acc[w][r][pc] * cf;
     }
     const int h = g * REP + r;
     if (fp.splits == 1) {
-      float f = lg > 0.f ? 1.f / lg : 0.f;
-      if (p.gate) f *= 1.f / (1.f + expf(-rb::to_f(row_in[og + h])));
+      if (turn) ag = turn_back(ag, pg, c, (float)n, p.turn_freq, p.turn_dims, p.turn_inter);
+      const float f = (lg > 0.f ? 1.f / lg : 0.f) * gate_factor(p.gate, p.dt, (int64_t)b * p.gld, p.gmode, h, HD, c);
       reinterpret_cast<T*>(p.out)[(int64_t)b * p.H * HD + (int64_t)h * HD + c] = rb::from_f<T>(ag * f);
     } else {
       const int64_t o = ((int64_t)b * p.H + h) * fp.splits + split;
@@ -620,24 +675,30 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
 }
 
 template <typename T, int HD>
-__global__ void sink_window_decode_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, const T* __restrict__ qkvg,
-                                                int64_t ld, int og, int H, int gate, T* __restrict__ out, int splits) {
+__global__ void sink_window_decode_merge_kernel(FastParams fp) {
+  const DecodeParams& p = fp.d;
+  __shared__ float so[HD];
   const int64_t bh = blockIdx.x;
-  const int c = threadIdx.x;
+  const int c = threadIdx.x, splits = fp.splits, b = (int)(bh / p.H), h = (int)(bh % p.H);
   rb::pdl_trigger();
   rb::pdl_wait();
   float mg = -INFINITY;
-  for (int s = 0; s < splits; ++s) mg = fmaxf(mg, part_ml[(bh * splits + s) * 2]);
+  for (int s = 0; s < splits; ++s) mg = fmaxf(mg, fp.part_ml[(bh * splits + s) * 2]);
   float lg = 0.f, ag = 0.f;
   for (int s = 0; s < splits; ++s) {
-    const float ms = part_ml[(bh * splits + s) * 2];
+    const float ms = fp.part_ml[(bh * splits + s) * 2];
     const float cf = (ms == -INFINITY) ? 0.f : expf(ms - mg);
-    lg += part_ml[(bh * splits + s) * 2 + 1] * cf;
-    ag += part_acc[(bh * splits + s) * HD + c] * cf;
+    lg += fp.part_ml[(bh * splits + s) * 2 + 1] * cf;
+    ag += fp.part_acc[(bh * splits + s) * HD + c] * cf;
   }
-  float f = lg > 0.f ? 1.f / lg : 0.f;
-  if (gate) f *= 1.f / (1.f + expf(-rb::to_f(qkvg[(bh / H) * ld + og + (bh % H)])));
-  out[bh * HD + c] = rb::from_f<T>(ag * f);
+  if (p.turn_dims > 0) {
+    so[c] = ag;
+    __syncthreads();
+    if (c < p.turn_dims)
+      ag = turn_back(ag, so[turn_partner(c, p.turn_dims, p.turn_inter)], c, (float)p.lens[p.slots ? p.slots[b] : b], p.turn_freq, p.turn_dims, p.turn_inter);
+  }
+  const float f = (lg > 0.f ? 1.f / lg : 0.f) * gate_factor(p.gate, p.dt, (int64_t)b * p.gld, p.gmode, h, HD, c);
+  reinterpret_cast<T*>(p.out)[bh * HD + c] = rb::from_f<T>(ag * f);
 }
 
 template <typename T, int HD>
@@ -648,14 +709,14 @@ int launch_fast(const FastParams& fp, int B, cudaStream_t s) {
   switch (p.H / p.G) {
     case 1: RB_L(1); break;
     case 2: RB_L(2); break;
+    case 3: RB_L(3); break;
     case 4: RB_L(4); break;
+    case 6: RB_L(6); break;
     case 8: RB_L(8); break;
     default: return -1;
   }
 #undef RB_L
-  if (fp.splits > 1)
-    rb::launch_pdl(sink_window_decode_merge_kernel<T, HD>, dim3(B * p.H), dim3(HD), 0, s, (const float*)fp.part_acc, (const float*)fp.part_ml,
-                   reinterpret_cast<const T*>(p.qkvg), p.ld, p.H * HD + p.G * HD + p.G / p.vshare * HD, p.H, p.gate, reinterpret_cast<T*>(p.out), fp.splits);
+  if (fp.splits > 1) rb::launch_pdl(sink_window_decode_merge_kernel<T, HD>, dim3(B * p.H), dim3(HD), 0, s, fp);
   return 0;
 }
 
@@ -672,10 +733,11 @@ extern "C" int rb_value_norm_store(const void* qkvg, int64_t ld, int dt, void* v
 
 extern "C" int rb_sink_window_prefill(const void* qkvg, int64_t ld, const void* vn, void* out, const void* temp, const void* sink, const int* cu,
                                       int n_seqs, int max_seqlen, int H, int G, int d, int dv, float scale, int window, int keep, float slope_base,
-                                      int gate, int dt, int vshare, int64_t vld, int dto, cudaStream_t s) {
+                                      const void* gate, int64_t gld, int gmode, int chunk, float softcap, int dt, int vshare, int64_t vld, int dto,
+                                      cudaStream_t s) {
   if (n_seqs == 0 || max_seqlen == 0) return 0;
-  if (dv > 256 || d > 512 || H % G || vshare < 1 || G % vshare) return -1;
-  PrefillParams p{qkvg, ld, vn, out, temp, sink, cu, H, G, d, dv, window, keep, gate, dt, scale, slope_base, vshare, dto, vld};
+  if (dv > 256 || d > 512 || H % G || vshare < 1 || G % vshare || (gmode != 0 && gate == nullptr)) return -1;
+  PrefillParams p{qkvg, ld, vn, out, temp, sink, cu, H, G, d, dv, window, keep, dt, scale, slope_base, vshare, dto, vld, gate, gld, gmode, chunk, softcap};
   const int nj = dv <= 32 ? 1 : dv <= 64 ? 2 : dv <= 128 ? 4 : 8;
   const int dp = (d + 3) & ~3;
   const size_t smem = sizeof(float) * ((size_t)(BQ + BK) * (dp + 4) + (size_t)BK * (nj * 32 + 4) + (size_t)BQ * (BK + 1));
@@ -697,27 +759,35 @@ extern "C" int rb_sink_window_prefill(const void* qkvg, int64_t ld, const void* 
 
 extern "C" int rb_sink_window_decode(const void* qkvg, int64_t ld, void* out, const void* temp, const void* sink, void* kc, void* vc,
                                      const int* lens, const int* slots, int B, int H, int G, int d, int dv, int rows, float scale, int window,
-                                     int keep, float slope_base, int gate, int do_norm, float eps, int dt, int vshare, int dto, cudaStream_t s) {
+                                     int keep, float slope_base, const void* gate, int64_t gld, int gmode, int chunk, float softcap,
+                                     const float* turn_freq, int turn_dims, int turn_inter, int do_norm, float eps, int dt, int vshare, int dto,
+                                     cudaStream_t s) {
   if (B == 0) return 0;
   const int rep = min(H / G, kMaxRep);
-  if (H % G || dv > kDecThreads * kMaxColsPerThread || vshare < 1 || G % vshare) return -1;
-  DecodeParams p{qkvg, ld, out, temp, sink, kc, vc, lens, slots, H, G, d, dv, rows, window, keep, gate, do_norm, dt, scale, slope_base, eps, vshare, dto};
-  const size_t smem = sizeof(float) * ((size_t)rep * d + (size_t)rep * kDecThreads + rep * 5 + 32 + dv + kDecThreads);
+  if (H % G || dv > kDecThreads * kMaxColsPerThread || vshare < 1 || G % vshare || (gmode != 0 && gate == nullptr)) return -1;
+  if (turn_dims % 2 || turn_dims > dv || (turn_dims > 0 && turn_freq == nullptr)) return -1;
+  DecodeParams p{qkvg, ld, out, temp, sink, kc, vc, lens, slots, H, G, d, dv, rows, window, keep, do_norm, dt, scale, slope_base, eps, vshare, dto,
+                 gate, gld, gmode, chunk, softcap, turn_freq, turn_dims, turn_inter};
+  size_t smem = sizeof(float) * ((size_t)rep * d + (size_t)rep * kDecThreads + rep * 5 + 32 + dv + kDecThreads);
+  if (turn_dims > 0 && smem < sizeof(float) * (size_t)rep * dv) smem = sizeof(float) * (size_t)rep * dv;
   if (smem > 48 * 1024) cudaFuncSetAttribute(sink_window_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   sink_window_decode_kernel<<<dim3(B, G, RB_CEIL_DIV(H / G, kMaxRep)), kDecThreads, smem, s>>>(p);
   return 0;
 }
 
-// 16-bit fast path of the decode form (dt 1 / 2, d == dv in {64, 128}, H / G in {1, 2, 4, 8}, 16-byte aligned rows); part_acc
+// 16-bit fast path of the decode form (dt 1 / 2, d == dv in {64, 128}, H / G in {1, 2, 3, 4, 6, 8}, 16-byte aligned rows); part_acc
 // [B, H, splits, d] and part_ml [B, H, splits, 2] fp32 are scratch for splits > 1.  Returns -1 for shapes it does not take.
 extern "C" int rb_sink_window_decode_fast(const void* qkvg, int64_t ld, void* out, const void* temp, const void* sink, void* kc, void* vc,
                                           const int* lens, const int* slots, float* part_acc, float* part_ml, int splits, int B, int H, int G, int d,
-                                          int rows, float scale, int window, int keep, float slope_base, int gate, int do_norm, float eps, int dt,
-                                          int vshare, cudaStream_t s) {
+                                          int rows, float scale, int window, int keep, float slope_base, const void* gate, int64_t gld, int gmode,
+                                          int chunk, float softcap, const float* turn_freq, int turn_dims, int turn_inter, int do_norm, float eps,
+                                          int dt, int vshare, cudaStream_t s) {
   if (B == 0) return 0;
   if ((dt != 1 && dt != 2) || (d != 64 && d != 128) || H % G || vshare < 1 || G % vshare || ld % 8 || ((uintptr_t)qkvg & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15))
     return -1;
-  FastParams fp{DecodeParams{qkvg, ld, out, temp, sink, kc, vc, lens, slots, H, G, d, d, rows, window, keep, gate, do_norm, dt, scale, slope_base, eps, vshare, dt},
+  if ((gmode != 0 && gate == nullptr) || turn_dims % 2 || turn_dims > d || (turn_dims > 0 && turn_freq == nullptr)) return -1;
+  FastParams fp{DecodeParams{qkvg, ld, out, temp, sink, kc, vc, lens, slots, H, G, d, d, rows, window, keep, do_norm, dt, scale, slope_base, eps, vshare, dt,
+                             gate, gld, gmode, chunk, softcap, turn_freq, turn_dims, turn_inter},
                 part_acc, part_ml, splits};
   if (dt == 1) return d == 128 ? launch_fast<__nv_bfloat16, 128>(fp, B, s) : launch_fast<__nv_bfloat16, 64>(fp, B, s);
   return d == 128 ? launch_fast<__half, 128>(fp, B, s) : launch_fast<__half, 64>(fp, B, s);

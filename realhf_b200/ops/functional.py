@@ -706,31 +706,35 @@ def centred_norm_ref(x, w, eps: float):
     return dx * torch.rsqrt(dx.pow(2).mean(-1, keepdim=True) + eps) * w.float()
 
 
-def centred_norm(x, w, eps: float, out_dtype):
-    """Bias-free LayerNorm of every row of x [T, W] (fp32 statistics, the variance as the mean of the squared deviations), times w,
-    in out_dtype."""
+def centred_norm(x, w, eps: float, out_dtype, rms: bool = False):
+    """Bias-free LayerNorm of every row of x [T, W] (fp32 statistics, the variance as the mean of the squared deviations), or with
+    `rms` RMSNorm, times w (a vector, or one number for all columns), in out_dtype."""
     if use_native(x):
         out = torch.empty(x.shape, dtype=out_dtype, device=x.device)
-        lib().centred_norm(None, x.contiguous(), None, 1.0, 1.0, None, None, 1.0, w, out, eps)
+        lib().centred_norm(None, x.contiguous(), None, 1.0, 1.0, None, None, 1.0, w, out, eps, rms)
         return out
-    return centred_norm_ref(x, w, eps).to(out_dtype)
+    return (group_rmsnorm_ref(x, w, 1, eps) if rms else centred_norm_ref(x, w, eps)).to(out_dtype)
 
 
 def residual_add_centred_norm_(x, y, w, eps: float, scale=None, mult: float = 1.0, y2=None, a: float = 1.0, b: float = 1.0, next_w=None,
-                               out_dtype=None):
-    """x += mult * scale * LayerNorm(a y + b y2) * w in place (bias-free LayerNorm; `scale` a vector or None; y2 None: the branch
-    output is a y), the sum formed in fp32 and stored in x's dtype.  With `next_w`, also returns LayerNorm(x) * next_w of the
-    updated row in out_dtype (the next sublayer's input), from the same kernel."""
+                               out_dtype=None, rms: bool = False, gate=None):
+    """x += mult * scale * N((a y + b y2) * sigmoid(gate)) * w in place (N: bias-free LayerNorm, or RMSNorm with `rms`; w a vector or
+    one number; `scale` a vector or None; y2 None: the branch output is a y; `gate` logits, possibly a column slice, or None), the
+    sum formed in fp32 and stored in x's dtype.  With `next_w`, also returns N(x) * next_w of the updated row in out_dtype (the
+    next sublayer's input), from the same kernel."""
     if use_native(x) and x.is_contiguous():
         out = torch.empty(x.shape, dtype=out_dtype, device=x.device) if next_w is not None else None
-        lib().centred_norm(x, y.contiguous(), y2.contiguous() if y2 is not None else None, a, b, w, scale, mult, next_w, out, eps)
+        lib().centred_norm(x, y.contiguous(), y2.contiguous() if y2 is not None else None, a, b, w, scale, mult, next_w, out, eps, rms, gate)
         return out
+    norm = (lambda v, w_: group_rmsnorm_ref(v, w_, 1, eps)) if rms else (lambda v, w_: centred_norm_ref(v, w_, eps))
     br = a * y.float() + (b * y2.float() if y2 is not None else 0.0)
-    n = centred_norm_ref(br, w, eps)
+    if gate is not None:
+        br = br * torch.sigmoid(gate.float())
+    n = norm(br, w)
     if scale is not None:
         n = n * scale.float()
     x.copy_((x.float() + mult * n).to(x.dtype))
-    return centred_norm_ref(x, next_w, eps).to(out_dtype) if next_w is not None else None
+    return norm(x, next_w).to(out_dtype) if next_w is not None else None
 
 
 def clamped_glu_ref(gu, limit: float, alpha: float):
@@ -820,9 +824,10 @@ def relu2(x):
     return (r * r).to(x.dtype)
 
 
-def relu2_linear(x, w_up):
-    """relu(x @ w_up^T)^2.  16-bit CUDA operands of more than 128 rows run projection and activation as ONE kernel (the activation
-    in the epilogue of the CTA-pair tcgen05 GEMM, like `gated_linear`); everything else composes the two ops."""
+def relu2_linear(x, w_up, bias=None, act_cols: Optional[int] = None):
+    """relu(x @ w_up^T (+ bias))^2, on the first `act_cols` outputs only when given (the others keep the plain projection).  16-bit CUDA
+    operands of more than 128 rows run projection and activation as ONE kernel (the activation in the epilogue of the CTA-pair
+    tcgen05 GEMM, like `gated_linear`); everything else composes the two ops."""
     if use_native(x) and x.dtype in (torch.bfloat16, torch.float16) and gemm_impl() is not None:
         from realhf_b200.ops import gemm as G
         x2 = x.reshape(-1, x.shape[-1])
@@ -830,9 +835,17 @@ def relu2_linear(x, w_up):
                 and os.environ.get("REAL_GEMM_GLU", "1") == "1"):
             if x2.stride(-1) != 1 or x2.stride(0) % 8 != 0 or x2.data_ptr() % 16 != 0:
                 x2 = x2.contiguous()
-            out = lib().gemm_relu2(x2, w_up, G._sms(x.device))
+            out = lib().gemm_relu2(x2, w_up, G._sms(x.device), bias, act_cols or 0)
             return out.view(*x.shape[:-1], w_up.shape[0])
-    return relu2(linear(x, w_up))
+    y = linear(x, w_up, bias)
+    if act_cols is None:
+        return relu2(y)
+    if use_native(y):
+        lib().relu2_cols_(y, act_cols)
+        return y
+    r = torch.relu(y[..., :act_cols].float())
+    y[..., :act_cols] = (r * r).to(y.dtype)
+    return y
 
 
 def concat_cast(a, b, out_dtype):
