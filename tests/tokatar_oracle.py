@@ -52,19 +52,19 @@ def attend(q, k, v, first_pos: int, scale: float, chunk: Optional[int] = None, s
     T, H, _ = q.shape
     G = k.shape[1]
     out = torch.zeros(T, H, v.shape[-1], dtype=q.dtype)
+    group = torch.arange(H) // (H // G)
     for t in range(T):
         i = first_pos + t
         lo = 0 if chunk is None else (i // chunk) * chunk
-        for h in range(H):
-            g = h // (H // G)
-            s = (k[lo:i + 1, g] @ q[t, h]) * scale
-            if softcap is not None:
-                s = softcap * torch.tanh(s / softcap)
-            mx = s.max()
-            if plus_one:
-                mx = torch.clamp(mx, min=0.0)
-            e = torch.exp(s - mx)
-            out[t, h] = (e / (e.sum() + (torch.exp(-mx) if plus_one else 0.0))) @ v[lo:i + 1, g]
+        s = torch.einsum("nhd,hd->hn", k[lo:i + 1][:, group], q[t]) * scale
+        if softcap is not None:
+            s = softcap * torch.tanh(s / softcap)
+        mx = s.max(1, keepdim=True).values
+        if plus_one:
+            mx = mx.clamp(min=0.0)
+        e = torch.exp(s - mx)
+        den = e.sum(1, keepdim=True) + (torch.exp(-mx) if plus_one else 0.0)
+        out[t] = torch.einsum("hn,nhd->hd", e / den, v[lo:i + 1][:, group])
     return out
 
 
@@ -81,7 +81,7 @@ def attention(h, w, m: dict, pos, st: dict):
     q = rotate((h @ w["q"].T).view(T, H, d), pos, f, False)
     k = append(st, "k", rotate((h @ w["k"].T).view(T, G, d), pos, f, False))
     v = append(st, "v", (h @ w["v"].T).view(T, G, dv))
-    o = attend(q, k, v, k.shape[0] - T, m["scale"], m["mask"]["size"], softcap=m["softcap"])
+    o = attend(q, k, v, k.shape[0] - T, m["scale"], (m.get("mask") or {}).get("size"), softcap=m["softcap"])
     return (o.reshape(T, H * dv) * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
 
 
@@ -97,7 +97,7 @@ def attention_2(h, w, m: dict, pos, st: dict, eps: float):
     q = rotate(q.view(T, H, d), pos, f, True)
     k = append(st, "k", rotate(k.view(T, G, d), pos, f, True))
     v = append(st, "v", rotate(v.view(T, G, dv), pos, fv, True))
-    o = attend(q, k, v, k.shape[0] - T, m["scale"], m["mask"]["size"], plus_one=True)
+    o = attend(q, k, v, k.shape[0] - T, m["scale"], (m.get("mask") or {}).get("size"), plus_one=True)
     o = rotate(o, -pos, fv, True)
     return (o.reshape(T, H * dv) * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
 
