@@ -1,8 +1,8 @@
 """Prefill / decode throughput of a heterogeneous-stack design next to the closest homogeneous model of equal size, and the
 roofline position of its kernels next to the like kernels of that model.  Reached through `bench.py --serve-bench rapodra`,
-`--serve-bench tizodra`, `--serve-bench defilorn` or `--serve-bench buvesun` (the default workload of bench.py is unaffected).
-Buvesun is also timed beside a Defilorn of equal size, the closest heterogeneous stack (window attention, a matrix-state mixer, routed
-feed-forwards with a shared expert).
+`--serve-bench tizodra`, `--serve-bench defilorn`, `--serve-bench buvesun` or `--serve-bench tokatar` (the default workload of bench.py
+is unaffected).  Buvesun and Tokatar are also timed beside a Defilorn of equal size, the closest heterogeneous stack (window attention,
+rotated latent attention, a matrix-state mixer, dense and routed feed-forwards).
 
 Both models run through `models.generation`: prefill = `prefill_into_state` (the packed prefill `generate` performs) into a
 standing decode state, decode = the CUDA-graph loop of `generate` with the sampler in the graph; random weights, bf16.  Timing: CUDA events, >= 3 warm-up calls, weights + state far larger than L2 per call for
@@ -106,10 +106,33 @@ def buvesun_config(s: dict, n_layers: int = 4) -> dict:
                 norm=dict(eps=1e-5), residual_mult=0.7, vocab=s["vocab"], width=s["width"])
 
 
+TOKATAR_SIZES = {
+    # the Defilorn sizes plus: chunk (a window of the same length there), rotated dimensions, soft cap
+    "1b-like": dict(DEFILORN_SIZES["1b-like"], chunk=512, rot_dims=128, softcap=30.0),
+    "7b-like": dict(DEFILORN_SIZES["7b-like"], chunk=1024, rot_dims=128, softcap=30.0),
+}
+
+
+def tokatar_config(s: dict, n_layers: int = 4) -> dict:
+    """Soft-capped chunked attention, chunked attention with turned values, latent attention in turn; dense feed-forwards."""
+    rot = dict(base=5e5, dims=s["rot_dims"])
+    dense = dict(kind="dense", ff=s["ff"])
+    base = dict(dim=s["dim"], heads=s["heads"], kv_heads=s["kv_heads"], vdim=s["vdim"], scale=s["dim"] ** -0.5, mask=dict(size=s["chunk"]))
+    att = dict(type="attention", mlp=dense, mixer=dict(base, softcap=s["softcap"], rot=dict(rot, scaling=dict(factor=8.0, high=4.0, low=1.0, original=4096))))
+    att2 = dict(type="attention_2", mlp=dense, mixer=dict(base, rot=rot))
+    lat = dict(type="latent_attention", mlp=dense,
+               mixer=dict(dim=s["nope"], heads=s["heads"], kv_rank=s["kv_rank"], rot_dim=s["rot"], vdim=s["vdim"], scale=(s["nope"] + s["rot"]) ** -0.5,
+                          rot=dict(base=1e6, dims=s["rot"])))
+    kinds = [att, att2, lat]
+    return dict(architecture="Tokatar", embedding=dict(scale=8.0), layers=[kinds[i % 3] for i in range(n_layers)], norm=dict(eps=1e-5),
+                vocab=s["vocab"], width=s["width"])
+
+
 def _hetero_model(design: str, s: dict, n_layers: int, dev):
     from realhf_b200.models import hf_io
     from realhf_b200.models.real_model import ReaLModel
-    cfg = {"rapodra": rapodra_config, "tizodra": tizodra_config, "defilorn": defilorn_config, "buvesun": buvesun_config}[design](s, n_layers)
+    cfg = {"rapodra": rapodra_config, "tizodra": tizodra_config, "defilorn": defilorn_config, "buvesun": buvesun_config,
+           "tokatar": tokatar_config}[design](s, n_layers)
     m = ReaLModel(hf_io.family(design).config_from_dict(cfg, False), dtype=torch.bfloat16, device=dev).init_random_fast()
     for p in m.parameters():
         p.requires_grad_(False)
@@ -160,7 +183,7 @@ def model_numbers(name: str, s: dict, n_layers: int, batch: int, prompt_len: int
     ids = torch.randint(3, s["vocab"], (batch * prompt_len,), device=dev)
     cu = torch.arange(0, batch + 1, device=dev, dtype=torch.int32) * prompt_len
     arms = [(design, new), ("llama-equal-size", old)]
-    if design == "buvesun":
+    if design in ("buvesun", "tokatar"):
         arms.insert(1, ("defilorn-equal-size", _hetero_model("defilorn", s, n_layers, dev)))
     for label, m in arms:
         # prefill: the packed prefill into a standing decode state (`prefill_into_state`, what `generate` calls), so that the
@@ -632,8 +655,145 @@ def buvesun_kernel_numbers(name: str, s: dict, batch: int, prompt_len: int, ctx:
     return rows
 
 
+def tokatar_kernel_numbers(name: str, s: dict, batch: int, prompt_len: int, ctx: int, dev, peaks: Dict[str, float]) -> List[dict]:
+    """The Tokatar kernels next to the like kernels of the closest models at the same token count and head sizes: Defilorn's norms,
+    gate and latent attention, Buvesun's wrapped norm, rotation and window attention, LLaMA's norm, rotation and attention.
+    Attention FLOPs count the visible (query, key) pairs."""
+    from realhf_b200.models import hf_io
+    from realhf_b200.models.hetero_block import packed_meta
+    from realhf_b200.models.sharding import latent_rope_sections
+    from realhf_b200.ops import attention as A
+    from realhf_b200.ops import functional as OF
+    bf = torch.bfloat16
+    rc = hf_io.family("tokatar").config_from_dict(tokatar_config(s, 3), False)
+    a1, a2, la = rc.blocks[0].wattn, rc.blocks[1].wattn, rc.blocks[2].attn
+    bw = hf_io.family("buvesun").config_from_dict(buvesun_config(BUVESUN_SIZES[name], 2), False).blocks[0].wattn
+    dl = hf_io.family("defilorn").config_from_dict(defilorn_config(s, 3), False).blocks[2].attn
+    W, H, G, d, dv, C, F = s["width"], s["heads"], s["kv_heads"], s["dim"], s["vdim"], s["chunk"], s["ff"]
+    T = batch * prompt_len
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    rows = []
+
+    def add(kernel, like, ms, nbytes, flops):
+        floor_ms = max(nbytes / (peaks["hbm_gbs"] * 1e9), flops / (peaks["bf16_tflops"] * 1e12)) * 1e3
+        rows.append(dict(bench="kernel", size=name, kernel=kernel, like=like, ms=round(ms, 4), gbytes=round(nbytes / 1e9, 4),
+                         gflop=round(flops / 1e9, 2), roofline_ms=round(floor_ms, 4), frac_of_measured_roofline=round(floor_ms / ms, 4)))
+
+    def t(fn, iters=10):
+        return _time(fn, iters, flush=flush)
+    cu = torch.arange(0, batch + 1, device=dev, dtype=torch.int32) * prompt_len
+    meta = packed_meta(cu, T, torch.arange(batch, dtype=torch.int32, device=dev), None, prompt_len)
+    # ---- row-wise
+    x32 = torch.randn(T, W, device=dev)
+    xb = x32.to(bf)
+    w, one = torch.ones(W, device=dev, dtype=bf), torch.ones(1, device=dev, dtype=bf)
+    gl = torch.randn(T, F + W, device=dev).to(bf)[:, F:]
+    add("residual_add_centred_norm_ (rms: residual gate, output norm, layer scale, add, next norm; prefill)", False,
+        t(lambda: OF.residual_add_centred_norm_(x32, xb, one, 1e-5, w, next_w=one, out_dtype=bf, rms=True, gate=gl)), T * W * 14, 0)
+    add("residual_add_centred_norm_ (buvesun: two branches, output norm, layer scale, add, next norm; prefill)", True,
+        t(lambda: OF.residual_add_centred_norm_(x32, xb, w, 1e-5, w, 0.7, xb, 0.6, 1.1, w, bf)), T * W * 14, 0)
+    add("add_rms_norm_ (defilorn: fp32 stream += branch, next norm; prefill)", True, t(lambda: OF.add_rms_norm_(x32, xb, w, 1e-5, bf, 1.0)), T * W * 12, 0)
+    # ---- feed-forward
+    up, upb = (torch.randn(F + W, W, device=dev) * W ** -0.5).to(bf), torch.zeros(F + W, device=dev, dtype=bf)
+    add("relu2_linear (up | residual gate, bias, activation on the up columns in the epilogue; prefill)", False,
+        t(lambda: OF.relu2_linear(xb, up, upb, act_cols=F), 5), (T * W + T * (F + W) + (F + W) * W) * 2, 2.0 * T * W * (F + W))
+    add("relu2_linear (tizodra: no gate rows, no bias; prefill)", True, t(lambda: OF.relu2_linear(xb, up[:F]), 5),
+        (T * W + T * F + F * W) * 2, 2.0 * T * W * F)
+    xd = xb[:batch].contiguous()
+    add("relu2_linear (up | residual gate; decode)", False, t(lambda: OF.relu2_linear(xd, up, upb, act_cols=F)), (F + W) * W * 2, 2.0 * batch * W * (F + W))
+    add("linear (same matrix, no activation; decode)", True, t(lambda: OF.linear(xd, up)), (F + W) * W * 2, 2.0 * batch * W * (F + W))
+    # ---- chunked attention
+    ld = H * d + G * (d + dv) + H * dv
+    wide = torch.randn(T, ld + W, device=dev).to(bf)
+    wq, wk = torch.ones(H * d, device=dev, dtype=bf), torch.ones(G * d, device=dev, dtype=bf)
+    rows_c = a1.cache_rows(prompt_len + 64)
+    kc, vc = (torch.zeros(batch, G, rows_c, n, device=dev, dtype=bf) for n in (d, dv))
+    kw = dict(pos=meta.pos, k_cache=kc, v_cache=vc, tok_slot=meta.tok_slot, remain=meta.remain)
+    kept = batch * min(prompt_len, rows_c) * G * (d + dv) * 2
+    add("window_prepare_ (attention: rotate q and k, cache fill; prefill)", False, t(lambda: A.window_prepare_(wide, a1, None, None, 1e-5, **kw)),
+        T * (H + G) * d * 4 + T * G * dv * 2 + kept, 0)
+    add("window_prepare_ (attention_2: norms over all heads, rotate q, k and v, cache fill; prefill)", False,
+        t(lambda: A.window_prepare_(wide, a2, wq, wk, 1e-5, **kw)), T * ((H + G) * d + G * dv) * 4 + kept, 0)
+
+    def buvesun_prepare():
+        A.rotate_qk_(wide, bw, pos=meta.pos)
+        A.value_norm_store(wide, bw, 1e-5, kc, vc, meta.tok_slot, meta.pos, meta.remain)
+    add("rotate_heads_ + value_norm_store (buvesun: half of every head, cache fill; prefill)", True, t(buvesun_prepare),
+        T * (H + G) * bw.rotary.dims * 4 + T * G * dv * 4 + kept, 0)
+    qkv_l = torch.randn(T, (H + 2 * G) * d, device=dev).to(bf)
+    cos, sin = OF.rope_tables(prompt_len + 64, d, 10000.0, dev)
+    add("apply_rope (llama, prefill: q and k, table look-up)", True, t(lambda: OF.apply_rope(qkv_l[:, :(H + G) * d], cos, sin, meta.pos, H + G, d)),
+        T * (H + G) * d * 4, 0)
+    pairs = batch * sum(p % C + 1 for p in range(prompt_len))
+    att_bytes = T * ((H + G) * (d + dv) + H * dv) * 2
+    add("sink_window_attention (attention: chunked, soft cap, element gate; prefill, tcgen05)", False,
+        t(lambda: A.sink_window_attention(wide, A.window_values(wide, a1), a1, None, None, meta.pos, cu, prompt_len), 5), att_bytes,
+        2.0 * pairs * H * (d + dv))
+    add("sink_window_attention (attention_2: chunked, unit sink, then turn back + element gate; prefill, tcgen05)", False,
+        t(lambda: A.sink_window_attention(wide, A.window_values(wide, a2), a2, None, None, meta.pos, cu, prompt_len), 5), att_bytes,
+        2.0 * pairs * H * (d + dv))
+    o = torch.randn(T, H * dv, device=dev).to(bf)
+    add("turn_gate_ (turn back + element gate alone; prefill)", False, t(lambda: A.turn_gate_(o, a2, A.window_gate(wide, a2), pos=meta.pos)), T * H * dv * 6, 0)
+    add("sigmoid_gate_ (defilorn; prefill)", True, t(lambda: A.sigmoid_gate_(o, A.window_gate(wide, a2))), T * H * dv * 6, 0)
+    win_pairs = batch * sum(min(p + 1, bw.window) for p in range(prompt_len))
+    add("sink_window_attention (buvesun: window of the chunk's length; prefill, tcgen05)", True,
+        t(lambda: A.sink_window_attention(wide, A.window_values(wide, a2), bw, None, None, meta.pos, cu, prompt_len), 5),
+        T * (H + G) * (d + dv) * 2, 2.0 * win_pairs * H * (d + dv))
+    full_pairs = batch * prompt_len * (prompt_len + 1) // 2
+    add("varlen attention tcgen05 (llama, prefill, full causal)", True, t(lambda: A.varlen_attention_qkv(qkv_l, cu, prompt_len, H, G, d, None, True), 5),
+        T * (2 * H + 2 * G) * d * 2, 4.0 * full_pairs * H * d)
+    at = ctx // C * C + C // 2 + C // 4                       # a position three quarters into its chunk
+    keys = at % C + 1
+    lens = torch.full((batch,), at, dtype=torch.int32, device=dev)
+    rows_d = a1.cache_rows(ctx + C)
+    kc, vc = (torch.randn(batch, G, rows_d, n, device=dev).to(bf) for n in (d, dv))
+    q1 = torch.randn(batch, ld + W, device=dev).to(bf)
+    dec_bytes = batch * (keys * G * (d + dv) + 3 * H * dv) * 2
+    add(f"window_prepare_ (attention_2; decode, {batch} rows)", False, t(lambda: A.window_prepare_(q1, a2, wq, wk, 1e-5, cache_lens=lens)),
+        batch * ((H + G) * d + G * dv) * 4, 0)
+    add(f"rotate_heads_ (buvesun; decode, {batch} rows)", True, t(lambda: A.rotate_qk_(q1, bw, cache_lens=lens)), batch * (H + G) * bw.rotary.dims * 4, 0)
+    for label, a in (("attention: soft cap, element gate", a1), ("attention_2: unit sink, turn back, element gate", a2)):
+        add(f"sink_window_decode_attention ({label}; {keys} keys)", False,
+            t(lambda: A.sink_window_decode_attention(q1, a, None, None, kc, vc, lens, None, 1e-5)), dec_bytes, 2.0 * batch * H * keys * (d + dv))
+    wkeys = min(at + 1, bw.window)
+    add(f"sink_window_decode_attention (buvesun; {wkeys} keys)", True, t(lambda: A.sink_window_decode_attention(q1, bw, None, None, kc, vc, lens, None, 1e-5)),
+        batch * wkeys * G * (d + dv) * 2, 2.0 * batch * H * wkeys * (d + dv))
+    lens_l = torch.full((batch,), ctx, dtype=torch.int32, device=dev)
+    kl, vl = (torch.zeros(batch, G, ctx + 64, d, device=dev, dtype=bf).permute(0, 2, 1, 3) for _ in range(2))
+    qkv1 = torch.randn(batch, (H + 2 * G) * d, device=dev).to(bf)
+    cos2, sin2 = OF.rope_tables(ctx + 64, d, 10000.0, dev)
+    add(f"decode_attention (llama, ctx {ctx}, all {ctx + 1} keys)", True, t(lambda: A.decode_attention(qkv1, kl, vl, lens_l, H, G, d, None, cos2, sin2)),
+        batch * (ctx + 1) * G * d * 4, 4.0 * batch * H * (ctx + 1) * d)
+    # ---- latent attention: half layout + head gate beside interleaved + sink + element gate
+    r, n, rot = la.kv_rank, la.qk_dim, la.rot_dim
+    wc = torch.ones(r, device=dev, dtype=bf)
+    wu = (torch.randn(H * (n + dv), r, device=dev) * r ** -0.5).to(bf)
+    sink = torch.zeros(H, device=dev, dtype=bf)
+    for like, a in ((False, la), (True, dl)):
+        fam = "defilorn: interleaved, sink, element gate apart" if like else "half layout, head gate"
+        pl = torch.randn(T, sum(latent_rope_sections(a)), device=dev).to(bf)
+        pd = pl[:batch].contiguous()
+        wql = torch.ones(a.q_rank, device=dev, dtype=bf) if a.q_rank else None
+        cache = torch.randn(batch, prompt_len + 64, r + rot, device=dev).to(bf)
+        add(f"latent_rope_prepare ({fam}; prefill)", like,
+            t(lambda: A.latent_rope_prepare(pl, a, wql, wc, 1e-5, meta.pos, cache, meta.tok_slot, meta.remain)), T * ((r + rot) * 6 + 4 * (a.q_rank or 0)), 0)
+        _, lt = A.latent_rope_prepare(pl, a, wql, wc, 1e-5, meta.pos, None)
+        kv = OF.linear(lt[:, :r], wu)
+        q = torch.randn(T, H * (n + rot), device=dev).to(bf)
+        gate = torch.randn(T, (H + 7) // 8 * 8, device=dev).to(bf)[:, :H] if not like else None
+        sk = sink if like else None
+        add(f"latent_rope_attention ({fam}; prefill)", like, t(lambda: A.latent_rope_attention(q, kv, lt, a, sk, meta.pos, cu, prompt_len, gate=gate), 5),
+            T * (H * (n + rot) + H * (n + dv) + rot + H * dv) * 2, 2.0 * full_pairs * H * (n + rot + dv))
+        cache = torch.randn(batch, ctx + 64, r + rot, device=dev).to(bf)
+        qd, gd = q[:batch].contiguous(), gate[:batch] if gate is not None else None
+        add(f"latent_rope_decode_attention ({fam}; ctx {ctx}, all {ctx + 1} keys)", like,
+            t(lambda: A.latent_rope_decode_attention(qd, a, wu, sk, cache, lens_l, None, gate=gd)),
+            batch * (ctx + 1) * (r + rot) * 2 + H * (n + dv) * r * 4, 2.0 * batch * H * ((ctx + 1) * (2 * r + rot) + (n + dv) * r))
+    return rows
+
+
 def run(design: str, sizes: List[str] = None, n_layers: int = 4) -> List[dict]:
-    assert design in ("rapodra", "tizodra", "defilorn", "buvesun")
+    assert design in ("rapodra", "tizodra", "defilorn", "buvesun", "tokatar")
     dev = torch.device("cuda:0")
     torch.cuda.set_device(dev)
     peaks = dict(hbm_gbs=6650.0, bf16_tflops=1590.0, source="fallback")
@@ -644,12 +804,13 @@ def run(design: str, sizes: List[str] = None, n_layers: int = 4) -> List[dict]:
         if "hbm_gbs" in d and "bf16_tflops" in d:
             peaks = dict(hbm_gbs=float(d["hbm_gbs"]), bf16_tflops=float(d["bf16_tflops"]), source="measured")
     results = [dict(bench="peaks", **peaks)]
-    table = {"rapodra": SIZES, "tizodra": TIZODRA_SIZES, "defilorn": DEFILORN_SIZES, "buvesun": BUVESUN_SIZES}[design]
+    table = {"rapodra": SIZES, "tizodra": TIZODRA_SIZES, "defilorn": DEFILORN_SIZES, "buvesun": BUVESUN_SIZES,
+             "tokatar": TOKATAR_SIZES}[design]
     for name in sizes or list(table):
         s = table[name]
         results += model_numbers(name, s, n_layers, batch=32, prompt_len=1024, new_tokens=33, dev=dev, design=design)
         kn = {"rapodra": kernel_numbers, "tizodra": tizodra_kernel_numbers, "defilorn": defilorn_kernel_numbers,
-              "buvesun": buvesun_kernel_numbers}[design]
+              "buvesun": buvesun_kernel_numbers, "tokatar": tokatar_kernel_numbers}[design]
         results += kn(name, s, batch=32, prompt_len=1024, ctx=2048, dev=dev, peaks=peaks)
     for r in results:
         print(json.dumps(r), flush=True)

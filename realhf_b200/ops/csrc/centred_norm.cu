@@ -39,7 +39,8 @@ struct NormParams {
   const void* gate; int64_t ldg; int dtg;   // [T, W] gate logits or null
 };
 
-RB_DEVICE float sig(float x) { return 1.f / (1.f + expf(-x)); }
+// fast intrinsics, fp32 accuracy (a few ulp): with exact expf and division the gate cost as much as the rest of the kernel
+RB_DEVICE float sig(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 RB_DEVICE float4 ld4_w(const NormParams& p, const void* w, int e) {
   if (!p.w_one) return rb::ld4_any(w, p.dtw, e);
   const float v = ld_any(w, p.dtw, 0);

@@ -575,6 +575,7 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
 #pragma unroll
     for (int i = 0; i < 8; ++i) acc[r][i] = 0.f;
   }
+  const float cap2 = p.softcap > 0.f ? 2.f / p.softcap : 0.f;
   const unsigned gmask = (LPR == 32) ? 0xffffffffu : (((1u << LPR) - 1u) << (rsel * LPR));
   auto consume = [&](const float* kf, const float* vf, int idx) {
     const float dist = (float)(n - pos_of(idx));
@@ -585,7 +586,7 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
       for (int i = 0; i < 8; ++i) s = fmaf(q[r][i], kf[i], s);
 #pragma unroll
       for (int o = LPR / 2; o > 0; o >>= 1) s += __shfl_xor_sync(gmask, s, o, LPR);
-      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      if (p.softcap > 0.f) s = p.softcap - __fdividef(2.f * p.softcap, 1.f + __expf(fminf(s * cap2, 80.f)));   // cap tanh(s / cap)
       s -= slope[r] * dist;
       const float mn = fmaxf(m[r], s);
       const float corr = (m[r] == -INFINITY) ? 0.f : __expf(m[r] - mn), pr = __expf(s - mn);

@@ -1,5 +1,5 @@
 // What happens to a token's projection row before, and to its attention output after, the attention itself (`WindowAttentionConfig`
-// with rotary / full_norm / value_rotary).  fp32 arithmetic with exact sincosf / expf whatever the storage type (compiled without
+// with rotary / full_norm / value_rotary).  fp32 arithmetic with exact sincosf whatever the storage type (compiled without
 // fast-math); one CTA per token, whose cos / sin tables (fp32 position x fp32 frequency) are formed once in shared memory.
 //
 //   window_prepare   row [q (H d) | k (G d) | v (G dv) | ..] in place: q and k divided by their root mean square over ALL their heads
@@ -20,7 +20,7 @@ namespace {
 using rb::ld_any;
 using rb::st_any;
 
-constexpr int kThreads = 256, kMaxHalf = 512;
+constexpr int kThreads = 128, kMaxHalf = 512;
 
 template <int V> RB_DEVICE void ldn(const void* p, int dt, int64_t i, float* f) {
   if constexpr (V == 4) {
@@ -34,6 +34,8 @@ template <int V> RB_DEVICE void stn(void* p, int dt, int64_t i, const float* f) 
   if constexpr (V == 4) rb::st4_any(p, dt, i, make_float4(f[0], f[1], f[2], f[3]));
   else st_any(p, dt, i, f[0]);
 }
+
+RB_DEVICE float sig(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }   // fp32 accuracy (a few ulp)
 
 RB_DEVICE int row_position(const int* pos, const int* lens, const int* slots, int64_t t) {
   if (pos != nullptr) return pos[t];
@@ -191,9 +193,9 @@ __global__ void __launch_bounds__(kThreads) turn_gate_kernel(void* __restrict__ 
           [=](int e, float* a, int m) {
             if (gmode == 2 && m == 4) {
               const float4 g = rb::ld4_any(gate, dt, t * gld + e);
-              a[0] /= 1.f + expf(-g.x); a[1] /= 1.f + expf(-g.y); a[2] /= 1.f + expf(-g.z); a[3] /= 1.f + expf(-g.w);
+              a[0] *= sig(g.x); a[1] *= sig(g.y); a[2] *= sig(g.z); a[3] *= sig(g.w);
             } else if (gmode != 0) {
-              for (int i = 0; i < m; ++i) a[i] /= 1.f + expf(-ld_any(gate, dt, t * gld + (gmode == 1 ? (e + i) / dv : e + i)));
+              for (int i = 0; i < m; ++i) a[i] *= sig(ld_any(gate, dt, t * gld + (gmode == 1 ? (e + i) / dv : e + i)));
             }
             if (m == 4) { stn<4>(x, dt, base + e, a); return; }
             for (int i = 0; i < m; ++i) st_any(x, dt, base + e + i, a[i]);
