@@ -555,6 +555,7 @@ def _sink_tc_ok(qkvg, v_n, a) -> bool:
     weights rounded to the operand type for the P.V product); `REAL_WINDOW_ATTN=simt` selects the all-fp32 CUDA-core kernel."""
     return (os.environ.get("REAL_WINDOW_ATTN", "tcgen05") == "tcgen05" and qkvg.dtype in (torch.bfloat16, torch.float16)
             and a.qk_dim == a.v_dim and a.qk_dim in (64, 128) and qkvg.stride(0) % 8 == 0 and qkvg.data_ptr() % 16 == 0
+            and not (a.softcap is not None and (a.head_temp or a.keep_first or a.scale <= 0))
             and (a.n_heads * a.qk_dim) % 8 == 0 and v_n.data_ptr() % 16 == 0 and v_n.stride(0) % 8 == 0)
 
 

@@ -32,8 +32,10 @@
 // first by all three roles), a per-head sink logit that starts the running maximum with denominator 1, and the row's output
 // times sigmoid(gate logit of its head, or of the output element).  `chunk` > 0 replaces the window: a query sees the keys of its own
 // chunk of positions up to itself (the tiles below the first row's chunk are not walked, a later row's chunk start is its lower
-// mask edge).  kCap: score = softcap * tanh(s * scale / softcap); the cap is monotone, so the row maximum is taken before it and
-// capped once, and only the pass that forms the weights evaluates tanh per element.
+// mask edge).  kSimple: no distance term, no temperature, no kept first keys and a positive scale: the row maximum is taken over the raw
+// products and scaled once, a weight costs one FMA and one exp2, the mask one comparison.  kCap (kSimple only): score = softcap *
+// tanh(s * scale / softcap); the cap is monotone, so the raw maximum is capped once, and only the pass that forms the weights
+// evaluates tanh per element.
 #include "gemm_common.cuh"
 
 namespace {
@@ -88,11 +90,13 @@ template <> RB_DEVICE uint32_t pack2<__half>(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
-// cap * tanh(t / cap) in the log2 domain (times log2 e), tanh(x) = 1 - 2 / (1 + 2^(2 x log2 e)): c = 2 log2 e / cap, k = cap log2 e.
-// Absolute error a few ulp of k; saturates to +-k.
-RB_DEVICE float soft_cap2(float t, float c, float k) { return k - __fdividef(2.f * k, 1.f + exp2f(fminf(t * c, 80.f))); }
+// cap * tanh(s * scale / cap) + add in the log2 domain, tanh(x) = 1 - 2 / (1 + 2^(2 x log2 e)): c = 2 log2 e * scale / cap,
+// k = cap log2 e, k_add = k + add.  Absolute error a few ulp of k; saturates to +-k.
+RB_DEVICE float soft_cap2(float s, float c, float k, float k_add) {
+  return fmaf(-2.f * k, __fdividef(1.f, 1.f + exp2f(fminf(s * c, 80.f))), k_add);
+}
 
-template <int kD, typename T, int kFmt, bool kSink = false, bool kCap = false>
+template <int kD, typename T, int kFmt, bool kSink = false, bool kCap = false, bool kSimple = false>
 __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q,
                                                                    const __grid_constant__ CUtensorMap tma_k,
                                                                    const __grid_constant__ CUtensorMap tma_v, AttnParams p) {
@@ -229,12 +233,12 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
     const int row_lo = (kSink && chunk > 0) ? q_pos / chunk * chunk : win > 0 ? q_pos - win + 1 : 0;   // first visible key of the row
     const int last_lo = (kSink && chunk > 0) ? (q0 + kBQ - 1) / chunk * chunk : q0 + kBQ - win;      // of the tile's last row
     const bool bounded = win > 0 || (kSink && chunk > 0);
-    const float cap_c = kCap ? 2.f * 1.4426950408889634f / p.softcap : 0.f, cap_k = kCap ? p.softcap * 1.4426950408889634f : 0.f;
+    const float cap_c = kCap ? 2.f * 1.4426950408889634f * p.scale / p.softcap : 0.f, cap_k = kCap ? p.softcap * 1.4426950408889634f : 0.f;
     // kSink: scores live in the log2 domain, t = s * c2 - slope2 * (q_pos - key_pos); the sink starts the maximum
     float c2 = 0.f, slope2 = 0.f;
     if constexpr (kSink) {
-      c2 = (kCap ? p.scale : sl2) * (p.temp ? rb::to_f(reinterpret_cast<const T*>(p.temp)[head]) : 1.f);   // (kCap: natural units until the cap)
-      slope2 = p.slope_base >= 0.f ? exp2f(-p.slope_base * (float)(head + 1) / (float)p.nq) * 1.4426950408889634f : 0.f;
+      c2 = sl2 * (p.temp ? rb::to_f(reinterpret_cast<const T*>(p.temp)[head]) : 1.f);
+      if constexpr (!kSimple) slope2 = p.slope_base >= 0.f ? exp2f(-p.slope_base * (float)(head + 1) / (float)p.nq) * 1.4426950408889634f : 0.f;
       if (p.sink) { m_run = rb::to_f(reinterpret_cast<const T*>(p.sink)[head]) * 1.4426950408889634f; l_run = 1.f; }
     }
     float O[kD];
@@ -269,7 +273,11 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
       const int lim = (p.causal ? min(L, q_pos + 1) : L) - kv0;  // local key columns [lo, lim) are visible to this row
       const int lo = bounded ? row_lo - kv0 : 0;
       const int kept = kSink ? p.keep - kv0 : 0;                 // kSink: local columns below `kept` stay visible under `lo`
-      auto hidden = [&](int col) { return col >= lim || (col < lo && (!kSink || col >= kept)); };
+      const uint32_t n_vis = (uint32_t)max(lim - lo, 0);
+      auto hidden = [&](int col) {
+        if constexpr (kSimple) return (uint32_t)(col - lo) >= n_vis;
+        return col >= lim || (col < lo && (!kSink || col >= kept));
+      };
       const float base = kSink ? slope2 * (float)(kv0 - q_pos) : 0.f;
       float mx = -INFINITY;
 #pragma unroll
@@ -280,13 +288,14 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           float s = __uint_as_float(r[i]);
-          if constexpr (kCap) s *= c2;
-          else if constexpr (kSink) s = fmaf(s, c2, fmaf(slope2, (float)(c * 32 + i), base));
+          if constexpr (kSink && !kSimple) s = fmaf(s, c2, fmaf(slope2, (float)(c * 32 + i), base));
           if (need_mask && hidden(c * 32 + i)) s = -INFINITY;
           mx = fmaxf(mx, s);
         }
       }
-      if constexpr (kCap) { if (mx != -INFINITY) mx = soft_cap2(mx, cap_c, cap_k); }
+      if constexpr (kSimple) {
+        if (mx != -INFINITY) mx = kCap ? soft_cap2(mx, cap_c, cap_k, cap_k) : mx * c2;
+      }
       const float m_new = fmaxf(m_run, mx);
       const float m_eff = (m_new == -INFINITY) ? 0.f : m_new;  // fully masked so far: keep exp2 arguments finite
       const float alpha = kSink ? exp2f(m_run - m_eff) : exp2f((m_run - m_eff) * sl2);
@@ -303,8 +312,11 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
         for (int i = 0; i < 32; i += 2) {
           float e0, e1;
           if constexpr (kCap) {
-            e0 = exp2f(soft_cap2(__uint_as_float(r[i]) * c2, cap_c, cap_k) + neg_m);
-            e1 = exp2f(soft_cap2(__uint_as_float(r[i + 1]) * c2, cap_c, cap_k) + neg_m);
+            e0 = exp2f(soft_cap2(__uint_as_float(r[i]), cap_c, cap_k, cap_k + neg_m));
+            e1 = exp2f(soft_cap2(__uint_as_float(r[i + 1]), cap_c, cap_k, cap_k + neg_m));
+          } else if constexpr (kSimple) {
+            e0 = exp2f(fmaf(__uint_as_float(r[i]), c2, neg_m));
+            e1 = exp2f(fmaf(__uint_as_float(r[i + 1]), c2, neg_m));
           } else if constexpr (kSink) {
             e0 = exp2f(fmaf(__uint_as_float(r[i]), c2, fmaf(slope2, (float)(c * 32 + i), base)) + neg_m);
             e1 = exp2f(fmaf(__uint_as_float(r[i + 1]), c2, fmaf(slope2, (float)(c * 32 + i + 1), base)) + neg_m);
@@ -377,11 +389,11 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_fwd_kernel(const __grid_
   }
 }
 
-template <int kD, typename T, int kFmt, bool kSink = false, bool kCap = false>
+template <int kD, typename T, int kFmt, bool kSink = false, bool kCap = false, bool kSimple = false>
 int launch_attn_fwd(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnParams& p, int B,
                     int max_seqlen, cudaStream_t s) {
   using C = ACfg<kD>;
-  auto kern = attn_fwd_kernel<kD, T, kFmt, kSink, kCap>;
+  auto kern = attn_fwd_kernel<kD, T, kFmt, kSink, kCap, kSimple>;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmemBytes) != cudaSuccess) return -30;
@@ -430,7 +442,7 @@ extern "C" int rb_attn_fwd(const void* q, const void* k, const void* v, void* ou
 // Window attention with a sink on the tensor cores (see the kSink notes at the top): q / k / v as for rb_attn_fwd (equal query /
 // value head size of 64 or 128), temp / sink [nq] in the operand type or null, gate logits at gate[t * gate_ld + h] (gate_mode 1) or
 // gate[t * gate_ld + h * hd + c] (gate_mode 2) or null, window <= 0 = every earlier key, keep = first keys that stay visible,
-// chunk > 0 = chunked instead of windowed, softcap > 0 = capped scores (no distance term then), slope_base < 0 = no distance term.
+// chunk > 0 = chunked instead of windowed, softcap > 0 = capped scores (kSimple cases only), slope_base < 0 = no distance term.
 extern "C" int rb_attn_fwd_sink(const void* q, const void* k, const void* v, void* out, const int* cu_seqlens, int64_t q_ld, int64_t k_ld,
                                 int64_t v_ld, int64_t out_ld, int T, int B, int nq, int nkv, int hd, int max_seqlen, float scale, int window,
                                 int keep, const void* temp, const void* sink, const void* gate, int64_t gate_ld, int gate_mode, int chunk,
@@ -441,7 +453,8 @@ extern "C" int rb_attn_fwd_sink(const void* q, const void* k, const void* v, voi
   if ((q_ld | k_ld | v_ld | out_ld) % 8 != 0) return -4;
   if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)out) & 15) return -5;
   if (gate != nullptr && gate_mode == 2 && (gate_ld % 8 != 0 || ((uintptr_t)gate & 15))) return -6;
-  if (softcap > 0.f && slope_base >= 0.f) return -7;
+  const bool simple = slope_base < 0.f && temp == nullptr && scale > 0.f && (window <= 0 || keep == 0);
+  if (softcap > 0.f && !simple) return -7;
   if (chunk > 0 && window > 0) return -8;
   CUtensorMap mq, mk, mv;
   const int bf = dt == 1;
@@ -450,13 +463,14 @@ extern "C" int rb_attn_fwd_sink(const void* q, const void* k, const void* v, voi
   if (!make_tmap(&mv, v, bf, T, (uint64_t)(nkv / vshare) * hd, v_ld, 64, 64)) return -12;
   AttnParams p{cu_seqlens, out, nullptr, out_ld, T, nq, nkv, scale, 1, window > 0 ? window : 0, window > 0 ? keep : 0, temp, sink, gate, gate_ld,
                slope_base, vshare, gate_mode, chunk, softcap};
-#define RB_GO(CAP)                                                                                                \
-  if (hd == 128)                                                                                                  \
-    return bf ? launch_attn_fwd<128, __nv_bfloat16, 1, true, CAP>(mq, mk, mv, p, B, max_seqlen, s)               \
-              : launch_attn_fwd<128, __half, 0, true, CAP>(mq, mk, mv, p, B, max_seqlen, s);                      \
-  return bf ? launch_attn_fwd<64, __nv_bfloat16, 1, true, CAP>(mq, mk, mv, p, B, max_seqlen, s)                  \
-            : launch_attn_fwd<64, __half, 0, true, CAP>(mq, mk, mv, p, B, max_seqlen, s)
-  if (softcap > 0.f) { RB_GO(true); }
-  RB_GO(false);
+#define RB_GO(CAP, SIMPLE)                                                                                                \
+  if (hd == 128)                                                                                                          \
+    return bf ? launch_attn_fwd<128, __nv_bfloat16, 1, true, CAP, SIMPLE>(mq, mk, mv, p, B, max_seqlen, s)               \
+              : launch_attn_fwd<128, __half, 0, true, CAP, SIMPLE>(mq, mk, mv, p, B, max_seqlen, s);                      \
+  return bf ? launch_attn_fwd<64, __nv_bfloat16, 1, true, CAP, SIMPLE>(mq, mk, mv, p, B, max_seqlen, s)                  \
+            : launch_attn_fwd<64, __half, 0, true, CAP, SIMPLE>(mq, mk, mv, p, B, max_seqlen, s)
+  if (softcap > 0.f) { RB_GO(true, true); }
+  if (simple) { RB_GO(false, true); }
+  RB_GO(false, false);
 #undef RB_GO
 }
