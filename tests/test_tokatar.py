@@ -29,7 +29,7 @@ EXACT = [CPU, GPU32]
 
 
 def tol(dtype):
-    return 2e-4 if dtype == torch.float32 else 0.12
+    return 2e-4 if dtype == torch.float32 else 0.04
 
 
 def row_errs(got, want):
