@@ -298,3 +298,4 @@ from realhf_b200.api.from_hf import tizodra  # noqa: E402,F401  (registers the f
 from realhf_b200.api.from_hf import defilorn  # noqa: E402,F401  (registers the family)
 from realhf_b200.api.from_hf import buvesun  # noqa: E402,F401  (registers the family)
 from realhf_b200.api.from_hf import tokatar  # noqa: E402,F401  (registers the family)
+from realhf_b200.api.from_hf import nufatar  # noqa: E402,F401  (registers the family)

@@ -202,6 +202,9 @@ class WindowAttentionConfig:
         per output element (n_heads * v_dim) and the concatenated heads are multiplied element by element;
       * `qk_norm`: every query / key head is RMS-normalised over qk_dim with a weight (one for queries, one for keys); with
         `full_norm` all query heads (all key heads) of a token are one vector with one root mean square, the weights span them;
+      * `kv_shared`: the values are the keys as projected (no value projection, one cache); needs v_dim = qk_dim;
+      * `bias_rows` B > 0: a learned number per head and distance bucket is added to the scaled score (`scale` and the temperature do
+        not multiply it), from a table [B, n_heads]; `distance_buckets` maps distances to rows, logarithmically up to `bias_max`;
       * `value_rotary`: value heads are rotated by their position too (and cached rotated), and every head's output is turned back by
         the query's position before the gate: the output then depends on distances only;
       * `n_maps` = 2: differential attention.  Queries and keys have two maps per head ([map 1 | map 2], 2 qk_dim wide), each a
@@ -230,8 +233,17 @@ class WindowAttentionConfig:
     element_gate: bool = False
     full_norm: bool = False
     value_rotary: Optional[RotaryConfig] = None
+    kv_shared: bool = False
+    bias_rows: int = 0
+    bias_max: float = 0.0
 
     def __post_init__(self):
+        if self.kv_shared and (self.v_dim != self.qk_dim or self.value_norm or self.rotary is not None or self.value_rotary is not None
+                               or self.n_maps != 1 or self.qk_norm):
+            raise ValueError("kv_shared: v_dim = qk_dim, keys and values as projected (no norm, no rotation), one score map")
+        if self.bias_rows and (self.bias_rows < 2 or self.bias_max <= self.bias_rows // 2 or self.slope_base is not None or self.softcap is not None
+                               or self.n_maps != 1):
+            raise ValueError("bias_rows: at least 2, bias_max > bias_rows / 2, without another distance term, a cap or a second map")
         if isinstance(self.rotary, dict):
             self.rotary = RotaryConfig(**self.rotary)
         if isinstance(self.value_rotary, dict):
@@ -279,7 +291,30 @@ class WindowAttentionConfig:
     @property
     def prepared(self) -> bool:
         """Query / key norm, rotations and cache rows of a token are one kernel (`ops.attention.window_prepare_`)."""
-        return self.n_maps == 1 and (self.full_norm or self.value_rotary is not None or (self.rotary is not None and not self.value_norm))
+        return self.n_maps == 1 and (self.full_norm or self.value_rotary is not None or not self.value_norm)
+
+    @property
+    def turns(self) -> bool:
+        """That kernel has work to do on a decoded token's row (else it only stores a prompt's cache rows)."""
+        return self.full_norm or self.rotary is not None or self.value_rotary is not None
+
+    @property
+    def value_width(self) -> int:
+        """Columns of the value section of the projection row."""
+        return 0 if self.kv_shared else self.n_kv_heads * self.v_dim
+
+    def distance_buckets(self) -> List[int]:
+        """Row of the bias table for the distances 0, 1, ..; every distance beyond the list reads the last entry.  With B rows, exact
+        rows below B / 2, then B / 2 + floor(ln(n / (B / 2)) / ln(bias_max / (B / 2)) (B - B / 2)), at most B - 1."""
+        import math
+        B, half = self.bias_rows, self.bias_rows // 2
+        out, n = [], 0
+        while True:
+            b = n if n < half else min(B - 1, half + math.floor(math.log(n / half) / math.log(self.bias_max / half) * (B - half)))
+            out.append(b)
+            if b == B - 1:
+                return out
+            n += 1
 
 
 @dataclasses.dataclass
@@ -288,15 +323,22 @@ class DeltaRuleConfig:
     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q,  with a scalar decay g in (0, 1) and a write strength beta in
     (0, 1) per head and token.  q / k have `n_kv_heads` heads (head h reads q / k head h // (n_heads / n_kv_heads)), pass a causal
     depthwise convolution of `conv_taps` taps and SiLU (so does v), and are scaled to unit length; o is RMS-normalised per head
-    and gated by SiLU of a projection.  A sequence's decode state is S plus the last conv_taps - 1 projection outputs."""
+    and gated by SiLU (`gate` "silu") or sigmoid ("sigmoid") of a projection.  A sequence's decode state is S plus the last
+    conv_taps - 1 projection outputs.  With `decay_rank` the decay is one number per head and key channel (it scales the row of S that
+    belongs to the channel), its logits the product of two projections of that inner rank; with `gate_rank` the gate's are too."""
     n_heads: int
     n_kv_heads: int
     qk_dim: int
     v_dim: int
     conv_taps: int
     unit_eps: float = 1e-6         # q, k <- x / sqrt(sum(x^2) + unit_eps)
+    decay_rank: Optional[int] = None
+    gate_rank: Optional[int] = None
+    gate: str = "silu"             # silu | sigmoid
 
     def __post_init__(self):
+        if self.gate not in ("silu", "sigmoid"):
+            raise ValueError("gate: silu | sigmoid")
         if self.n_heads % self.n_kv_heads:
             raise ValueError("n_heads must be a multiple of n_kv_heads")
         if self.conv_taps < 1:
@@ -305,6 +347,16 @@ class DeltaRuleConfig:
     @property
     def conv_channels(self) -> int:
         return 2 * self.n_kv_heads * self.qk_dim + self.n_heads * self.v_dim
+
+    @property
+    def n_decays(self) -> int:
+        """Decays per token: one per head, or one per head and key channel."""
+        return self.n_heads * (self.qk_dim if self.decay_rank else 1)
+
+    @property
+    def low_rank_width(self) -> int:
+        """Outputs of the second factors (`attn.low.weight`): decay inputs, then gate logits."""
+        return (self.n_decays if self.decay_rank else 0) + (self.n_heads * self.v_dim if self.gate_rank else 0)
 
 
 @dataclasses.dataclass
@@ -364,12 +416,13 @@ class DecayConfig:
 class LoopConfig:
     """Blocks start .. stop - 1 (0-based) run `times` times in a row with the same weights, every pass with a cache / state of its
     own.  With `inject`, the embedding output x0 is mixed back in at the start of a pass: mode "linear": every pass,
-    x <- W_in [x; x0], W_in [hidden, 2 hidden]; mode "add": every pass but the first, x <- x + x0."""
+    x <- W_in [x; x0], W_in [hidden, 2 hidden]; mode "add": every pass but the first, x <- x + x0; mode "step": every pass,
+    x <- x + s_t with a learned vector per pass ([times, hidden])."""
     start: int
     stop: int
     times: int
     inject: bool = True
-    inject_mode: str = "linear"    # linear | add
+    inject_mode: str = "linear"    # linear | add | step
 
 
 @dataclasses.dataclass
@@ -398,9 +451,11 @@ class BlockConfig:
     delta: Optional[DeltaRuleConfig] = None
     mlstm: Optional[MLSTMConfig] = None
     decay: Optional[DecayConfig] = None
-    # mixer "parallel": `wattn` and `decay` read the same input side by side; the result is branch_scales[0] * window attention +
-    # branch_scales[1] * decayed linear attention (each after its own output projection)
+    # mixer "parallel": `wattn` and `decay` (or `delta`) read the same input side by side; the result is branch_scales[0] * window
+    # attention + branch_scales[1] * the recurrent side (each after its own output projection; with `branch_norm` each RMS-normalised
+    # over the model width first, with a weight)
     branch_scales: Tuple[float, float] = (1.0, 1.0)
+    branch_norm: bool = False
 
     def __post_init__(self):
         if isinstance(self.attn, dict):
@@ -415,7 +470,7 @@ class BlockConfig:
             self.decay = DecayConfig(**self.decay)
         self.branch_scales = (float(self.branch_scales[0]), float(self.branch_scales[1]))
         want = {"latent_attention": self.attn, "window_attention": self.wattn, "delta": self.delta, "mlstm": self.mlstm, "decay": self.decay,
-                "parallel": self.wattn if self.decay is not None else None}
+                "parallel": self.wattn if (self.decay is None) != (self.delta is None) else None}
         if self.mixer not in want:
             raise ValueError(f"unknown mixer `{self.mixer}`")
         if want[self.mixer] is None:
@@ -424,6 +479,13 @@ class BlockConfig:
             self.mlp = BlockMLPConfig(**self.mlp)
         if self.mlp is not None and isinstance(self.mlp.moe, dict):
             self.mlp.moe = ReaLMoEConfig(**self.mlp.moe)
+
+
+def _delta_params(a: DeltaRuleConfig, h: int) -> int:
+    nv = a.n_heads * a.v_dim
+    n = h * (2 * a.n_kv_heads * a.qk_dim + nv + a.n_heads) + nv * h + a.conv_channels * a.conv_taps + a.n_heads + a.n_decays + a.v_dim
+    n += (h + a.n_decays) * a.decay_rank if a.decay_rank else h * a.n_heads
+    return n + ((h + nv) * a.gate_rank if a.gate_rank else h * nv)
 
 
 @dataclasses.dataclass
@@ -478,6 +540,7 @@ class ReaLModelConfig:
     layer_scale: bool = False            # every branch output (after its output norm) times a learned vector (`attn.ls.weight`,
                                          # `mlp.ls.weight`) before it joins the stream (wrapped stacks, see `wrapped`)
     scalar_norm: bool = False            # the sublayers' norms and the final one have ONE learned factor instead of a vector (RMSNorm)
+    parallel_ff: bool = False            # one norm per block: x <- x + (mixer(N(x)) + ff(N(x))) (heterogeneous stacks)
     gated_residual: bool = False         # every branch output is multiplied element by element by sigmoid(W h + b), h the sublayer's
                                          # input, before its output norm (`sharding.residual_gate_fused`: where W lives)
 
@@ -494,7 +557,7 @@ class ReaLModelConfig:
             return [(i, False) for i in range(1, L + 1)]
         runs = [(i + 1, False) for i in range(lp.start)]
         for p in range(lp.times):
-            runs += [(i + 1, i == lp.start and (p > 0 or lp.inject_mode == "linear")) for i in range(lp.start, lp.stop)]
+            runs += [(i + 1, i == lp.start and (p > 0 or lp.inject_mode != "add")) for i in range(lp.start, lp.stop)]
         return runs + [(i + 1, False) for i in range(lp.stop, L)]
 
     def __post_init__(self):
@@ -505,8 +568,8 @@ class ReaLModelConfig:
                 raise ValueError("`loop` needs a heterogeneous stack (`blocks`)")
             if not (0 <= self.loop.start < self.loop.stop <= self.n_layers and self.loop.times >= 1):
                 raise ValueError("loop: 0 <= start < stop <= n_layers and times >= 1 expected")
-            if self.loop.inject_mode not in ("linear", "add"):
-                raise ValueError("loop.inject_mode: linear | add")
+            if self.loop.inject_mode not in ("linear", "add", "step"):
+                raise ValueError("loop.inject_mode: linear | add | step")
         if self.is_critic and self.tied_embedding:
             raise ValueError("a critic cannot tie its embedding and output weights")
         if self.blocks is not None:
@@ -515,13 +578,20 @@ class ReaLModelConfig:
                 raise ValueError("`blocks` must describe every layer")
             if self.wrapped and (self.norm_groups != 1 or self.conv_taps or not self.sandwich_norm or self.layer_norm_type not in ("layer", "rms")):
                 raise ValueError("wrapped stacks: one norm group, no convolution, norms (\"layer\" or \"rms\") on both sides of every sublayer")
-            if not self.wrapped and (self.residual_mult != 1.0 or any(b.mixer in ("decay", "parallel") for b in self.blocks)):
-                raise ValueError("residual_mult and the decay / parallel mixers live in wrapped stacks")
+            if self.parallel_ff and (self.wrapped or self.norm_groups != 1 or self.sandwich_norm or self.conv_taps
+                                     or self.layer_norm_type not in ("rms", "gemma")):
+                raise ValueError("parallel_ff: one RMSNorm (\"rms\" or \"gemma\") per block and nothing else around its sublayers")
+            if not self.wrapped and (self.residual_mult != 1.0 or (not self.parallel_ff and any(b.mixer in ("decay", "parallel") for b in self.blocks))):
+                raise ValueError("residual_mult lives in wrapped stacks, the decay / parallel mixers there and in parallel_ff stacks")
+            if not self.parallel_ff and any(b.branch_norm for b in self.blocks):
+                raise ValueError("branch_norm lives in parallel_ff stacks")
             if self.scalar_norm and self.layer_norm_type != "rms":
                 raise ValueError("scalar_norm is a form of RMSNorm")
             for i, b in enumerate(self.blocks):
                 if b.mixer != "latent_attention":
                     continue
+                if self.parallel_ff and not b.attn.rotated:
+                    raise ValueError("parallel_ff stacks take latent attention in its rotated form")
                 if b.attn.rotated and not self.wrapped and (self.norm_groups != 1 or self.sandwich_norm or self.conv_taps):
                     raise ValueError("rotated latent attention lives in plain pre-norm and in wrapped stacks")
                 if self.wrapped and not b.attn.rotated:
@@ -539,7 +609,7 @@ class ReaLModelConfig:
         """Parameter count (used by the PP partitioner, the FLOP model and the allocation search)."""
         h, f, v = self.hidden_dim, self.intermediate_dim, self.vocab_size
         if self.blocks is not None:
-            n = 2 * v * h + (1 if self.scalar_norm else h)
+            n = (1 if self.tied_embedding else 2) * v * h + (1 if self.scalar_norm else h)
             # per sublayer, in units of h: norm(s), taps, scale, residual gate (a matrix and a bias)
             norms = (2 if self.sandwich_norm else 1) + self.conv_taps + int(self.layer_scale) + (h + 1 if self.gated_residual else 0)
             if self.scalar_norm:
@@ -547,22 +617,24 @@ class ReaLModelConfig:
                 n += 2 * (len(self.blocks) + sum(b.mlp is not None for b in self.blocks))
             for b in self.blocks:
                 if b.mixer in ("decay", "parallel"):
-                    a = b.decay
-                    n += h * a.width + a.n_heads * a.v_dim * (h + (1 if a.out_norm == "full" else 0)) + norms * h
+                    if b.decay is not None:
+                        a = b.decay
+                        n += h * a.width + a.n_heads * a.v_dim * (h + (1 if a.out_norm == "full" else 0)) + norms * h
+                    else:
+                        n += _delta_params(b.delta, h) + norms * h
                     if b.mixer == "parallel":
                         w = b.wattn
-                        n += h * (w.n_heads * w.qk_dim + w.n_kv_heads * (w.qk_dim + w.v_dim)) + w.n_heads * w.v_dim * h
+                        n += h * (w.n_heads * w.qk_dim + w.n_kv_heads * w.qk_dim + w.value_width) + w.n_heads * w.v_dim * h
+                        n += w.n_heads * (int(w.sink) + w.bias_rows) + (2 * h if b.branch_norm else 0)
                 elif b.mixer == "window_attention":
                     a = b.wattn
-                    qkv = a.n_heads * a.qk_dim + a.n_kv_heads * (a.qk_dim + a.v_dim)
+                    qkv = a.n_heads * a.qk_dim + a.n_kv_heads * a.qk_dim + a.value_width
                     qkv += (a.n_maps - 1) * (a.n_heads + a.n_kv_heads) * a.qk_dim
                     n += h * (qkv + a.gate_width) + (qkv if a.qkv_bias else 0) + a.n_heads * a.v_dim * h
-                    n += a.n_heads * (int(a.head_temp) + int(a.sink)) + norms * h
+                    n += a.n_heads * (int(a.head_temp) + int(a.sink) + a.bias_rows) + norms * h
                     n += ((a.n_heads + a.n_kv_heads if a.full_norm else 2) * a.qk_dim if a.qk_norm else 0) + (4 * a.qk_dim if a.n_maps == 2 else 0)
                 elif b.mixer == "delta":
-                    a = b.delta
-                    n += h * (2 * a.n_kv_heads * a.qk_dim + 2 * a.n_heads * a.v_dim + 2 * a.n_heads) + a.n_heads * a.v_dim * h
-                    n += a.conv_channels * a.conv_taps + 2 * a.n_heads + a.v_dim + norms * h
+                    n += _delta_params(b.delta, h) + norms * h
                 elif b.mixer == "mlstm":
                     a = b.mlstm
                     n += h * (2 * a.n_heads * a.qk_dim + 2 * a.n_heads * a.v_dim + 2 * a.n_heads) + 2 * a.n_heads
@@ -580,7 +652,7 @@ class ReaLModelConfig:
                 if b.mlp is not None:
                     e = b.mlp.moe.num_experts if b.mlp.kind == "moe" else 1
                     mats = 2 if b.mlp.kind == "relu2" else 3
-                    n += e * mats * h * b.mlp.ff + norms * h
+                    n += e * mats * h * b.mlp.ff + (0 if self.parallel_ff else norms * h)
                     if b.mlp.kind == "moe":
                         mo = b.mlp.moe
                         if mo.routing_type in ("softmax_all", "sigmoid"):
@@ -590,6 +662,8 @@ class ReaLModelConfig:
                             n += e * (h + 1)
             if self.loop is not None and self.loop.inject and self.loop.inject_mode == "linear":
                 n += 2 * h * h
+            if self.loop is not None and self.loop.inject and self.loop.inject_mode == "step":
+                n += self.loop.times * h
             return n
         qkv = h * self.head_dim * (self.n_q_heads + 2 * self.n_kv_heads)
         attn = qkv + self.n_q_heads * self.head_dim * h
@@ -827,15 +901,18 @@ class HFFamilySpec:
     config_from_dict: Optional[Callable[[dict, bool], ReaLModelConfig]] = None
     config_to_dict: Optional[Callable[[ReaLModelConfig], dict]] = None
     weight_file: Optional[str] = None
+    # sizes that a checkpoint's tensors carry and its `config.json` does not: (config dict, tensor name -> shape) -> completed dict
+    config_from_shapes: Optional[Callable[[dict, Dict[str, Tuple[int, ...]]], dict]] = None
 
 
 def register_hf_family(name: str, hf_cls_name: str, config_from_hf_converter, config_to_hf_converter,
                        sd_from_hf_converter, sd_to_hf_converter, embedding_param_names, tblock_param_names,
                        head_param_names, real_config_maker=None, make_test_config=None, config_from_dict=None, config_to_dict=None,
-                       weight_file=None):
+                       weight_file=None, config_from_shapes=None):
     if name in SUPPORTED_HF_FAMILIES:
         raise KeyError(f"HF family `{name}` already registered")
     SUPPORTED_HF_FAMILIES[name] = HFFamilySpec(name, hf_cls_name, config_from_hf_converter, config_to_hf_converter,
                                                sd_from_hf_converter, sd_to_hf_converter, embedding_param_names,
                                                tblock_param_names, head_param_names, make_test_config,
-                                               real_config_maker, config_from_dict, config_to_dict, weight_file)
+                                               real_config_maker, config_from_dict, config_to_dict, weight_file,
+                                               config_from_shapes)

@@ -118,14 +118,19 @@ class DecodeState:
             from realhf_b200.models import hetero_block as HB
             first = model.layers[0] if model.layers[0] >= 1 else 1
             self.k, self.v = [], []
-            self.m: List[Optional[torch.Tensor]] = []   # a third state tensor per run for blocks that hold one (mixer "parallel"), else None
+            self.m: list = []   # per run: what a block holds beside k and v (mixer "parallel": a tensor or a tuple of tensors), else None
             # tensors a slot's allocation zeroes / a decode step changes beyond an idempotent append: (tensor, slot dim)
             self.zeroed: List[Tuple[torch.Tensor, int]] = []
             run_of_block = {}
             for r, (i, _) in enumerate(model.local_runs()):
                 b = c.blocks[i - 1]
                 self.m.append(None)
-                if b.mixer in ("decay", "parallel"):
+                if b.mixer == "parallel" and b.delta is not None:
+                    d = b.delta
+                    self.m[-1] = (torch.zeros(B, d.n_heads, d.qk_dim, d.v_dim, dtype=torch.float32, device=dev),
+                                  torch.zeros(B, d.conv_taps - 1, d.conv_channels, dtype=torch.float32, device=dev))
+                    self.zeroed += [(t, 0) for t in self.m[-1]]
+                elif b.mixer in ("decay", "parallel"):
                     d = b.decay
                     mat = torch.zeros(B, d.n_heads, d.qk_dim, d.v_dim, dtype=torch.float32, device=dev)
                     self.zeroed.append((mat, 0))
@@ -138,7 +143,7 @@ class DecodeState:
                     w = b.wattn
                     rows = w.cache_rows(S)
                     self.k.append(torch.zeros(B, w.n_kv_heads * w.n_maps, rows, w.qk_dim, dtype=dt, device=dev))   # every map's keys
-                    self.v.append(torch.zeros(B, w.n_kv_heads, rows, w.v_dim, dtype=dt, device=dev))
+                    self.v.append(self.k[-1] if w.kv_shared else torch.zeros(B, w.n_kv_heads, rows, w.v_dim, dtype=dt, device=dev))
                     continue
                 if b.mixer == "mlstm":
                     ml = b.mlstm
@@ -184,6 +189,13 @@ class DecodeState:
         self.unfinished = torch.ones(B, dtype=torch.bool, device=dev)
         self.seed = torch.zeros(1, dtype=torch.long, device=dev)
         self.tok_hist = self.lp_hist = self.mask_hist = None
+
+    def state_tensors(self) -> List[torch.Tensor]:
+        """Every state tensor of every run, in a fixed order (a tensor that two entries share is listed twice)."""
+        out = self.k + self.v
+        for m in getattr(self, "m", []):
+            out = out + (list(m) if isinstance(m, tuple) else [m] if m is not None else [])
+        return out
 
     # ---- slot manager: a slot is one row of every state tensor
     def alloc(self, n: int) -> List[int]:
@@ -298,8 +310,8 @@ class StepSession:
         B = max(2 * old.B, old.B + n_needed - len(old.free_slots))
         new = DecodeState(self.model, B, self.max_len)
         done = set()
-        for a, b_ in zip(old.k + old.v + old.m + [old.cache_lens], new.k + new.v + new.m + [new.cache_lens]):
-            if a is None or id(a) in done:
+        for a, b_ in zip(old.state_tensors() + [old.cache_lens], new.state_tensors() + [new.cache_lens]):
+            if id(a) in done:
                 continue
             done.add(id(a))
             b_.narrow(old.slot_dim(a), 0, old.B).copy_(a)

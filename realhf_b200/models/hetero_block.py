@@ -19,8 +19,14 @@ per run (`state.k[r]`, `state.v[r]`), by mixer:
   * matrix-memory LSTM: `k[r]` the states with the normaliser as last column [n_slots, H, d, dv + 1] fp32, `v[r]` the running
     maxima [n_slots, H] fp32;
   * decayed linear attention (`decay`): `k[r]` the matrix states [n_slots, H, d, dv] fp32, `v[r]` empty;
-  * `parallel` (window attention beside decayed linear attention): `k[r]`, `v[r]` the rotated keys / values as for window
-    attention, and a third tensor `state.m[r]` with the matrix states [n_slots, H, d, dv] fp32 (`m[r]` is None for other mixers).
+  * `parallel` (window attention beside decayed linear attention or a delta rule): `k[r]`, `v[r]` the rotated keys / values as for
+    window attention, and in `state.m[r]` what the recurrent side keeps: the matrix states [n_slots, H, d, dv] fp32, or with a delta rule
+    the pair (matrix states, last taps - 1 projection outputs) (`m[r]` is None for other mixers).
+Window attention whose values are its keys (`kv_shared`) has one cache: `v[r]` is `k[r]`.
+
+A `parallel_ff` stack runs  x <- x + (mixer(N(x)) + ff(N(x)))  with one norm per block.  The mixer's output (a `parallel` mixer's two
+outputs, each with its own norm when `branch_norm` is set) and the feed-forward's travel as a `PendingSum` to the kernel that forms the
+next norm (`ops.functional.branch_add_norm_`), which also adds the vector that starts a pass of a loop in mode "step".
 
 A wrapped stack (`ReaLModelConfig.wrapped`) runs  x <- x + mult * ls * N_post(sigmoid(W h + b) * mixer(h)), h = N(x),  and the same
 for the feed-forward, N being the bias-free LayerNorm (`layer_norm_type` "layer") or RMSNorm ("rms"; `scalar_norm`: with one factor
@@ -55,7 +61,7 @@ class PackedMeta:
     cu_seqlens: Optional[torch.Tensor] = None
     max_seqlen: Optional[int] = None
     seq_slot: Optional[torch.Tensor] = None   # [n_seqs] int32 state slot of every sequence (None: keep no state)
-    m: Optional[List[Optional[torch.Tensor]]] = None   # DecodeState.m
+    m: Optional[list] = None                  # DecodeState.m
 
 
 def packed_meta(cu_seqlens: torch.Tensor, total: int, slots: Optional[torch.Tensor] = None, state=None,
@@ -113,28 +119,45 @@ def _mlp(model, i: int, h: torch.Tensor, mcfg) -> torch.Tensor:
     return OF.linear(a, p[f"{i}.mlp.down.weight"])
 
 
+def _window_rows_packed(model, i: int, a, rows: torch.Tensor, meta: PackedMeta, k_cache, v_cache) -> torch.Tensor:
+    """Attention of a packed batch on the block's projection rows [q | k | v | gate] (one score map), before the output projection."""
+    c, p = model.config, model.p
+    if a.prepared:
+        if a.turns or k_cache is not None:
+            attn_ops.window_prepare_(rows, a, p.get(f"{i}.attn.q_norm.weight"), p.get(f"{i}.attn.k_norm.weight"), c.layer_norm_epsilon, pos=meta.pos,
+                                     k_cache=k_cache, v_cache=v_cache, tok_slot=meta.tok_slot, remain=meta.remain)
+        v_n = attn_ops.window_values(rows, a)
+    else:
+        if a.rotary is not None:
+            attn_ops.rotate_qk_(rows, a, pos=meta.pos)
+        v_n = attn_ops.value_norm_store(rows, a, c.layer_norm_epsilon, k_cache, v_cache, meta.tok_slot, meta.pos, meta.remain)
+    return attn_ops.sink_window_attention(rows, v_n, a, p.get(f"{i}.attn.temp.weight"), p.get(f"{i}.attn.sink.weight"), meta.pos,
+                                          meta.cu_seqlens, meta.max_seqlen, rel=p.get(f"{i}.attn.rel.weight"))
+
+
+def _window_rows_decode(model, i: int, a, rows: torch.Tensor, k_cache, v_cache, cache_lens, slots) -> torch.Tensor:
+    c, p = model.config, model.p
+    if a.prepared:
+        if a.turns:
+            attn_ops.window_prepare_(rows, a, p.get(f"{i}.attn.q_norm.weight"), p.get(f"{i}.attn.k_norm.weight"), c.layer_norm_epsilon,
+                                     cache_lens=cache_lens, slots=slots)
+    elif a.rotary is not None:
+        attn_ops.rotate_qk_(rows, a, cache_lens=cache_lens, slots=slots)
+    return attn_ops.sink_window_decode_attention(rows, a, p.get(f"{i}.attn.temp.weight"), p.get(f"{i}.attn.sink.weight"), k_cache, v_cache,
+                                                 cache_lens, slots, c.layer_norm_epsilon, rel=p.get(f"{i}.attn.rel.weight"))
+
+
 def _window_attention_packed(model, i: int, li: int, h: torch.Tensor, meta: PackedMeta) -> torch.Tensor:
     c, p = model.config, model.p
     a = c.blocks[i - 1].wattn
-    keep = meta.k is not None
+    k_cache, v_cache = (meta.k[li], meta.v[li]) if meta.k is not None else (None, None)
     qkvg = OF.linear(h, p[f"{i}.attn.qkvg.weight"], p.get(f"{i}.attn.qkvg.bias"))
     if a.n_maps == 2:
         o = attn_ops.diff_window_attention(qkvg, a, p[f"{i}.attn.q_norm.weight"], p[f"{i}.attn.k_norm.weight"], p[f"{i}.attn.lambda.weight"],
-                                           c.layer_norm_epsilon, meta.k[li] if keep else None, meta.v[li] if keep else None, meta.tok_slot,
-                                           meta.pos, meta.remain, meta.cu_seqlens, meta.max_seqlen)
+                                           c.layer_norm_epsilon, k_cache, v_cache, meta.tok_slot, meta.pos, meta.remain, meta.cu_seqlens,
+                                           meta.max_seqlen)
         return OF.linear(o, p[f"{i}.attn.o.weight"])
-    if a.prepared:
-        attn_ops.window_prepare_(qkvg, a, p.get(f"{i}.attn.q_norm.weight"), p.get(f"{i}.attn.k_norm.weight"), c.layer_norm_epsilon, pos=meta.pos,
-                                 k_cache=meta.k[li] if keep else None, v_cache=meta.v[li] if keep else None, tok_slot=meta.tok_slot,
-                                 remain=meta.remain)
-        v_n = attn_ops.window_values(qkvg, a)
-    else:
-        if a.rotary is not None:
-            attn_ops.rotate_qk_(qkvg, a, pos=meta.pos)
-        v_n = attn_ops.value_norm_store(qkvg, a, c.layer_norm_epsilon, meta.k[li] if keep else None, meta.v[li] if keep else None,
-                                        meta.tok_slot, meta.pos, meta.remain)
-    o = attn_ops.sink_window_attention(qkvg, v_n, a, p.get(f"{i}.attn.temp.weight"), p.get(f"{i}.attn.sink.weight"), meta.pos,
-                                       meta.cu_seqlens, meta.max_seqlen)
+    o = _window_rows_packed(model, i, a, qkvg, meta, k_cache, v_cache)
     return _with_residual_gate(model, i, OF.linear(o, p[f"{i}.attn.o.weight"]), qkvg)
 
 
@@ -146,41 +169,42 @@ def _window_attention_decode(model, i: int, li: int, h: torch.Tensor, k_caches, 
         o = attn_ops.diff_window_decode_attention(qkvg, a, p[f"{i}.attn.q_norm.weight"], p[f"{i}.attn.k_norm.weight"], p[f"{i}.attn.lambda.weight"],
                                                   c.layer_norm_epsilon, k_caches[li], v_caches[li], cache_lens, slots)
         return OF.linear(o, p[f"{i}.attn.o.weight"])
-    if a.prepared:
-        attn_ops.window_prepare_(qkvg, a, p.get(f"{i}.attn.q_norm.weight"), p.get(f"{i}.attn.k_norm.weight"), c.layer_norm_epsilon,
-                                 cache_lens=cache_lens, slots=slots)
-    elif a.rotary is not None:
-        attn_ops.rotate_qk_(qkvg, a, cache_lens=cache_lens, slots=slots)
-    o = attn_ops.sink_window_decode_attention(qkvg, a, p.get(f"{i}.attn.temp.weight"), p.get(f"{i}.attn.sink.weight"), k_caches[li],
-                                              v_caches[li], cache_lens, slots, c.layer_norm_epsilon)
+    o = _window_rows_decode(model, i, a, qkvg, k_caches[li], v_caches[li], cache_lens, slots)
     return _with_residual_gate(model, i, OF.linear(o, p[f"{i}.attn.o.weight"]), qkvg)
 
 
+def _delta_rows_packed(model, i: int, d, rows: torch.Tensor, meta: PackedMeta, s_state, conv_state) -> torch.Tensor:
+    """Delta rule of a packed batch on its projection rows (`sharding.delta_sections`), gated, before the output projection."""
+    p = model.p
+    low = rec_ops.delta_low(rows, d, p.get(f"{i}.attn.low.weight"))
+    u = rec_ops.delta_prepare(rows, p[f"{i}.attn.conv.weight"], p[f"{i}.attn.A_log.weight"], p[f"{i}.attn.dt_bias.weight"], d, meta.pos, conv_state,
+                              meta.tok_slot, meta.remain, low=low)
+    o = rec_ops.delta_rule_scan(u, d, meta.cu_seqlens, s_state, meta.seq_slot if s_state is not None else None)
+    return rec_ops.gated_head_norm(o, p[f"{i}.attn.o_norm.weight"], rec_ops.delta_gate(rows, low, d), model.config.layer_norm_epsilon, model.dtype,
+                                   d.gate)
+
+
+def _delta_rows_decode(model, i: int, d, rows: torch.Tensor, s_state, conv_state, slots) -> torch.Tensor:
+    p = model.p
+    low = rec_ops.delta_low(rows, d, p.get(f"{i}.attn.low.weight"))
+    u = rec_ops.delta_prepare_step(rows, p[f"{i}.attn.conv.weight"], p[f"{i}.attn.A_log.weight"], p[f"{i}.attn.dt_bias.weight"], d, conv_state, slots,
+                                   low=low)
+    o = rec_ops.delta_rule_step(u, d, s_state, slots)
+    return rec_ops.gated_head_norm(o, p[f"{i}.attn.o_norm.weight"], rec_ops.delta_gate(rows, low, d), model.config.layer_norm_epsilon, model.dtype,
+                                   d.gate)
+
+
 def _delta_packed(model, i: int, li: int, h: torch.Tensor, meta: PackedMeta) -> torch.Tensor:
-    c, p = model.config, model.p
-    d = c.blocks[i - 1].delta
-    keep = meta.k is not None
+    p = model.p
+    s_state, conv_state = (meta.k[li], meta.v[li]) if meta.k is not None else (None, None)
     proj = OF.linear(h, p[f"{i}.attn.in.weight"])
-    u = rec_ops.delta_prepare(proj, p[f"{i}.attn.conv.weight"], p[f"{i}.attn.A_log.weight"], p[f"{i}.attn.dt_bias.weight"], d, meta.pos,
-                              meta.v[li] if keep else None, meta.tok_slot, meta.remain)
-    o = rec_ops.delta_rule_scan(u, d, meta.cu_seqlens, meta.k[li] if keep else None, meta.seq_slot if keep else None)
-    return OF.linear(_delta_out(model, i, d, o, proj), p[f"{i}.attn.o.weight"])
-
-
-def _delta_out(model, i: int, d, o: torch.Tensor, proj: torch.Tensor) -> torch.Tensor:
-    g0 = 2 * d.n_kv_heads * d.qk_dim + d.n_heads * d.v_dim
-    return rec_ops.gated_head_norm(o, model.p[f"{i}.attn.o_norm.weight"], proj[:, g0:g0 + d.n_heads * d.v_dim],
-                                   model.config.layer_norm_epsilon, model.dtype)
+    return OF.linear(_delta_rows_packed(model, i, model.config.blocks[i - 1].delta, proj, meta, s_state, conv_state), p[f"{i}.attn.o.weight"])
 
 
 def _delta_decode(model, i: int, li: int, h: torch.Tensor, k_caches, v_caches, slots) -> torch.Tensor:
-    c, p = model.config, model.p
-    d = c.blocks[i - 1].delta
+    p = model.p
     proj = OF.linear(h, p[f"{i}.attn.in.weight"])
-    u = rec_ops.delta_prepare_step(proj, p[f"{i}.attn.conv.weight"], p[f"{i}.attn.A_log.weight"], p[f"{i}.attn.dt_bias.weight"], d,
-                                   v_caches[li], slots)
-    o = rec_ops.delta_rule_step(u, d, k_caches[li], slots)
-    return OF.linear(_delta_out(model, i, d, o, proj), p[f"{i}.attn.o.weight"])
+    return OF.linear(_delta_rows_decode(model, i, model.config.blocks[i - 1].delta, proj, k_caches[li], v_caches[li], slots), p[f"{i}.attn.o.weight"])
 
 
 def _mlstm_packed(model, i: int, li: int, h: torch.Tensor, meta: PackedMeta) -> torch.Tensor:
@@ -272,7 +296,7 @@ def _decay_decode(model, i: int, li: int, h: torch.Tensor, k_caches, cache_lens,
 
 
 def _parallel_split(b, proj: torch.Tensor):
-    """The fused projection row of a `parallel` block as two views: [window attention q | k | v] and [decay q | k | v | gate]."""
+    """The fused projection row of a `parallel` block as two views: [window attention q | k | v] and the recurrent side's sections."""
     from realhf_b200.models.sharding import wattn_sections
     nl = sum(wattn_sections(b.wattn))
     return proj[:, :nl], proj[:, nl:]
@@ -280,33 +304,32 @@ def _parallel_split(b, proj: torch.Tensor):
 
 def _parallel_packed(model, i: int, li: int, h: torch.Tensor, meta: PackedMeta):
     """Both branches of a `parallel` block on the packed batch, each after its own output projection."""
-    c, p = model.config, model.p
-    b = c.blocks[i - 1]
-    w, d = b.wattn, b.decay
-    keep = meta.k is not None
+    p = model.p
+    b = model.config.blocks[i - 1]
+    k_cache, v_cache, m = (meta.k[li], meta.v[li], meta.m[li]) if meta.k is not None else (None, None, None)
     left, right = _parallel_split(b, OF.linear(h, p[f"{i}.attn.in.weight"]))
-    if w.rotary is not None:
-        attn_ops.rotate_qk_(left, w, pos=meta.pos)
-    v_n = attn_ops.value_norm_store(left, w, c.layer_norm_epsilon, meta.k[li] if keep else None, meta.v[li] if keep else None, meta.tok_slot,
-                                    meta.pos, meta.remain)
-    o = attn_ops.sink_window_attention(left, v_n, w, None, None, meta.pos, meta.cu_seqlens, meta.max_seqlen)
-    y_l = OF.linear(o, p[f"{i}.attn.o.weight"])
-    s = rec_ops.decay_scan(rec_ops.decay_prepare(right, d, pos=meta.pos), d, meta.cu_seqlens, meta.m[li] if keep else None,
-                           meta.seq_slot if keep else None)
-    return BranchOut(y_l, OF.linear(_decay_branch(model, i, d, right, s), p[f"{i}.attn.o2.weight"]))
+    y_l = OF.linear(_window_rows_packed(model, i, b.wattn, left, meta, k_cache, v_cache), p[f"{i}.attn.o.weight"])
+    if b.delta is not None:
+        o = _delta_rows_packed(model, i, b.delta, right, meta, *(m if m is not None else (None, None)))
+    else:
+        d = b.decay
+        s = rec_ops.decay_scan(rec_ops.decay_prepare(right, d, pos=meta.pos), d, meta.cu_seqlens, m, meta.seq_slot if m is not None else None)
+        o = _decay_branch(model, i, d, right, s)
+    return BranchOut(y_l, OF.linear(o, p[f"{i}.attn.o2.weight"]))
 
 
 def _parallel_decode(model, i: int, li: int, h: torch.Tensor, k_caches, v_caches, m_caches, cache_lens, slots):
-    c, p = model.config, model.p
-    b = c.blocks[i - 1]
-    w, d = b.wattn, b.decay
+    p = model.p
+    b = model.config.blocks[i - 1]
     left, right = _parallel_split(b, OF.linear(h, p[f"{i}.attn.in.weight"]))
-    if w.rotary is not None:
-        attn_ops.rotate_qk_(left, w, cache_lens=cache_lens, slots=slots)
-    o = attn_ops.sink_window_decode_attention(left, w, None, None, k_caches[li], v_caches[li], cache_lens, slots, c.layer_norm_epsilon)
-    y_l = OF.linear(o, p[f"{i}.attn.o.weight"])
-    s = rec_ops.decay_step(rec_ops.decay_prepare(right, d, cache_lens=cache_lens, slots=slots), d, m_caches[li], slots)
-    return BranchOut(y_l, OF.linear(_decay_branch(model, i, d, right, s), p[f"{i}.attn.o2.weight"]))
+    y_l = OF.linear(_window_rows_decode(model, i, b.wattn, left, k_caches[li], v_caches[li], cache_lens, slots), p[f"{i}.attn.o.weight"])
+    if b.delta is not None:
+        o = _delta_rows_decode(model, i, b.delta, right, *m_caches[li], slots)
+    else:
+        d = b.decay
+        s = rec_ops.decay_step(rec_ops.decay_prepare(right, d, cache_lens=cache_lens, slots=slots), d, m_caches[li], slots)
+        o = _decay_branch(model, i, d, right, s)
+    return BranchOut(y_l, OF.linear(o, p[f"{i}.attn.o2.weight"]))
 
 
 @dataclasses.dataclass
@@ -357,6 +380,61 @@ def _first_wrapped_norm(model, i: int, x: torch.Tensor, pending) -> torch.Tensor
     return OF.centred_norm(settle(model, x, pending), w, model.config.layer_norm_epsilon, model.dtype, _rms(model.config))
 
 
+@dataclasses.dataclass
+class PendingSum:
+    """What a block of a `parallel_ff` stack still owes the stream: x += (a N1(y) + b N2(y2)) + ff [+ step], N1 / N2 RMS norms with the
+    weights w1 / w2 (None: no norm).  The kernel of the next norm adds it on the way."""
+    y: Optional[torch.Tensor] = None
+    y2: Optional[torch.Tensor] = None
+    ff: Optional[torch.Tensor] = None
+    w1: Optional[torch.Tensor] = None
+    w2: Optional[torch.Tensor] = None
+    a: float = 1.0
+    b: float = 1.0
+    step: Optional[torch.Tensor] = None
+
+
+def _add_sum(model, x: torch.Tensor, ps: PendingSum, next_w: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    c = model.config
+    return OF.branch_add_norm_(x, ps.y, ps.y2, ps.ff, c.layer_norm_epsilon, ps.a, ps.b, ps.w1, ps.w2, ps.step, next_w, norm_offset(c), model.dtype)
+
+
+def _parallel_ff_norm(model, i: int, x: torch.Tensor, pending: Optional[PendingSum]) -> torch.Tensor:
+    """The one norm of block i of a `parallel_ff` stack."""
+    c, w = model.config, model.p[f"{i}.attn.ln.weight"]
+    if pending is not None:
+        return _add_sum(model, x, pending, w)
+    return OF.sublayer_input(x, w, 1, c.layer_norm_epsilon, None, None, model.dtype, w_offset=norm_offset(c))
+
+
+def _finish_parallel_ff(model, i: int, b, x: torch.Tensor, h: torch.Tensor, y, defer: bool) -> Optional[PendingSum]:
+    p = model.p
+    out = y if isinstance(y, BranchOut) else BranchOut(y)
+    sa, sb = b.branch_scales if out.y2 is not None else (1.0, 1.0)
+    ps = PendingSum(out.y, out.y2, _mlp(model, i, h, b.mlp) if b.mlp is not None else None, p.get(f"{i}.attn.out_l.weight"),
+                    p.get(f"{i}.attn.out_r.weight"), sa, sb)
+    if defer:
+        return ps
+    _add_sum(model, x, ps)
+    return None
+
+
+def start_pass(model, i: int, x: torch.Tensor, x0: torch.Tensor, pending, n: int):
+    """Start of pass n (from 0) of the loop, right before its first block i.  Returns (x, pending): in mode "step" of a `parallel_ff`
+    stack the vector joins what the next norm kernel adds, elsewhere the stream is settled and injected into."""
+    c = model.config
+    if c.loop.inject_mode != "step":
+        return loop_inject(model, i, settle(model, x, pending), x0), None
+    step = model.p[f"{i}.loop_step.weight"][n]
+    if c.parallel_ff:
+        pending = pending if pending is not None else PendingSum()
+        pending.step = step
+        return x, pending
+    x = settle(model, x, pending)
+    OF.branch_add_norm_(x, None, None, None, c.layer_norm_epsilon, step=step)
+    return x, None
+
+
 def norm_offset(c) -> float:
     """What is added to a stored norm weight: 1 for weights stored around zero (`layer_norm_type` "gemma")."""
     return 1.0 if c.layer_norm_type == "gemma" else 0.0
@@ -374,7 +452,7 @@ def loop_inject(model, i: int, x: torch.Tensor, x0: torch.Tensor) -> torch.Tenso
 
 def plain_prenorm(c) -> bool:
     """One RMSNorm per sublayer and nothing else around it: a sublayer's residual add can wait for the next norm kernel."""
-    return not c.wrapped and c.norm_groups == 1 and not c.sandwich_norm and not c.conv_taps
+    return not c.wrapped and not c.parallel_ff and c.norm_groups == 1 and not c.sandwich_norm and not c.conv_taps
 
 
 def first_norm(model, i: int, x: torch.Tensor, pending: Optional[torch.Tensor]) -> torch.Tensor:
@@ -389,6 +467,9 @@ def settle(model, x: torch.Tensor, pending: Optional[torch.Tensor]) -> torch.Ten
     """Add a branch output that a block left pending (the caller needs the stream itself)."""
     if isinstance(pending, PendingBranch):
         _add_pending(model, x, pending)
+        return x
+    if isinstance(pending, PendingSum):
+        _add_sum(model, x, pending)
         return x
     if pending is not None:
         OF.residual_add_norm_(x, pending, None, 1, model.config.layer_norm_epsilon)
@@ -429,10 +510,13 @@ def block_packed(model, i: int, li: int, x: torch.Tensor, meta: PackedMeta, pend
     a = b.attn
     G, eps = c.norm_groups, c.layer_norm_epsilon
     keep = meta.k is not None
-    if c.wrapped:
-        h = _first_wrapped_norm(model, i, x, pending)
+    if c.wrapped or c.parallel_ff:
         mixer = {"window_attention": _window_attention_packed, "delta": _delta_packed, "mlstm": _mlstm_packed, "latent_attention": _latent_rope_packed,
                  "decay": _decay_packed, "parallel": _parallel_packed}[b.mixer]
+        if c.parallel_ff:
+            h = _parallel_ff_norm(model, i, x, pending)
+            return x, _finish_parallel_ff(model, i, b, x, h, mixer(model, i, li, h, meta), defer)
+        h = _first_wrapped_norm(model, i, x, pending)
         return x, _finish_wrapped_block(model, i, b, x, h, mixer(model, i, li, h, meta), defer)
     if b.mixer != "latent_attention" or a.rotated:
         defer = defer and plain_prenorm(c)
@@ -480,13 +564,16 @@ def _mixer_decode(model, b, i: int, li: int, h: torch.Tensor, k_caches, v_caches
 
 def block_decode(model, i: int, li: int, x: torch.Tensor, k_caches: List[torch.Tensor], v_caches: List[torch.Tensor],
                  cache_lens: torch.Tensor, slots: Optional[torch.Tensor], pending: Optional[torch.Tensor] = None, defer: bool = False,
-                 m_caches: Optional[List[Optional[torch.Tensor]]] = None):
+                 m_caches: Optional[list] = None):
     """Block i for one new token per row; x [B, H] is updated in place.  Row b lives in state slot slots[b] (None: slot b).
     Returns (x, pending) as `block_packed` does."""
     c, p = model.config, model.p
     b = c.blocks[i - 1]
     a = b.attn
     G, eps = c.norm_groups, c.layer_norm_epsilon
+    if c.parallel_ff:
+        h = _parallel_ff_norm(model, i, x, pending)
+        return x, _finish_parallel_ff(model, i, b, x, h, _mixer_decode(model, b, i, li, h, k_caches, v_caches, m_caches, cache_lens, slots), defer)
     if c.wrapped:
         h = _first_wrapped_norm(model, i, x, pending)
         return x, _finish_wrapped_block(model, i, b, x, h, _mixer_decode(model, b, i, li, h, k_caches, v_caches, m_caches, cache_lens, slots), defer)
@@ -519,6 +606,8 @@ def final_norm(model, x: torch.Tensor, pending: Optional[torch.Tensor] = None) -
         if isinstance(pending, PendingBranch):
             return _add_pending(model, x, pending, w)
         return OF.centred_norm(x, w, c.layer_norm_epsilon, model.dtype, _rms(c))
+    if isinstance(pending, PendingSum):
+        return _add_sum(model, x, pending, w)
     if pending is not None and plain_prenorm(c):
         return OF.add_rms_norm_(x, pending, w, c.layer_norm_epsilon, model.dtype, norm_offset(c))
     return OF.sublayer_input(settle(model, x, pending), w, c.norm_groups, c.layer_norm_epsilon, None, None, model.dtype, w_offset=norm_offset(c))

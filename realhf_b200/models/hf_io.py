@@ -65,7 +65,10 @@ def config_from_hf_path(family_name: str, path: str, is_critic: bool = False) ->
     fam = family(family_name)
     if fam.config_from_dict is not None:
         with open(os.path.join(path, "config.json")) as f:
-            return fam.config_from_dict(json.load(f), is_critic)
+            d = json.load(f)
+        if fam.config_from_shapes is not None:
+            d = fam.config_from_shapes(d, tensor_shapes(path))
+        return fam.config_from_dict(d, is_critic)
     fast = os.path.join(path, "real_model_config.json")
     if os.environ.get("REAL_TRUST_SAVED_MODEL_CONFIG", "1") == "1" and os.path.exists(fast):
         cfg = _config_from_saved_json(fast, family_name, is_critic)
@@ -105,6 +108,20 @@ def _weight_map(path: str) -> Dict[str, str]:
 
 from realhf_b200.base.saveload_utils import load_weight_file as _read_file  # noqa: E402
 from realhf_b200.base.saveload_utils import split_state_dict_into_shards as _split_into_files  # noqa: E402
+
+
+def tensor_shapes(path: str) -> Dict[str, Tuple[int, ...]]:
+    """Name -> shape of every tensor of a checkpoint directory (safetensors headers only; other formats are read)."""
+    out: Dict[str, Tuple[int, ...]] = {}
+    for fn in sorted(set(_weight_map(path).values())):
+        full = os.path.join(path, fn)
+        if fn.endswith(".safetensors"):
+            with open(full, "rb") as f:
+                head = json.loads(f.read(int.from_bytes(f.read(8), "little")))
+            out.update({k: tuple(v["shape"]) for k, v in head.items() if k != "__metadata__"})
+        else:
+            out.update({k: tuple(v.shape) for k, v in _read_file(full).items()})
+    return out
 
 
 def load_hf_state_dict(path: str, names: Optional[List[str]] = None) -> Dict[str, torch.Tensor]:

@@ -616,12 +616,13 @@ class ReaLModel(nn.Module):
             if 0 in self.layers:
                 x = x0 = self._embed(input_ids, meta.pos)
             pend = None  # a block's last branch output, added by the next norm kernel (plain pre-norm stacks)
+            n_pass = 0
             for li, (i, starts_pass) in enumerate(self.local_runs()):
-                if starts_pass and c.loop.inject:
-                    x = HB.loop_inject(self, i, HB.settle(self, x, pend), x0)
-                    pend = None
-                elif x is x0 and c.loop is not None:
+                if x is x0 and c.loop is not None and c.loop.inject_mode != "step":
                     x = x0.clone()  # the blocks update the stream in place; the loop reads the embedding output again
+                if starts_pass and c.loop.inject:
+                    x, pend = HB.start_pass(self, i, x, x0, pend, n_pass)
+                    n_pass += 1
                 x, pend = HB.block_packed(self, i, li, x, meta, pend, defer=trace is None)
                 if trace is not None:
                     trace.append(x.clone())
@@ -665,12 +666,12 @@ class ReaLModel(nn.Module):
     @torch.no_grad()
     def decode_step(self, input_ids: Optional[torch.Tensor], k_caches: List[torch.Tensor], v_caches: List[torch.Tensor],
                     cache_lens: torch.Tensor, hidden: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None,
-                    m_caches: Optional[List[Optional[torch.Tensor]]] = None) -> torch.Tensor:
+                    m_caches: Optional[list] = None) -> torch.Tensor:
         """input_ids [B] -> final hidden [B, H] (last stage: after ln_f).  Appends K/V at `cache_lens` in place.
         Caches: one [B, S, nkv_local, hd] tensor per local block.  Capturable in a CUDA graph (no host sync).
         Heterogeneous stacks: the caches are the per-block state tensors of `DecodeState` (see models/hetero_block.py) and
         `slots` [B] int32 names the state slot of every row (None: row b is slot b; `cache_lens` is indexed by slot); `m_caches`
-        is `DecodeState.m`, the third state tensor of the blocks that hold one."""
+        is `DecodeState.m`, what the blocks with more than two state tensors hold beside them."""
         c = self.config
         if c.blocks is not None:
             from realhf_b200.models import hetero_block as HB
@@ -678,12 +679,13 @@ class ReaLModel(nn.Module):
             if 0 in self.layers:
                 x = x0 = self._embed(input_ids, cache_lens, slots)   # a new token's position is its slot's length
             pend = None
+            n_pass = 0
             for li, (i, starts_pass) in enumerate(self.local_runs()):
-                if starts_pass and c.loop.inject:
-                    x = HB.loop_inject(self, i, HB.settle(self, x, pend), x0)
-                    pend = None
-                elif x is x0 and c.loop is not None:
+                if x is x0 and c.loop is not None and c.loop.inject_mode != "step":
                     x = x0.clone()
+                if starts_pass and c.loop.inject:
+                    x, pend = HB.start_pass(self, i, x, x0, pend, n_pass)
+                    n_pass += 1
                 x, pend = HB.block_decode(self, i, li, x, k_caches, v_caches, cache_lens, slots, pend, defer=True, m_caches=m_caches)
             if c.n_layers in self.layers:
                 return HB.final_norm(self, x, pend)

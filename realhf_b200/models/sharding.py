@@ -102,7 +102,8 @@ def wattn_sections(w) -> Tuple[int, ...]:
     """Rows of the fused input projection of a window-attention block: [queries | keys | values | output-gate logits].  The gate
     section (one row per head, or per output element) is padded so that it ends at a multiple of 8 rows counted from its own start
     (per head) or from the tensor's (per element): what follows it starts on a 16-byte boundary; the padding rows are never read."""
-    sec = (w.n_heads * w.n_maps * w.qk_dim, w.n_kv_heads * w.n_maps * w.qk_dim, w.n_kv_heads * w.v_dim)   # n_maps = 2: two score maps per head
+    sec = (w.n_heads * w.n_maps * w.qk_dim, w.n_kv_heads * w.n_maps * w.qk_dim)                # n_maps = 2: two score maps per head
+    sec += () if w.kv_shared else (w.value_width,)                                              # (shared: the values are the keys)
     if not w.out_gate:
         return sec
     return sec + ((_pad8(sum(sec) + w.gate_width) - sum(sec),) if w.element_gate else (_pad8(w.n_heads),))
@@ -139,10 +140,31 @@ def latent_rope_sections(a) -> Tuple[int, ...]:
 
 
 def delta_sections(d) -> Tuple[int, ...]:
-    """Rows of the fused input projection of a delta-rule block: [q | k | v | output gate | write strength, decay input].  The
-    convolution acts on the first three sections, which are therefore contiguous; the last section holds one row per head for
-    beta, then one per head for the decay, padded to a multiple of 8."""
-    return (d.n_kv_heads * d.qk_dim, d.n_kv_heads * d.qk_dim, d.n_heads * d.v_dim, d.n_heads * d.v_dim, _pad8(2 * d.n_heads))
+    """Rows of the fused input projection of a delta-rule block: [q | k | v | output gate | write strength, decay input | first factors
+    of the decay and of the gate].  The convolution acts on the first three sections, which are therefore contiguous.  The gate section
+    is absent with `gate_rank`, the decay inputs (one row per head, after one per head for the write strength; the section is padded
+    to a multiple of 8) with `decay_rank`; the last section holds decay_rank, then gate_rank rows (each padded to a multiple of 8)."""
+    nv = d.n_heads * d.v_dim
+    sec = (d.n_kv_heads * d.qk_dim, d.n_kv_heads * d.qk_dim, nv) + (() if d.gate_rank else (nv,))
+    sec += (_pad8(d.n_heads if d.decay_rank else 2 * d.n_heads),)
+    return sec + ((sum(delta_low_ranks(d)),) if d.low_rank_width else ())
+
+
+def delta_low_ranks(d) -> Tuple[int, int]:
+    """Padded inner ranks of the decay's and the gate's two-factor projections (0: one projection)."""
+    return _pad8(d.decay_rank or 0), _pad8(d.gate_rank or 0)
+
+
+def _delta_specs(add, d, H: int, o_name: str):
+    """Everything of a delta rule but its input projection.  `attn.low` holds the second factors, block-diagonal: [decay inputs | gate
+    logits] x [decay_rank | gate_rank], so that both are one product of the first factors' outputs."""
+    add("attn.conv.weight", (d.conv_channels, d.conv_taps), None)
+    add("attn.A_log.weight", (d.n_heads,), None, init="zeros")
+    add("attn.dt_bias.weight", (d.n_decays,), None, init="zeros")
+    if d.low_rank_width:
+        add("attn.low.weight", (d.low_rank_width, sum(delta_low_ranks(d))), None)
+    add("attn.o_norm.weight", (d.v_dim,), None, init="ones")
+    add(o_name, (H, d.n_heads * d.v_dim), None)
 
 
 def decay_sections(d) -> Tuple[int, ...]:
@@ -164,6 +186,8 @@ def _hetero_block_specs(cfg: ReaLModelConfig, layer_idx: int, P) -> List[ParamSp
         out.append(P(*args, **kw))
     if cfg.loop is not None and cfg.loop.inject and cfg.loop.inject_mode == "linear" and layer_idx == cfg.loop.start + 1:
         add("loop_in.weight", (H, 2 * H), None)
+    if cfg.loop is not None and cfg.loop.inject and cfg.loop.inject_mode == "step" and layer_idx == cfg.loop.start + 1:
+        add("loop_step.weight", (cfg.loop.times, H), None)
     norm_init = "zeros" if cfg.layer_norm_type == "gemma" else "ones"    # "gemma": the factor is 1 + weight
     NW = 1 if cfg.scalar_norm else H
     rg_mixer, rg_mlp = residual_gate_fused(cfg, layer_idx)
@@ -172,17 +196,25 @@ def _hetero_block_specs(cfg: ReaLModelConfig, layer_idx: int, P) -> List[ParamSp
         add("attn.canon.weight", (H, cfg.conv_taps), None)
     if b.mixer in ("decay", "parallel"):
         # one projection for everything that reads the mixer's input: [window attention q | k | v] (mixer "parallel" only), then the
-        # decayed linear attention's [q | k | v | gate]; each branch has its own output projection
-        d = b.decay
-        sec = (wattn_sections(b.wattn) if b.mixer == "parallel" else ()) + decay_sections(d)
+        # recurrent side's sections; each branch has its own output projection
+        d, w = b.decay, b.wattn
+        sec = (wattn_sections(w) if b.mixer == "parallel" else ()) + (decay_sections(d) if d is not None else delta_sections(b.delta))
         add("attn.in.weight", (sum(sec), H), None, sec)
-        if d.out_norm == "full":
+        if d is not None and d.out_norm == "full":
             add("attn.o_norm.weight", (d.n_heads * d.v_dim,), None, init="ones")
         if b.mixer == "parallel":
-            add("attn.o.weight", (H, b.wattn.n_heads * b.wattn.v_dim), None)
-            add("attn.o2.weight", (H, d.n_heads * d.v_dim), None)
+            if w.bias_rows:
+                add("attn.rel.weight", (w.bias_rows, w.n_heads), None, init="zeros")
+            if w.sink:
+                add("attn.sink.weight", (w.n_heads,), None, init="zeros")
+            add("attn.o.weight", (H, w.n_heads * w.v_dim), None)
+        if d is None:
+            _delta_specs(add, b.delta, H, "attn.o2.weight")
         else:
-            add("attn.o.weight", (H, d.n_heads * d.v_dim), None)
+            add("attn.o2.weight" if b.mixer == "parallel" else "attn.o.weight", (H, d.n_heads * d.v_dim), None)
+        if b.branch_norm:
+            add("attn.out_l.weight", (H,), None, init="ones")
+            add("attn.out_r.weight", (H,), None, init="ones")
     elif b.mixer == "window_attention":
         w = b.wattn
         sec = in_sections(cfg, layer_idx)
@@ -193,6 +225,8 @@ def _hetero_block_specs(cfg: ReaLModelConfig, layer_idx: int, P) -> List[ParamSp
             add("attn.temp.weight", (w.n_heads,), None, init="ones")
         if w.sink:
             add("attn.sink.weight", (w.n_heads,), None, init="zeros")
+        if w.bias_rows:
+            add("attn.rel.weight", (w.bias_rows, w.n_heads), None, init="zeros")
         if w.qk_norm:
             add("attn.q_norm.weight", (w.qk_dim * (w.n_heads if w.full_norm else 1),), None, init="ones")
             add("attn.k_norm.weight", (w.qk_dim * (w.n_kv_heads if w.full_norm else 1),), None, init="ones")
@@ -224,11 +258,7 @@ def _hetero_block_specs(cfg: ReaLModelConfig, layer_idx: int, P) -> List[ParamSp
         d = b.delta
         sec = delta_sections(d)
         add("attn.in.weight", (sum(sec), H), None, sec)
-        add("attn.conv.weight", (d.conv_channels, d.conv_taps), None)
-        add("attn.A_log.weight", (d.n_heads,), None, init="zeros")
-        add("attn.dt_bias.weight", (d.n_heads,), None, init="zeros")
-        add("attn.o_norm.weight", (d.v_dim,), None, init="ones")
-        add("attn.o.weight", (H, d.n_heads * d.v_dim), None)
+        _delta_specs(add, d, H, "attn.o.weight")
     else:
         own = a.kv_from is None
         q_sec = (a.n_heads * a.qk_dim,) + ((a.kv_rank,) if own else ())
@@ -247,7 +277,8 @@ def _hetero_block_specs(cfg: ReaLModelConfig, layer_idx: int, P) -> List[ParamSp
         add("attn.ls.weight", (H,), None, init="ones")
     if b.mlp is not None:
         F = b.mlp.ff
-        add("mlp.ln.weight", (NW,), None, init=norm_init)
+        if not cfg.parallel_ff:
+            add("mlp.ln.weight", (NW,), None, init=norm_init)
         if cfg.conv_taps:
             add("mlp.canon.weight", (H, cfg.conv_taps), None)
         if b.mlp.kind == "moe":

@@ -325,7 +325,8 @@ def latent_decode_attention(qc, w_ln, w_ukv, cache, cache_lens, slots, n_heads: 
 
 # ------------------------------------------------------------------------------------------------ window attention with a sink
 # (`WindowAttentionConfig`): grouped key / value heads; per-head temperature, linear distance penalty, soft cap, sliding window
-# that keeps the first tokens or chunks of positions, sink logit in the denominator, sigmoid output gate per head or element.
+# that keeps the first tokens or chunks of positions, learned distance bias, sink logit in the denominator, sigmoid output gate per
+# head or element.  A block whose values are its keys (`kv_shared`) has no v section and one cache (v_cache is k_cache).
 # Scores, weights and the value norm are fp32.  Rotations and query / key norms happen before (`window_prepare_`, `rotate_qk_`).
 # The projection output `qkvg` [T, ld] holds [q (H x d) | k (G x d) | v (G x dv) | gate logits (H or H x dv, padded)] per row.
 # Caches: k_cache [n_slots, G, rows, d], v_cache [n_slots, G, rows, dv]; position p of a sequence lives in row p when
@@ -346,9 +347,20 @@ def head_slopes(n_heads: int, slope_base: Optional[float], device) -> torch.Tens
     return torch.exp2(-slope_base * torch.arange(1, n_heads + 1, dtype=torch.float32, device=device) / n_heads)
 
 
+def distance_bias(rel, a):
+    """fp32 [n_heads, n] from the learned table `rel` [bias_rows, n_heads]: the bias of every distance (`a.distance_buckets`); distances
+    beyond the last column read it.  Cached on the weight; None without a bias."""
+    from realhf_b200.ops.functional import cached_on
+    if not a.bias_rows:
+        return None
+    return cached_on(rel, f"_bias_{a.bias_rows}_{float(a.bias_max)!r}",
+                     lambda w: w.float()[torch.tensor(a.distance_buckets(), device=w.device)].t().contiguous())
+
+
 def _wa_offsets(a):
-    nq, nk, nv = a.n_heads * a.qk_dim, a.n_kv_heads * a.qk_dim, a.n_kv_heads * a.v_dim
-    return nq, nq + nk, nq + nk + nv
+    """Column offsets of the key section, the value section and what follows it (shared: the key section is the value section)."""
+    nq, nk = a.n_heads * a.qk_dim, a.n_kv_heads * a.qk_dim
+    return nq, nq + nk, nq + nk + a.value_width
 
 
 def window_gate(qkvg, a):
@@ -358,9 +370,9 @@ def window_gate(qkvg, a):
 
 
 def window_values(qkvg, a):
-    """The value heads of a window-attention block's projection rows, [T, G * dv] (a view)."""
-    _, ok_, ov = _wa_offsets(a)
-    return qkvg[:, ok_:ov]
+    """The value heads of a window-attention block's projection rows, [T, G * dv] (a view; the keys when they are shared)."""
+    oq, ok_, ov = _wa_offsets(a)
+    return qkvg[:, oq:ok_] if a.kv_shared else qkvg[:, ok_:ov]
 
 
 def _sink_logits(a, sink, like):
@@ -388,27 +400,27 @@ def window_prepare_(qkvg, a, wq, wk, eps: float, pos=None, cache_lens=None, slot
     rot, vrot = a.rotary, a.value_rotary
     fq = rotary_table(rot, qkvg.device)[0] if rot is not None else None
     fv = rotary_table(vrot, qkvg.device)[0] if vrot is not None else None
-    if rot is not None and rotary_table(rot, qkvg.device)[1] != 1.0:
-        raise ValueError("window attention takes rotations without a factor on cos and sin")
+    ms = rotary_table(rot, qkvg.device)[1] if rot is not None else 1.0
     if not a.full_norm:
         wq = wk = None
     if use_native(qkvg) and d <= 1024 and dv <= 1024:
-        lib().window_prepare_(qkvg, wq, wk, fq, fv, pos, cache_lens if pos is None else None, slots if pos is None else None, k_cache, v_cache,
+        lib().window_prepare_(qkvg, wq, wk, fq, fv, pos, cache_lens if pos is None else None, slots if pos is None else None, k_cache,
+                              None if a.kv_shared else v_cache,
                               tok_slot if k_cache is not None else None, remain if k_cache is not None else None, H, G, d, dv,
                               rot.dims if rot else 0, bool(rot.interleaved) if rot else False, vrot.dims if vrot else 0,
-                              bool(vrot.interleaved) if vrot else False, a.keep_first, eps)
+                              bool(vrot.interleaved) if vrot else False, a.keep_first, eps, ms)
         return qkvg
     from realhf_b200.ops.recurrent import _rotate_heads_ref
     T = qkvg.shape[0]
     oq, ok_, ov = _wa_offsets(a)
     n = pos if pos is not None else cache_lens[slots.long() if slots is not None else torch.arange(T, device=qkvg.device)]
-    q, k, v = qkvg[:, :oq].float(), qkvg[:, oq:ok_].float(), qkvg[:, ok_:ov].float().reshape(T, G, dv)
+    q, k, v = qkvg[:, :oq].float(), qkvg[:, oq:ok_].float(), qkvg[:, ok_:ov].float().reshape(T, -1, dv)
     if wq is not None:
         q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps) * wq.float()
         k = k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps) * wk.float()
     q, k = q.reshape(T, H, d), k.reshape(T, G, d)
     if rot is not None:
-        q, k = _rotate_heads_ref(q, n, rot, fq), _rotate_heads_ref(k, n, rot, fq)
+        q, k = _rotate_heads_ref(q, n, rot, fq, ms), _rotate_heads_ref(k, n, rot, fq, ms)
     if vrot is not None:
         v = _rotate_heads_ref(v, n, vrot, fv)
     qkvg[:, :ov] = torch.cat([q.reshape(T, -1), k.reshape(T, -1), v.reshape(T, -1)], -1).to(qkvg.dtype)
@@ -447,7 +459,7 @@ def _apply_gate_ref(o, gate):
 def value_norm_store_ref(qkvg, a, eps, k_cache, v_cache, tok_slot, pos, remain):
     T = qkvg.shape[0]
     oq, ok_, ov = _wa_offsets(a)
-    v = qkvg[:, ok_:ov].float().view(T, a.n_kv_heads, a.v_dim)
+    v = window_values(qkvg, a).float().reshape(T, a.n_kv_heads, a.v_dim)
     if a.value_norm:
         v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)
     v = v.to(qkvg.dtype)
@@ -458,7 +470,8 @@ def value_norm_store_ref(qkvg, a, eps, k_cache, v_cache, tok_slot, pos, remain):
         r = cache_row(pos.long(), a.keep_first, rows)[keep]
         s = tok_slot[keep].long()
         k_cache[s, :, r] = qkvg[keep, oq:ok_].view(-1, a.n_kv_heads, a.qk_dim)
-        v_cache[s, :, r] = v[keep]
+        if not a.kv_shared:
+            v_cache[s, :, r] = v[keep]
     return v.reshape(T, a.n_kv_heads * a.v_dim)
 
 
@@ -482,7 +495,9 @@ def rotate_qk_(qkv, a, pos=None, cache_lens=None, slots=None):
     values are stored in the tensor's dtype).  Packed form: `pos` [T] int32; step form (`pos` None): row b's position is
     cache_lens[slots[b]] (slots None: cache_lens[b]).  Keys are therefore cached rotated."""
     rot = a.rotary
-    inv_freq = rotary_table(rot, qkv.device)[0]
+    inv_freq, ms = rotary_table(rot, qkv.device)
+    if ms != 1.0:
+        raise ValueError("this kernel takes rotations without a factor on cos and sin")
     n_h = a.n_heads + a.n_kv_heads
     if use_native(qkv):
         lib().rotate_heads_(qkv, pos, cache_lens if pos is None else None, slots if pos is None else None, inv_freq, n_h, a.qk_dim, rot.dims,
@@ -512,7 +527,7 @@ def _sink_softmax_pv(s, ok, sink_h, v):
     return (e / den) @ v
 
 
-def sink_window_attention_ref(qkvg, v_n, a, temp, sink, cu_seqlens):
+def sink_window_attention_ref(qkvg, v_n, a, temp, sink, cu_seqlens, rel=None):
     T = qkvg.shape[0]
     H, G, d, dv = a.n_heads, a.n_kv_heads, a.qk_dim, a.v_dim
     oq, ok_, ov = _wa_offsets(a)
@@ -520,7 +535,7 @@ def sink_window_attention_ref(qkvg, v_n, a, temp, sink, cu_seqlens):
     k = qkvg[:, oq:ok_].float().view(T, G, d)
     v = v_n.float().reshape(T, G, dv)
     sink = _sink_logits(a, sink, qkvg)
-    slopes = head_slopes(H, a.slope_base, qkvg.device)
+    slopes, bias = head_slopes(H, a.slope_base, qkvg.device), distance_bias(rel, a)
     out = torch.zeros(T, H, dv, dtype=torch.float32, device=qkvg.device)
     cu = cu_seqlens.tolist()
     for b in range(len(cu) - 1):
@@ -544,6 +559,8 @@ def sink_window_attention_ref(qkvg, v_n, a, temp, sink, cu_seqlens):
             if a.softcap is not None:
                 sc = a.softcap * torch.tanh(sc / a.softcap)
             sc = sc - slopes[h] * dist
+            if bias is not None:
+                sc = sc + bias[h][(i - j).clamp(0, bias.shape[1] - 1)]
             out[s0:e0, h] = _sink_softmax_pv(sc, ok, sink[h].float() if sink is not None else None, v[s0:e0, g])
     if a.value_rotary is None:                      # (else the output is turned back first: turn_gate_)
         out = _apply_gate_ref(out, window_gate(qkvg, a))
@@ -551,24 +568,31 @@ def sink_window_attention_ref(qkvg, v_n, a, temp, sink, cu_seqlens):
 
 
 def _sink_tc_ok(qkvg, v_n, a) -> bool:
-    """The tcgen05 form takes 16-bit operands with equal query / value head size of 64 or 128 (softmax statistics in fp32, the
-    weights rounded to the operand type for the P.V product); `REAL_WINDOW_ATTN=simt` selects the all-fp32 CUDA-core kernel."""
+    """The tcgen05 form takes 16-bit operands with query and value head sizes of 64 or 128 (softmax statistics in fp32, the weights
+    rounded to the operand type for the P.V product), different ones only without temperature, distance terms, cap and kept first keys;
+    a distance bias only with a table that fits the shared memory.  `REAL_WINDOW_ATTN=simt` selects the all-fp32 CUDA-core kernel."""
+    plain = a.slope_base is None and not (a.window is not None and a.keep_first)
+    if a.qk_dim != a.v_dim and not (plain and not a.head_temp and a.softcap is None and not a.bias_rows and a.scale > 0):
+        return False
+    if a.bias_rows and not (plain and min(len(a.distance_buckets()), a.window or 1 << 30) <= 8000):
+        return False
     return (os.environ.get("REAL_WINDOW_ATTN", "tcgen05") == "tcgen05" and qkvg.dtype in (torch.bfloat16, torch.float16)
-            and a.qk_dim == a.v_dim and a.qk_dim in (64, 128) and qkvg.stride(0) % 8 == 0 and qkvg.data_ptr() % 16 == 0
+            and a.qk_dim in (64, 128) and a.v_dim in (64, 128) and qkvg.stride(0) % 8 == 0 and qkvg.data_ptr() % 16 == 0
             and not (a.softcap is not None and (a.head_temp or a.keep_first or a.scale <= 0))
             and (a.n_heads * a.qk_dim) % 8 == 0 and v_n.data_ptr() % 16 == 0 and v_n.stride(0) % 8 == 0)
 
 
-def sink_window_attention(qkvg, v_n, a, temp, sink, pos, cu_seqlens, max_seqlen=None):
+def sink_window_attention(qkvg, v_n, a, temp, sink, pos, cu_seqlens, max_seqlen=None, rel=None):
     """Packed causal attention of a window-attention block over the batch's own keys (every sequence starts at position 0):
-    softmax_j(q_i . k_j * scale * temp_h - slope_h (i - j)) with the sink logit in the denominator (soft-capped with `a.softcap`), over
-    j <= i with i - j < window or j < keep_first (or of the same chunk); times the sigmoid gate.  With `a.value_rotary` the output
-    comes turned back by the query's position, before the gate.  Returns [T, H * dv] in the model dtype."""
-    out = _sink_window_attention(qkvg, v_n, a, temp, sink, pos, cu_seqlens, max_seqlen)
+    softmax_j(q_i . k_j * scale * temp_h - slope_h (i - j) + bias_h(i - j)) with the sink logit in the denominator (soft-capped with
+    `a.softcap`; `rel` the learned distance table), over j <= i with i - j < window or j < keep_first (or of the same chunk); times the
+    sigmoid gate.  With `a.value_rotary` the output comes turned back by the query's position, before the gate.  Returns [T, H * dv] in
+    the model dtype."""
+    out = _sink_window_attention(qkvg, v_n, a, temp, sink, pos, cu_seqlens, max_seqlen, rel)
     return turn_gate_(out, a, window_gate(qkvg, a), pos=pos) if a.value_rotary is not None else out
 
 
-def _sink_window_attention(qkvg, v_n, a, temp, sink, pos, cu_seqlens, max_seqlen):
+def _sink_window_attention(qkvg, v_n, a, temp, sink, pos, cu_seqlens, max_seqlen, rel):
     if use_native(qkvg) and a.qk_dim <= 512 and a.v_dim <= 256:     # (larger heads: the PyTorch form, on the device)
         T = qkvg.shape[0]
         out = torch.empty(T, a.n_heads * a.v_dim, dtype=qkvg.dtype, device=qkvg.device)
@@ -578,26 +602,28 @@ def _sink_window_attention(qkvg, v_n, a, temp, sink, pos, cu_seqlens, max_seqlen
         gate = window_gate(qkvg, a) if a.value_rotary is None else None
         shape = (a.scale, a.window if a.window is not None else -1, a.keep_first, a.slope_base if a.slope_base is not None else -1.0, gate,
                  a.element_gate, a.chunk or 0, a.softcap or 0.0)
+        bias = distance_bias(rel, a)
         if _sink_tc_ok(qkvg, v_n, a) and not (gate is not None and a.element_gate and gate.data_ptr() % 16):
-            lib().sink_window_attention_tc(qkvg, v_n, out, temp, sink, cu_seqlens, max_seqlen, a.n_heads, a.n_kv_heads, a.qk_dim, *shape)
+            lib().sink_window_attention_tc(qkvg, v_n, out, temp, sink, cu_seqlens, max_seqlen, a.n_heads, a.n_kv_heads, a.qk_dim, *shape,
+                                           v_dim=a.v_dim, bias=bias, kv_shared=a.kv_shared)
         else:
-            lib().sink_window_attention(qkvg, v_n, out, temp, sink, cu_seqlens, max_seqlen, a.n_heads, a.n_kv_heads, a.qk_dim, a.v_dim, *shape)
+            lib().sink_window_attention(qkvg, v_n, out, temp, sink, cu_seqlens, max_seqlen, a.n_heads, a.n_kv_heads, a.qk_dim, a.v_dim, *shape, bias=bias)
         return out
-    return sink_window_attention_ref(qkvg, v_n, a, temp, sink, cu_seqlens)
+    return sink_window_attention_ref(qkvg, v_n, a, temp, sink, cu_seqlens, rel)
 
 
-def sink_window_decode_attention_ref(qkvg, a, temp, sink, k_cache, v_cache, cache_lens, slots, eps):
+def sink_window_decode_attention_ref(qkvg, a, temp, sink, k_cache, v_cache, cache_lens, slots, eps, rel=None):
     B = qkvg.shape[0]
     H, G, d, dv = a.n_heads, a.n_kv_heads, a.qk_dim, a.v_dim
     oq, ok_, ov = _wa_offsets(a)
     rows = k_cache.shape[2]
     sink = _sink_logits(a, sink, qkvg)
-    slopes = head_slopes(H, a.slope_base, qkvg.device)
+    slopes, bias = head_slopes(H, a.slope_base, qkvg.device), distance_bias(rel, a)
     out = torch.zeros(B, H, dv, dtype=torch.float32, device=qkvg.device)
     for b in range(B):
         s = int(slots[b]) if slots is not None else b
         n = int(cache_lens[s])                                     # the new token's position
-        v_new = qkvg[b, ok_:ov].float().view(G, dv)
+        v_new = window_values(qkvg[b:b + 1], a)[0].float().view(G, dv)
         if a.value_norm:
             v_new = v_new * torch.rsqrt(v_new.pow(2).mean(-1, keepdim=True) + eps)
         r = cache_row(n, a.keep_first, rows)
@@ -616,13 +642,13 @@ def sink_window_decode_attention_ref(qkvg, a, temp, sink, k_cache, v_cache, cach
                 sc = sc * temp[h].float()
             if a.softcap is not None:
                 sc = a.softcap * torch.tanh(sc / a.softcap)
-            sc = (sc - slopes[h] * (n - j).float()).unsqueeze(0)
+            sc = (sc - slopes[h] * (n - j).float() + (bias[h][(n - j).clamp(max=bias.shape[1] - 1)] if bias is not None else 0.0)).unsqueeze(0)
             out[b, h] = _sink_softmax_pv(sc, torch.ones_like(sc, dtype=torch.bool), sink[h].float() if sink is not None else None, vv[g])[0]
     out = out.reshape(B, H * dv)
     return turn_gate_(out, a, window_gate(qkvg, a), cache_lens=cache_lens, slots=slots).to(qkvg.dtype)
 
 
-def sink_window_decode_attention(qkvg, a, temp, sink, k_cache, v_cache, cache_lens, slots, eps: float):
+def sink_window_decode_attention(qkvg, a, temp, sink, k_cache, v_cache, cache_lens, slots, eps: float, rel=None):
     """One new token per row against the caches of its slot (slots None: row b is slot b).  The row's key and normalised value
     are appended in place at the row of position cache_lens[slot] (cache_lens itself is not changed), then the token attends to
     every cached position its window and `keep_first` (or its chunk) allow, itself included; turning back and gate as in the packed
@@ -635,9 +661,10 @@ def sink_window_decode_attention(qkvg, a, temp, sink, k_cache, v_cache, cache_le
                                            a.qk_dim, a.v_dim, a.scale, a.window if a.window is not None else -1, a.keep_first,
                                            a.slope_base if a.slope_base is not None else -1.0, window_gate(qkvg, a), a.element_gate, a.chunk or 0,
                                            a.softcap or 0.0, rotary_table(vr, qkvg.device)[0] if vr is not None else None,
-                                           vr.dims if vr is not None else 0, bool(vr.interleaved) if vr is not None else False, bool(a.value_norm), eps)
+                                           vr.dims if vr is not None else 0, bool(vr.interleaved) if vr is not None else False, bool(a.value_norm), eps,
+                                           bias=distance_bias(rel, a), kv_shared=a.kv_shared)
         return out
-    return sink_window_decode_attention_ref(qkvg, a, temp, sink, k_cache, v_cache, cache_lens, slots, eps)
+    return sink_window_decode_attention_ref(qkvg, a, temp, sink, k_cache, v_cache, cache_lens, slots, eps, rel)
 
 
 # ------------------------------------------------------------------------------------------------ differential window attention

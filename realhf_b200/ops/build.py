@@ -40,7 +40,7 @@ NVCC_FLAGS = [
 ]
 # kernels that must keep IEEE division / exact expf (optimizer, the fp32-exact mechanisms of heterogeneous stacks) opt out of fast-math
 NO_FAST_MATH = {"adam.cu", "seqmix.cu", "latent_attn.cu", "posenc.cu", "sinkattn.cu", "delta.cu", "mlstm.cu", "latent_rope.cu", "moe_route.cu",
-                "centred_norm.cu", "decay.cu", "window_prepare.cu"}
+                "centred_norm.cu", "decay.cu", "window_prepare.cu", "branch_norm.cu"}
 
 
 def _cutlass_include() -> list[str]:

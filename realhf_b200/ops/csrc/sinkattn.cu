@@ -3,6 +3,7 @@
 //
 //   score(i, j) = q_i . k_j * scale * temp_h - slope_h * (i - j),   slope_h = 2^(-slope_base (h + 1) / H)
 //                 softcap > 0: softcap * tanh(q_i . k_j * scale * temp_h / softcap) instead
+//                 bias: + bias[h][min(i - j, n_bias - 1)], a learned number per head and distance (fp32 table)
 //   visible:      j <= i and (i - j < window or j < keep_first)                (window < 0: every j <= i)
 //                 chunk > 0: j <= i and floor(j / chunk) = floor(i / chunk) instead
 //   weights:      exp(score - m) / (sum_visible exp(score - m) + exp(sink_h - m))   (the sink is a bare logit: key-less, value-less)
@@ -12,6 +13,7 @@
 //
 // Everything is fp32 arithmetic whatever the storage type (a type code per launch: 0 fp32, 1 bf16, 2 fp16); exact expf (compiled
 // without fast-math).  The projection output `qkvg` [T, ld] holds [q (H x d) | k (G x d) | v (G x dv) | gate logits] per row.
+// A block whose values are its keys has no v section (kv_shared; d = dv) and one cache (vc = kc).
 // Caches: kc [n_slots, G, rows, d], vc [n_slots, G / vshare, rows, dv]; position p lives in row p when p < keep_first, else in row
 // keep_first + (p - keep_first) % (rows - keep_first).  `vshare` consecutive key heads read the same value head (1: a value head
 // per key head; 2: the two score maps of differential attention over one set of values), and the projection row then holds
@@ -47,6 +49,9 @@ RB_DEVICE float gate_factor(const void* g, int dt, int64_t row, int mode, int h,
   if (mode == 0) return 1.f;
   return 1.f / (1.f + expf(-ld_any(g, dt, row + (mode == 1 ? h : h * dv + col))));
 }
+
+// learned distance bias of head h (null: none)
+RB_DEVICE float dist_bias(const float* bias, int n_bias, int h, int dist) { return bias == nullptr ? 0.f : bias[(int64_t)h * n_bias + min(dist, n_bias - 1)]; }
 
 // a head's output turned back by position n: the pair of column c is (c, partner); o = the column's own value, po its partner's
 RB_DEVICE int turn_partner(int c, int dims, int interleaved) { return interleaved ? c ^ 1 : (c < dims / 2 ? c + dims / 2 : c - dims / 2); }
@@ -109,6 +114,7 @@ struct PrefillParams {
   int vshare, dto; int64_t vld;
   const void* gate; int64_t gld; int gmode;   // gate logits (type dt): row t at gate + t * gld; mode 0 none, 1 per head, 2 per element
   int chunk; float softcap;
+  const float* bias; int n_bias;   // [H, n_bias] or null
 };
 
 // NJ = ceil(dv / 32): a thread owns 2 query rows x NJ float4 column groups of the output tile
@@ -189,7 +195,7 @@ __global__ void __launch_bounds__(kPfThreads) sink_window_prefill_kernel(Prefill
         const bool vis = j < kend && j <= i && i <= q_last && j >= c_lo && (p.window < 0 || i - j < p.window || j < p.keep);
         float sc = s[r][c] * qmul;
         if (p.softcap > 0.f) sc = p.softcap * tanhf(sc / p.softcap);
-        s[r][c] = vis ? sc - slope * (float)(i - j) : -INFINITY;
+        s[r][c] = vis ? sc - slope * (float)(i - j) + dist_bias(p.bias, p.n_bias, h, i - j) : -INFINITY;
         mx = fmaxf(mx, s[r][c]);
       }
 #pragma unroll
@@ -323,6 +329,8 @@ struct DecodeParams {
   const void* gate; int64_t gld; int gmode;   // as in PrefillParams
   int chunk; float softcap;
   const float* turn_freq; int turn_dims, turn_inter;   // turn_dims > 0: the output is turned back by the position (frequencies [dims / 2])
+  const float* bias; int n_bias;   // [H, n_bias] or null
+  int kv_shared;                   // the values are the keys: no v section, vc = kc
 };
 
 __global__ void __launch_bounds__(kDecThreads) sink_window_decode_kernel(DecodeParams p) {
@@ -340,7 +348,7 @@ __global__ void __launch_bounds__(kDecThreads) sink_window_decode_kernel(DecodeP
   const int n = p.lens[slot];               // the new token's position
   const int64_t base = (int64_t)b * p.ld;
   const int gv = g / p.vshare, Gv = p.G / p.vshare;
-  const int ok = p.H * d, ov = ok + p.G * d;
+  const int ok = p.H * d, ov = p.kv_shared ? ok : ok + p.G * d;
   const int64_t cbase = ((int64_t)slot * p.G + g) * p.rows, vbase = ((int64_t)slot * Gv + gv) * p.rows;
 
   for (int idx = tid; idx < rep * d; idx += kDecThreads) {
@@ -407,7 +415,7 @@ __global__ void __launch_bounds__(kDecThreads) sink_window_decode_kernel(DecodeP
       if (r < rep) {
         const float slope = p.slope_base >= 0.f ? exp2f(-p.slope_base * (float)(h0 + r + 1) / (float)p.H) : 0.f;
         if (p.softcap > 0.f) s[r] = p.softcap * tanhf(s[r] / p.softcap);
-        s[r] = have ? s[r] - slope * (float)(n - j) : -INFINITY;
+        s[r] = have ? s[r] - slope * (float)(n - j) + dist_bias(p.bias, p.n_bias, h0 + r, n - j) : -INFINITY;
         const float wm = rb::warp_max(s[r]);
         if (lane == 0) red[r * 4 + warp] = wm;
       }
@@ -478,8 +486,9 @@ __global__ void __launch_bounds__(kDecThreads) sink_window_decode_kernel(DecodeP
 }
 
 // ------------------------------------------------------------------------------------------------ decode, 16-bit fast path
-// Equal query / value head size HD of 64 or 128, 16-bit storage: the streaming design of the dense-cache decode kernel
-// (attn_decode.cu).  A group of HD / 8 lanes owns one cache row at a time with 16-byte loads, REP query heads share every load,
+// Query / value head sizes HD and DV of 64 or 128, 16-bit storage: the streaming design of the dense-cache decode kernel
+// (attn_decode.cu).  A group of HD / 8 lanes owns one cache row at a time with 16-byte loads (its DV value columns in DV / (HD / 8) per
+// lane; kShared: the values are the keys just loaded, one cache is read), REP query heads share every load,
 // the loop is unrolled x4, the softmax exponentials use the fast intrinsic (fp32 arithmetic; the all-fp32 kernel above keeps expf),
 // launches are programmatic dependent launches like the dense kernel's, and the visible keys are cut into `splits` ranges (grid.z)
 // whose partial (max, sum, acc) are merged
@@ -487,29 +496,39 @@ __global__ void __launch_bounds__(kDecThreads) sink_window_decode_kernel(DecodeP
 // tokens, then the window); index -> cache row needs no division (the ring wraps at most once inside a window).
 constexpr int kFastWarps = 4, kFastThreads = kFastWarps * 32;
 
-template <typename T> RB_DEVICE void f_load8(const T* p, float* f) {
-  rb::Pack<T, 8> v = *reinterpret_cast<const rb::Pack<T, 8>*>(p);
+// N (4, 8 or 16) consecutive elements, at most 8 per access
+template <int N, typename T> RB_DEVICE void f_load(const T* p, float* f) {
+  constexpr int M = N < 8 ? N : 8;
 #pragma unroll
-  for (int i = 0; i < 8; ++i) f[i] = rb::to_f(v.v[i]);
+  for (int k = 0; k < N; k += M) {
+    const rb::Pack<T, M> v = *reinterpret_cast<const rb::Pack<T, M>*>(p + k);
+#pragma unroll
+    for (int i = 0; i < M; ++i) f[k + i] = rb::to_f(v.v[i]);
+  }
 }
-template <typename T> RB_DEVICE void f_store8(T* p, const float* f) {
-  rb::Pack<T, 8> v;
+template <int N, typename T> RB_DEVICE void f_store(T* p, const float* f) {
+  constexpr int M = N < 8 ? N : 8;
 #pragma unroll
-  for (int i = 0; i < 8; ++i) v.v[i] = rb::from_f<T>(f[i]);
-  *reinterpret_cast<rb::Pack<T, 8>*>(p) = v;
+  for (int k = 0; k < N; k += M) {
+    rb::Pack<T, M> v;
+#pragma unroll
+    for (int i = 0; i < M; ++i) v.v[i] = rb::from_f<T>(f[k + i]);
+    *reinterpret_cast<rb::Pack<T, M>*>(p + k) = v;
+  }
 }
 
 struct FastParams {
   DecodeParams d;
-  float* part_acc;   // [B, H, splits, HD]
+  float* part_acc;   // [B, H, splits, DV]
   float* part_ml;    // [B, H, splits, 2]
   int splits;
 };
 
-template <typename T, int HD, int REP>
+template <typename T, int HD, int DV, int REP, bool kShared>
 __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(FastParams fp) {
   const DecodeParams& p = fp.d;
-  constexpr int LPR = HD / 8, RPW = 32 / LPR;
+  constexpr int LPR = HD / 8, RPW = 32 / LPR, VPL = DV / LPR;   // lanes per row, rows per warp, value columns per lane
+  static_assert(!kShared || HD == DV, "shared keys and values have one size");
   const int b = blockIdx.x, g = blockIdx.y, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane % LPR, rsel = lane / LPR;
   rb::pdl_trigger();
@@ -518,31 +537,31 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
   const int n = p.lens[slot];
   const T* row_in = reinterpret_cast<const T*>(p.qkvg) + (int64_t)b * p.ld;
   const int Gv = p.G / p.vshare, gv = g / p.vshare;
-  const int ok = p.H * HD, ov = ok + p.G * HD;
+  const int ok = p.H * HD, ov = kShared ? ok : ok + p.G * HD;
   T* kc = reinterpret_cast<T*>(p.kc) + ((int64_t)slot * p.G + g) * p.rows * HD;
-  T* vc = reinterpret_cast<T*>(p.vc) + ((int64_t)slot * Gv + gv) * p.rows * HD;   // (CTAs that share a value head append the same values)
+  T* vc = reinterpret_cast<T*>(p.vc) + ((int64_t)slot * Gv + gv) * p.rows * DV;   // (CTAs that share a value head append the same values)
 
-  float q[REP][8], slope[REP], kn[8], vn[8];
+  float q[REP][8], slope[REP], kn[8], vn[VPL];
 #pragma unroll
   for (int r = 0; r < REP; ++r) {
     const int h = g * REP + r;
-    f_load8(row_in + h * HD + sub * 8, q[r]);
+    f_load<8>(row_in + h * HD + sub * 8, q[r]);
     const float mul = p.scale * (p.temp ? rb::to_f(reinterpret_cast<const T*>(p.temp)[h]) : 1.f);
 #pragma unroll
     for (int i = 0; i < 8; ++i) q[r][i] *= mul;
     slope[r] = p.slope_base >= 0.f ? exp2f(-p.slope_base * (float)(h + 1) / (float)p.H) : 0.f;
   }
-  f_load8(row_in + ok + g * HD + sub * 8, kn);
-  f_load8(row_in + ov + gv * HD + sub * 8, vn);
+  f_load<8>(row_in + ok + g * HD + sub * 8, kn);
+  f_load<VPL>(row_in + ov + gv * DV + sub * VPL, vn);
   if (p.do_norm) {
     float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) ss = fmaf(vn[i], vn[i], ss);
+    for (int i = 0; i < VPL; ++i) ss = fmaf(vn[i], vn[i], ss);
 #pragma unroll
     for (int o = LPR / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o, LPR);
-    const float rs = 1.f / sqrtf(ss / (float)HD + p.eps);
+    const float rs = 1.f / sqrtf(ss / (float)DV + p.eps);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) vn[i] = rb::to_f(rb::from_f<T>(vn[i] * rs));     // as later steps will read it from the cache
+    for (int i = 0; i < VPL; ++i) vn[i] = rb::to_f(rb::from_f<T>(vn[i] * rs));     // as later steps will read it from the cache
   }
   const int ring = max(p.rows - p.keep, 1);
   const int lo = first_visible(n, p.window, p.chunk);
@@ -560,25 +579,25 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
   const int nk = ka + (n - lo + 1);                    // the last index is the new token itself
   if (split == 0 && warp == 0 && rsel == 0) {
     const int64_t rn = row_of(nk - 1);
-    f_store8(kc + rn * HD + sub * 8, kn);
-    f_store8(vc + rn * HD + sub * 8, vn);
+    f_store<8>(kc + rn * HD + sub * 8, kn);
+    if constexpr (!kShared) f_store<VPL>(vc + rn * DV + sub * VPL, vn);
   }
   const int cached = nk - 1;
   const int per = RB_CEIL_DIV(cached, fp.splits);
   const int i0 = min(cached, split * per), i1 = min(cached, i0 + per);
 
-  float m[REP], l[REP], acc[REP][8];
+  float m[REP], l[REP], acc[REP][VPL];
 #pragma unroll
   for (int r = 0; r < REP; ++r) {
     m[r] = -INFINITY; l[r] = 0.f;
     if (p.sink && split == 0 && warp == 0 && rsel == 0) { m[r] = rb::to_f(reinterpret_cast<const T*>(p.sink)[g * REP + r]); l[r] = 1.f; }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) acc[r][i] = 0.f;
+    for (int i = 0; i < VPL; ++i) acc[r][i] = 0.f;
   }
   const float cap2 = p.softcap > 0.f ? 2.f / p.softcap : 0.f;
   const unsigned gmask = (LPR == 32) ? 0xffffffffu : (((1u << LPR) - 1u) << (rsel * LPR));
   auto consume = [&](const float* kf, const float* vf, int idx) {
-    const float dist = (float)(n - pos_of(idx));
+    const int dist = n - pos_of(idx);
 #pragma unroll
     for (int r = 0; r < REP; ++r) {
       float s = 0.f;
@@ -587,35 +606,35 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
 #pragma unroll
       for (int o = LPR / 2; o > 0; o >>= 1) s += __shfl_xor_sync(gmask, s, o, LPR);
       if (p.softcap > 0.f) s = p.softcap - __fdividef(2.f * p.softcap, 1.f + __expf(fminf(s * cap2, 80.f)));   // cap tanh(s / cap)
-      s -= slope[r] * dist;
+      s += dist_bias(p.bias, p.n_bias, g * REP + r, dist) - slope[r] * (float)dist;
       const float mn = fmaxf(m[r], s);
       const float corr = (m[r] == -INFINITY) ? 0.f : __expf(m[r] - mn), pr = __expf(s - mn);
       l[r] = l[r] * corr + pr;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) acc[r][i] = fmaf(acc[r][i], corr, pr * vf[i]);
+      for (int i = 0; i < VPL; ++i) acc[r][i] = fmaf(acc[r][i], corr, pr * vf[i]);
       m[r] = mn;
     }
   };
-  constexpr int UNROLL = 4;
+  constexpr int UNROLL = REP * VPL >= 96 ? 2 : 4;      // (register budget)
   const int step = kFastWarps * RPW;
   int s0 = i0 + warp * RPW + rsel;
   for (; s0 + (UNROLL - 1) * step < i1; s0 += UNROLL * step) {
-    float kf[UNROLL][8], vf[UNROLL][8];
+    float kf[UNROLL][8], vf[UNROLL][kShared ? 1 : VPL];
 #pragma unroll
     for (int u = 0; u < UNROLL; ++u) {
       const int64_t rr = row_of(s0 + u * step);
-      f_load8(kc + rr * HD + sub * 8, kf[u]);
-      f_load8(vc + rr * HD + sub * 8, vf[u]);
+      f_load<8>(kc + rr * HD + sub * 8, kf[u]);
+      if constexpr (!kShared) f_load<VPL>(vc + rr * DV + sub * VPL, vf[u]);
     }
 #pragma unroll
-    for (int u = 0; u < UNROLL; ++u) consume(kf[u], vf[u], s0 + u * step);
+    for (int u = 0; u < UNROLL; ++u) consume(kf[u], kShared ? kf[u] : vf[u], s0 + u * step);
   }
   for (; s0 < i1; s0 += step) {
-    float kf[8], vf[8];
+    float kf[8], vf[kShared ? 1 : VPL];
     const int64_t rr = row_of(s0);
-    f_load8(kc + rr * HD + sub * 8, kf);
-    f_load8(vc + rr * HD + sub * 8, vf);
-    consume(kf, vf, s0);
+    f_load<8>(kc + rr * HD + sub * 8, kf);
+    if constexpr (!kShared) f_load<VPL>(vc + rr * DV + sub * VPL, vf);
+    consume(kf, kShared ? kf : vf, s0);
   }
   if (split == fp.splits - 1 && warp == 0 && rsel == 0) {
 #pragma unroll
@@ -623,7 +642,7 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
     consume(kn, vn, nk - 1);
   }
   __syncwarp();
-  __shared__ float sm_acc[kFastWarps][REP][HD];
+  __shared__ float sm_acc[kFastWarps][REP][DV];
   __shared__ float sm_m[kFastWarps][REP], sm_l[kFastWarps][REP];
 #pragma unroll
   for (int r = 0; r < REP; ++r) {
@@ -634,7 +653,7 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
       const float c1 = (m[r] == -INFINITY) ? 0.f : __expf(m[r] - mn), c2 = (m2 == -INFINITY) ? 0.f : __expf(m2 - mn);
       l[r] = l[r] * c1 + l2 * c2;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < VPL; ++i) {
         const float a2 = __shfl_xor_sync(0xffffffffu, acc[r][i], o);
         acc[r][i] = acc[r][i] * c1 + a2 * c2;
       }
@@ -642,13 +661,13 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
     }
     if (rsel == 0) {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) sm_acc[warp][r][sub * 8 + i] = acc[r][i];
+      for (int i = 0; i < VPL; ++i) sm_acc[warp][r][sub * VPL + i] = acc[r][i];
       if (sub == 0) { sm_m[warp][r] = m[r]; sm_l[warp][r] = l[r]; }
     }
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < REP * HD; idx += kFastThreads) {
-    const int r = idx / HD, c = idx % HD;
+  for (int idx = threadIdx.x; idx < REP * DV; idx += kFastThreads) {
+    const int r = idx / DV, c = idx % DV;
     float mg = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kFastWarps; ++w) mg = fmaxf(mg, sm_m[w][r]);
@@ -665,20 +684,20 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
     const int h = g * REP + r;
     if (fp.splits == 1) {
       if (turn) ag = turn_back(ag, pg, c, (float)n, p.turn_freq, p.turn_dims, p.turn_inter);
-      const float f = (lg > 0.f ? 1.f / lg : 0.f) * gate_factor(p.gate, p.dt, (int64_t)b * p.gld, p.gmode, h, HD, c);
-      reinterpret_cast<T*>(p.out)[(int64_t)b * p.H * HD + (int64_t)h * HD + c] = rb::from_f<T>(ag * f);
+      const float f = (lg > 0.f ? 1.f / lg : 0.f) * gate_factor(p.gate, p.dt, (int64_t)b * p.gld, p.gmode, h, DV, c);
+      reinterpret_cast<T*>(p.out)[(int64_t)b * p.H * DV + (int64_t)h * DV + c] = rb::from_f<T>(ag * f);
     } else {
       const int64_t o = ((int64_t)b * p.H + h) * fp.splits + split;
-      fp.part_acc[o * HD + c] = ag;
+      fp.part_acc[o * DV + c] = ag;
       if (c == 0) { fp.part_ml[o * 2] = mg; fp.part_ml[o * 2 + 1] = lg; }
     }
   }
 }
 
-template <typename T, int HD>
+template <typename T, int DV>
 __global__ void sink_window_decode_merge_kernel(FastParams fp) {
   const DecodeParams& p = fp.d;
-  __shared__ float so[HD];
+  __shared__ float so[DV];
   const int64_t bh = blockIdx.x;
   const int c = threadIdx.x, splits = fp.splits, b = (int)(bh / p.H), h = (int)(bh % p.H);
   rb::pdl_trigger();
@@ -690,7 +709,7 @@ __global__ void sink_window_decode_merge_kernel(FastParams fp) {
     const float ms = fp.part_ml[(bh * splits + s) * 2];
     const float cf = (ms == -INFINITY) ? 0.f : expf(ms - mg);
     lg += fp.part_ml[(bh * splits + s) * 2 + 1] * cf;
-    ag += fp.part_acc[(bh * splits + s) * HD + c] * cf;
+    ag += fp.part_acc[(bh * splits + s) * DV + c] * cf;
   }
   if (p.turn_dims > 0) {
     so[c] = ag;
@@ -698,15 +717,15 @@ __global__ void sink_window_decode_merge_kernel(FastParams fp) {
     if (c < p.turn_dims)
       ag = turn_back(ag, so[turn_partner(c, p.turn_dims, p.turn_inter)], c, (float)p.lens[p.slots ? p.slots[b] : b], p.turn_freq, p.turn_dims, p.turn_inter);
   }
-  const float f = (lg > 0.f ? 1.f / lg : 0.f) * gate_factor(p.gate, p.dt, (int64_t)b * p.gld, p.gmode, h, HD, c);
-  reinterpret_cast<T*>(p.out)[bh * HD + c] = rb::from_f<T>(ag * f);
+  const float f = (lg > 0.f ? 1.f / lg : 0.f) * gate_factor(p.gate, p.dt, (int64_t)b * p.gld, p.gmode, h, DV, c);
+  reinterpret_cast<T*>(p.out)[bh * DV + c] = rb::from_f<T>(ag * f);
 }
 
-template <typename T, int HD>
+template <typename T, int HD, int DV, bool kShared>
 int launch_fast(const FastParams& fp, int B, cudaStream_t s) {
   const DecodeParams& p = fp.d;
   dim3 grid(B, p.G, fp.splits);
-#define RB_L(REP) rb::launch_pdl(sink_window_decode_fast_kernel<T, HD, REP>, grid, dim3(kFastThreads), 0, s, fp)
+#define RB_L(REP) rb::launch_pdl(sink_window_decode_fast_kernel<T, HD, DV, REP, kShared>, grid, dim3(kFastThreads), 0, s, fp)
   switch (p.H / p.G) {
     case 1: RB_L(1); break;
     case 2: RB_L(2); break;
@@ -717,8 +736,16 @@ int launch_fast(const FastParams& fp, int B, cudaStream_t s) {
     default: return -1;
   }
 #undef RB_L
-  if (fp.splits > 1) rb::launch_pdl(sink_window_decode_merge_kernel<T, HD>, dim3(B * p.H), dim3(HD), 0, s, fp);
+  if (fp.splits > 1) rb::launch_pdl(sink_window_decode_merge_kernel<T, DV>, dim3(B * p.H), dim3(DV), 0, s, fp);
   return 0;
+}
+
+template <typename T>
+int launch_fast_sizes(const FastParams& fp, int B, cudaStream_t s) {
+  const int d = fp.d.d, dv = fp.d.dv;
+  if (fp.d.kv_shared) return d != dv ? -1 : d == 128 ? launch_fast<T, 128, 128, true>(fp, B, s) : launch_fast<T, 64, 64, true>(fp, B, s);
+  if (d == 128) return dv == 128 ? launch_fast<T, 128, 128, false>(fp, B, s) : launch_fast<T, 128, 64, false>(fp, B, s);
+  return dv == 128 ? launch_fast<T, 64, 128, false>(fp, B, s) : launch_fast<T, 64, 64, false>(fp, B, s);
 }
 
 }  // namespace
@@ -735,10 +762,11 @@ extern "C" int rb_value_norm_store(const void* qkvg, int64_t ld, int dt, void* v
 extern "C" int rb_sink_window_prefill(const void* qkvg, int64_t ld, const void* vn, void* out, const void* temp, const void* sink, const int* cu,
                                       int n_seqs, int max_seqlen, int H, int G, int d, int dv, float scale, int window, int keep, float slope_base,
                                       const void* gate, int64_t gld, int gmode, int chunk, float softcap, int dt, int vshare, int64_t vld, int dto,
-                                      cudaStream_t s) {
+                                      const float* bias, int n_bias, cudaStream_t s) {
   if (n_seqs == 0 || max_seqlen == 0) return 0;
+  if (bias != nullptr && n_bias < 1) return -1;
   if (dv > 256 || d > 512 || H % G || vshare < 1 || G % vshare || (gmode != 0 && gate == nullptr)) return -1;
-  PrefillParams p{qkvg, ld, vn, out, temp, sink, cu, H, G, d, dv, window, keep, dt, scale, slope_base, vshare, dto, vld, gate, gld, gmode, chunk, softcap};
+  PrefillParams p{qkvg, ld, vn, out, temp, sink, cu, H, G, d, dv, window, keep, dt, scale, slope_base, vshare, dto, vld, gate, gld, gmode, chunk, softcap, bias, n_bias};
   const int nj = dv <= 32 ? 1 : dv <= 64 ? 2 : dv <= 128 ? 4 : 8;
   const int dp = (d + 3) & ~3;
   const size_t smem = sizeof(float) * ((size_t)(BQ + BK) * (dp + 4) + (size_t)BK * (nj * 32 + 4) + (size_t)BQ * (BK + 1));
@@ -762,13 +790,14 @@ extern "C" int rb_sink_window_decode(const void* qkvg, int64_t ld, void* out, co
                                      const int* lens, const int* slots, int B, int H, int G, int d, int dv, int rows, float scale, int window,
                                      int keep, float slope_base, const void* gate, int64_t gld, int gmode, int chunk, float softcap,
                                      const float* turn_freq, int turn_dims, int turn_inter, int do_norm, float eps, int dt, int vshare, int dto,
-                                     cudaStream_t s) {
+                                     const float* bias, int n_bias, int kv_shared, cudaStream_t s) {
   if (B == 0) return 0;
   const int rep = min(H / G, kMaxRep);
   if (H % G || dv > kDecThreads * kMaxColsPerThread || vshare < 1 || G % vshare || (gmode != 0 && gate == nullptr)) return -1;
   if (turn_dims % 2 || turn_dims > dv || (turn_dims > 0 && turn_freq == nullptr)) return -1;
+  if ((bias != nullptr && n_bias < 1) || (kv_shared && (d != dv || kc != vc || vshare != 1 || do_norm))) return -1;
   DecodeParams p{qkvg, ld, out, temp, sink, kc, vc, lens, slots, H, G, d, dv, rows, window, keep, do_norm, dt, scale, slope_base, eps, vshare, dto,
-                 gate, gld, gmode, chunk, softcap, turn_freq, turn_dims, turn_inter};
+                 gate, gld, gmode, chunk, softcap, turn_freq, turn_dims, turn_inter, bias, n_bias, kv_shared};
   size_t smem = sizeof(float) * ((size_t)rep * d + (size_t)rep * kDecThreads + rep * 5 + 32 + dv + kDecThreads);
   if (turn_dims > 0 && smem < sizeof(float) * (size_t)rep * dv) smem = sizeof(float) * (size_t)rep * dv;
   if (smem > 48 * 1024) cudaFuncSetAttribute(sink_window_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -776,22 +805,23 @@ extern "C" int rb_sink_window_decode(const void* qkvg, int64_t ld, void* out, co
   return 0;
 }
 
-// 16-bit fast path of the decode form (dt 1 / 2, d == dv in {64, 128}, H / G in {1, 2, 3, 4, 6, 8}, 16-byte aligned rows); part_acc
-// [B, H, splits, d] and part_ml [B, H, splits, 2] fp32 are scratch for splits > 1.  Returns -1 for shapes it does not take.
+// 16-bit fast path of the decode form (dt 1 / 2, d and dv in {64, 128}, H / G in {1, 2, 3, 4, 6, 8}, 16-byte aligned rows); part_acc
+// [B, H, splits, dv] and part_ml [B, H, splits, 2] fp32 are scratch for splits > 1.  Returns -1 for shapes it does not take.
 extern "C" int rb_sink_window_decode_fast(const void* qkvg, int64_t ld, void* out, const void* temp, const void* sink, void* kc, void* vc,
                                           const int* lens, const int* slots, float* part_acc, float* part_ml, int splits, int B, int H, int G, int d,
-                                          int rows, float scale, int window, int keep, float slope_base, const void* gate, int64_t gld, int gmode,
+                                          int dv, int rows, float scale, int window, int keep, float slope_base, const void* gate, int64_t gld, int gmode,
                                           int chunk, float softcap, const float* turn_freq, int turn_dims, int turn_inter, int do_norm, float eps,
-                                          int dt, int vshare, cudaStream_t s) {
+                                          int dt, int vshare, const float* bias, int n_bias, int kv_shared, cudaStream_t s) {
   if (B == 0) return 0;
-  if ((dt != 1 && dt != 2) || (d != 64 && d != 128) || H % G || vshare < 1 || G % vshare || ld % 8 || ((uintptr_t)qkvg & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15))
+  if ((dt != 1 && dt != 2) || (d != 64 && d != 128) || (dv != 64 && dv != 128) || H % G || vshare < 1 || G % vshare || ld % 8 || ((uintptr_t)qkvg & 15) ||
+      ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15))
     return -1;
-  if ((gmode != 0 && gate == nullptr) || turn_dims % 2 || turn_dims > d || (turn_dims > 0 && turn_freq == nullptr)) return -1;
-  FastParams fp{DecodeParams{qkvg, ld, out, temp, sink, kc, vc, lens, slots, H, G, d, d, rows, window, keep, do_norm, dt, scale, slope_base, eps, vshare, dt,
-                             gate, gld, gmode, chunk, softcap, turn_freq, turn_dims, turn_inter},
+  if ((gmode != 0 && gate == nullptr) || turn_dims % 2 || turn_dims > dv || (turn_dims > 0 && turn_freq == nullptr)) return -1;
+  if ((bias != nullptr && n_bias < 1) || (kv_shared && (kc != vc || vshare != 1 || do_norm))) return -1;
+  FastParams fp{DecodeParams{qkvg, ld, out, temp, sink, kc, vc, lens, slots, H, G, d, dv, rows, window, keep, do_norm, dt, scale, slope_base, eps, vshare, dt,
+                             gate, gld, gmode, chunk, softcap, turn_freq, turn_dims, turn_inter, bias, n_bias, kv_shared},
                 part_acc, part_ml, splits};
-  if (dt == 1) return d == 128 ? launch_fast<__nv_bfloat16, 128>(fp, B, s) : launch_fast<__nv_bfloat16, 64>(fp, B, s);
-  return d == 128 ? launch_fast<__half, 128>(fp, B, s) : launch_fast<__half, 64>(fp, B, s);
+  return dt == 1 ? launch_fast_sizes<__nv_bfloat16>(fp, B, s) : launch_fast_sizes<__half>(fp, B, s);
 }
 
 extern "C" int rb_qk_head_norm(void* x, int64_t ld, int dt, const void* wq, const void* wk, int64_t T, int nq, int nk, int d, float eps,

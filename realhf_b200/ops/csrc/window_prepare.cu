@@ -5,8 +5,9 @@
 //   window_prepare   row [q (H d) | k (G d) | v (G dv) | ..] in place: q and k divided by their root mean square over ALL their heads
 //                    and multiplied by a weight each (wq, wk; null: no norm), the first `dims` dimensions of every q / k head and
 //                    the first `vdims` of every v head turned by the position (vdims 0: values untouched).  Packed form: position
-//                    pos[t]; with caches the k and v of the tokens a later decode step can still see (the first `keep` positions and
-//                    the last rows - keep of the sequence) also go to their cache row.  Step form: position lens[slot of row t]; the
+//                    pos[t]; cos and sin of q and k carry a factor (`mscale`); with caches the k and v of the tokens a later decode step can still see (the first `keep` positions and
+//                    the last rows - keep of the sequence) also go to their cache row (a row without a v section, whose values are its
+//                    keys, has one cache).  Step form: position lens[slot of row t]; the
 //                    decode kernel stores the row.
 //   turn_gate        attention output [T, H dv] in place: every head turned BACK by the position over its first `dims` columns (the
 //                    inverse of the values' rotation), then times sigmoid of a gate logit per head or per element.
@@ -42,8 +43,13 @@ RB_DEVICE int row_position(const int* pos, const int* lens, const int* slots, in
   return lens[slots != nullptr ? slots[t] : t];
 }
 
-RB_DEVICE void fill_table(float* cs, float* sn, float p, const float* freq, int half) {
-  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(p * freq[i], &sn[i], &cs[i]);
+RB_DEVICE void fill_table(float* cs, float* sn, float p, const float* freq, int half, float mscale = 1.f) {
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(p * freq[i], &s, &c);
+    sn[i] = s * mscale;
+    cs[i] = c * mscale;
+  }
 }
 
 // Walks the n_h heads of size hd: f(element offset inside the section, values, n values) after `pre` scaled the loaded elements and the
@@ -104,7 +110,7 @@ struct PrepareParams {
   const int* tok_slot; const int* remain;
   void* kc; void* vc;
   int H, G, d, dv, dims, inter, vdims, vinter, keep, rows;
-  float eps;
+  float eps, mscale;
 };
 
 template <int V>
@@ -116,7 +122,7 @@ __global__ void __launch_bounds__(kThreads) window_prepare_kernel(PrepareParams 
   rb::pdl_trigger();
   rb::pdl_wait();
   const int n = row_position(p.pos, p.lens, p.slots, t);
-  fill_table(cs, sn, (float)n, p.freq, p.dims / 2);
+  fill_table(cs, sn, (float)n, p.freq, p.dims / 2, p.mscale);
   fill_table(vcs, vsn, (float)n, p.vfreq, p.vdims / 2);
   int64_t slot = -1;
   int row = 0;
@@ -209,11 +215,11 @@ inline bool rot_vec(int dims, int inter) { return (inter ? dims : dims / 2) % 4 
 
 extern "C" int rb_window_prepare(void* x, int64_t ld, int dt, const void* wq, const void* wk, const float* freq, const float* vfreq, const int* pos,
                                  const int* lens, const int* slots, const int* tok_slot, const int* remain, void* kc, void* vc, int64_t T, int H,
-                                 int G, int d, int dv, int dims, int inter, int vdims, int vinter, int keep, int rows, float eps, cudaStream_t s) {
+                                 int G, int d, int dv, int dims, int inter, int vdims, int vinter, int keep, int rows, float eps, float mscale, cudaStream_t s) {
   if (T == 0) return 0;
   if (dims % 2 || dims > d || vdims % 2 || vdims > dv || dims / 2 > kMaxHalf || vdims / 2 > kMaxHalf || (pos == nullptr && lens == nullptr)) return -1;
-  if ((wq == nullptr) != (wk == nullptr) || (kc == nullptr) != (vc == nullptr)) return -1;
-  PrepareParams p{x, ld, dt, wq, wk, freq, vfreq, pos, lens, slots, tok_slot, remain, kc, vc, H, G, d, dv, dims, inter, vdims, vinter, keep, rows, eps};
+  if ((wq == nullptr) != (wk == nullptr) || (kc == nullptr && vc != nullptr)) return -1;
+  PrepareParams p{x, ld, dt, wq, wk, freq, vfreq, pos, lens, slots, tok_slot, remain, kc, vc, H, G, d, dv, dims, inter, vdims, vinter, keep, rows, eps, mscale};
   const bool vec = d % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && rot_vec(dims, inter) && rot_vec(vdims, vinter) && al16(x) && al16(kc) && al16(vc);
   return rb::launch_pdl(vec ? window_prepare_kernel<4> : window_prepare_kernel<1>, dim3((unsigned)T), dim3(kThreads), 0, s, p) == cudaSuccess ? 0 : 2;
 }

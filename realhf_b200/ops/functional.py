@@ -737,6 +737,25 @@ def residual_add_centred_norm_(x, y, w, eps: float, scale=None, mult: float = 1.
     return norm(x, next_w).to(out_dtype) if next_w is not None else None
 
 
+def branch_add_norm_(x, y=None, y2=None, ff=None, eps: float = 0.0, a: float = 1.0, b: float = 1.0, w1=None, w2=None, step=None, next_w=None,
+                     w_offset: float = 0.0, out_dtype=None):
+    """x += (a N1(y) + b N2(y2)) + ff + step in place (fp32 sum, stored in x's dtype): y, y2, ff [T, W] of one dtype or None, N1 / N2 RMS
+    norms with the weights w1 / w2 or nothing, `step` a vector [W] or None.  With `next_w`, also returns RMSNorm(x) * (next_w + w_offset)
+    of the updated rows in out_dtype, from the same kernel."""
+    if use_native(x) and x.is_contiguous():
+        out = torch.empty(x.shape, dtype=out_dtype, device=x.device) if next_w is not None else None
+        lib().branch_norm_(x, y, y2, ff, a, b, w1, w2, step, next_w, w_offset, out, eps)
+        return out
+    t = None
+    for v, w, m in ((y, w1, a), (y2, w2, b), (ff, None, 1.0)):
+        if v is not None:
+            n = m * (group_rmsnorm_ref(v, w, 1, eps) if w is not None else v.float())
+            t = n if t is None else t + n
+    xf = x.float() if t is None else x.float() + t
+    x.copy_((xf if step is None else xf + step.float()).to(x.dtype))
+    return group_rmsnorm_ref(x, next_w, 1, eps, w_offset).to(out_dtype) if next_w is not None else None
+
+
 def clamped_glu_ref(gu, limit: float, alpha: float):
     F_ = gu.shape[-1] // 2
     g = gu[..., :F_].float().clamp(max=limit)

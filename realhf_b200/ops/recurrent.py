@@ -3,19 +3,23 @@ matrix-memory LSTM (`MLSTMConfig`) and linear attention with a fixed decay per h
 block further down.
 
 Per head, with a matrix state S [d, dv] in fp32:   S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
-(the output is read after the update, so it contains what this token just wrote).  Everything that enters the recurrence is fp32.
+(the output is read after the update, so it contains what this token just wrote; g is one number per head, or with `decay_rank` one
+per row of S).  Everything that enters the recurrence is fp32.
 
 The stages, each = PyTorch reference (CPU tensors, also the numerics oracle of the kernel tests) + sm_100a kernel (`csrc/delta.cu`):
 
+  delta_low              with `decay_rank` / `gate_rank`: the second factors of the decay and of the gate applied to the first ones'
+                         outputs (a section of `proj`), one product: [T, decay inputs (H d) | gate logits (H dv)].
   delta_prepare(_step)   the fused projection output `proj` [T, ld] = [q (G x d) | k (G x d) | v (H x dv) | gate (H x dv) | beta
-                         logits (H) | decay inputs (H) | padding] -> fp32 `u` [T, C + 2H] = [q | k | v | beta | g]:  causal depthwise
-                         convolution + SiLU over the first C = 2 G d + H dv channels (inputs before a sequence's first token are zero; the packed
-                         form leaves the last taps - 1 raw inputs of every sequence in `conv_state` [n_slots, taps - 1, C] fp32,
-                         oldest first; the step form reads and shifts it), q and k scaled to unit length per head (q also by
-                         d^-1/2), beta = sigmoid, g = exp(-exp(A_log) softplus(a + dt_bias)).
+                         logits (H) | decay inputs (H) | padding | first factors] (gate and decay inputs may be in `low` instead) -> fp32
+                         `u` [T, C + H + N] = [q | k | v | beta | g], N = H or H d:  causal depthwise convolution + SiLU over the first
+                         C = 2 G d + H dv channels (inputs before a sequence's first token are zero; the packed form leaves the last
+                         taps - 1 raw inputs of every sequence in `conv_state` [n_slots, taps - 1, C] fp32, oldest first; the step form
+                         reads and shifts it), q and k scaled to unit length per head (q also by d^-1/2), beta = sigmoid,
+                         g = exp(-exp(A_log) softplus(a + dt_bias)).
   delta_rule_scan / _step  the recurrence over each sequence from S = 0 (leaving S in `s_state` [n_slots, H, d, dv] fp32), or one
                          token per row against `s_state`, updated in place.  o [T, H, dv] fp32.
-  gated_head_norm        o / rms(o) * w * silu(gate) per head -> [T, H * dv] in the model dtype.
+  gated_head_norm        o / rms(o) * w * silu(gate) or sigmoid(gate) per head -> [T, H * dv] in the model dtype.
 """
 
 from __future__ import annotations
@@ -34,8 +38,32 @@ def _offsets(d):
     return nqk, nv, H, C
 
 
-def _finish_prepare(y, proj, d, A_log, dt_bias):
-    """y [T, C] fp32 = convolved channels -> u [T, C + 2H]."""
+def delta_low(proj, d, w_low):
+    """[T, low_rank_width] from the first factors' section of the projection rows; None without `decay_rank` / `gate_rank`."""
+    if not d.low_rank_width:
+        return None
+    from realhf_b200.models.sharding import delta_sections
+    from realhf_b200.ops.functional import linear
+    sec = delta_sections(d)
+    o = sum(sec[:-1])
+    return linear(proj[:, o:o + sec[-1]], w_low)
+
+
+def _gate_logits(proj, low, d):
+    """Views of the write strength's logits [T, H] and the decay inputs [T, N]."""
+    nqk, nv, H, C = _offsets(d)
+    ob = C + (0 if d.gate_rank else nv)
+    return proj[:, ob:ob + H], (low[:, :d.n_decays] if d.decay_rank else proj[:, ob + H:ob + 2 * H])
+
+
+def delta_gate(proj, low, d):
+    """View of the output gate's logits [T, H * dv]."""
+    nqk, nv, H, C = _offsets(d)
+    return low[:, d.low_rank_width - nv:] if d.gate_rank else proj[:, C:C + nv]
+
+
+def _finish_prepare(y, proj, d, A_log, dt_bias, low):
+    """y [T, C] fp32 = convolved channels -> u [T, C + H + N]."""
     nqk, nv, H, C = _offsets(d)
     T = y.shape[0]
     y = y * torch.sigmoid(y)
@@ -43,12 +71,13 @@ def _finish_prepare(y, proj, d, A_log, dt_bias):
     k = y[:, nqk:2 * nqk].view(T, d.n_kv_heads, d.qk_dim)
     q = q * torch.rsqrt(q.pow(2).sum(-1, keepdim=True) + d.unit_eps) * d.qk_dim ** -0.5
     k = k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + d.unit_eps)
-    beta = torch.sigmoid(proj[:, C + nv:C + nv + H].float())
-    g = torch.exp(-torch.exp(A_log.float()) * F.softplus(proj[:, C + nv + H:C + nv + 2 * H].float() + dt_bias.float()))
-    return torch.cat([q.reshape(T, nqk), k.reshape(T, nqk), y[:, 2 * nqk:], beta, g], -1).contiguous()
+    bl, al = _gate_logits(proj, low, d)
+    rate = torch.exp(A_log.float()).repeat_interleave(d.n_decays // H)
+    g = torch.exp(-rate * F.softplus(al.float() + dt_bias.float()))
+    return torch.cat([q.reshape(T, nqk), k.reshape(T, nqk), y[:, 2 * nqk:], torch.sigmoid(bl.float()), g], -1).contiguous()
 
 
-def delta_prepare_ref(proj, conv_w, A_log, dt_bias, d, pos, conv_state, tok_slot, remain):
+def delta_prepare_ref(proj, conv_w, A_log, dt_bias, d, pos, conv_state, tok_slot, remain, low=None):
     nqk, nv, H, C = _offsets(d)
     taps = d.conv_taps
     x = proj[:, :C].float()
@@ -61,21 +90,22 @@ def delta_prepare_ref(proj, conv_w, A_log, dt_bias, d, pos, conv_state, tok_slot
     if conv_state is not None and taps > 1:
         keep = (remain < taps - 1) & (tok_slot >= 0)
         conv_state[tok_slot[keep].long(), (taps - 2 - remain[keep]).long()] = x[keep]
-    return _finish_prepare(y, proj, d, A_log, dt_bias)
+    return _finish_prepare(y, proj, d, A_log, dt_bias, low)
 
 
-def delta_prepare(proj, conv_w, A_log, dt_bias, d, pos, conv_state=None, tok_slot=None, remain=None):
+def delta_prepare(proj, conv_w, A_log, dt_bias, d, pos, conv_state=None, tok_slot=None, remain=None, low=None):
     if use_native(proj) and d.conv_taps <= 8:
         nqk, nv, H, C = _offsets(d)
-        u = torch.empty(proj.shape[0], C + 2 * H, dtype=torch.float32, device=proj.device)
+        u = torch.empty(proj.shape[0], C + H + d.n_decays, dtype=torch.float32, device=proj.device)
         keep = conv_state is not None and d.conv_taps > 1
-        lib().delta_prepare(proj, conv_w, A_log, dt_bias, u, pos, conv_state if keep else None, tok_slot if keep else None,
-                            remain if keep else None, None, d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim, d.conv_taps, d.unit_eps)
+        lib().delta_prepare(proj, conv_w, *_gate_logits(proj, low, d), A_log, dt_bias, u, pos, conv_state if keep else None,
+                            tok_slot if keep else None, remain if keep else None, None, d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim, d.conv_taps,
+                            d.unit_eps)
         return u
-    return delta_prepare_ref(proj, conv_w, A_log, dt_bias, d, pos, conv_state, tok_slot, remain)
+    return delta_prepare_ref(proj, conv_w, A_log, dt_bias, d, pos, conv_state, tok_slot, remain, low)
 
 
-def delta_prepare_step_ref(proj, conv_w, A_log, dt_bias, d, conv_state, slots):
+def delta_prepare_step_ref(proj, conv_w, A_log, dt_bias, d, conv_state, slots, low=None):
     nqk, nv, H, C = _offsets(d)
     taps = d.conv_taps
     x = proj[:, :C].float()
@@ -86,29 +116,29 @@ def delta_prepare_step_ref(proj, conv_w, A_log, dt_bias, d, conv_state, slots):
         st = conv_state[idx]                                               # [B, taps - 1, C], oldest first
         y = y + (st * cw[:, :taps - 1].t().unsqueeze(0)).sum(1)
         conv_state[idx] = torch.cat([st[:, 1:], x.unsqueeze(1)], 1)
-    return _finish_prepare(y, proj, d, A_log, dt_bias)
+    return _finish_prepare(y, proj, d, A_log, dt_bias, low)
 
 
-def delta_prepare_step(proj, conv_w, A_log, dt_bias, d, conv_state, slots):
+def delta_prepare_step(proj, conv_w, A_log, dt_bias, d, conv_state, slots, low=None):
     if use_native(proj) and d.conv_taps <= 8:
         nqk, nv, H, C = _offsets(d)
-        u = torch.empty(proj.shape[0], C + 2 * H, dtype=torch.float32, device=proj.device)
-        lib().delta_prepare(proj, conv_w, A_log, dt_bias, u, None, conv_state if d.conv_taps > 1 else None, None, None, slots,
-                            d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim, d.conv_taps, d.unit_eps)
+        u = torch.empty(proj.shape[0], C + H + d.n_decays, dtype=torch.float32, device=proj.device)
+        lib().delta_prepare(proj, conv_w, *_gate_logits(proj, low, d), A_log, dt_bias, u, None, conv_state if d.conv_taps > 1 else None, None, None,
+                            slots, d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim, d.conv_taps, d.unit_eps)
         return u
-    return delta_prepare_step_ref(proj, conv_w, A_log, dt_bias, d, conv_state, slots)
+    return delta_prepare_step_ref(proj, conv_w, A_log, dt_bias, d, conv_state, slots, low)
 
 
 def _split_u(u, d):
     nqk, nv, H, C = _offsets(d)
     T = u.shape[0]
     return (u[:, :nqk].view(T, d.n_kv_heads, d.qk_dim), u[:, nqk:2 * nqk].view(T, d.n_kv_heads, d.qk_dim),
-            u[:, 2 * nqk:C].view(T, H, d.v_dim), u[:, C:C + H], u[:, C + H:C + 2 * H])
+            u[:, 2 * nqk:C].view(T, H, d.v_dim), u[:, C:C + H], u[:, C + H:].view(T, H, -1))
 
 
 def _delta_token(S, q, k, v, beta, g):
-    """S [H, d, dv]; q, k [H, d]; v [H, dv]; beta, g [H] -> (S', o [H, dv])."""
-    S = S * g.view(-1, 1, 1)
+    """S [H, d, dv]; q, k [H, d]; v [H, dv]; beta [H]; g [H, 1] or [H, d] -> (S', o [H, dv])."""
+    S = S * g.unsqueeze(-1)
     w = beta.view(-1, 1) * (v - torch.einsum("hdv,hd->hv", S, k))
     S = S + k.unsqueeze(-1) * w.unsqueeze(1)
     return S, torch.einsum("hdv,hd->hv", S, q)
@@ -130,11 +160,12 @@ def delta_rule_scan_ref(u, d, cu_seqlens, s_state, slots):
 
 
 def delta_rule_scan(u, d, cu_seqlens, s_state=None, slots=None):
-    """u [T, C + 2H] fp32 (see `delta_prepare`), sequences given by cu_seqlens, each from S = 0.  Returns o [T, H, dv] fp32; with
+    """u [T, C + H + N] fp32 (see `delta_prepare`), sequences given by cu_seqlens, each from S = 0.  Returns o [T, H, dv] fp32; with
     `s_state` and `slots` [n_seqs] int32, sequence b's final state is left in s_state[slots[b]] (slots[b] < 0: dropped)."""
     if use_native(u) and d.qk_dim <= 512:
         o = torch.empty(u.shape[0], d.n_heads, d.v_dim, dtype=torch.float32, device=u.device)
-        lib().delta_rule_scan(u, o, cu_seqlens, s_state, slots if s_state is not None else None, d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim)
+        lib().delta_rule_scan(u, o, cu_seqlens, s_state, slots if s_state is not None else None, d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim,
+                              bool(d.decay_rank))
         return o
     return delta_rule_scan_ref(u, d, cu_seqlens, s_state, slots)
 
@@ -154,25 +185,25 @@ def delta_rule_step(u, d, s_state, slots):
     """One token per row: s_state[slots[b]] (slots None: row b is slot b) is updated in place.  Returns o [B, H, dv] fp32."""
     if use_native(u) and d.qk_dim <= 512:
         o = torch.empty(u.shape[0], d.n_heads, d.v_dim, dtype=torch.float32, device=u.device)
-        lib().delta_rule_step(u, o, s_state, slots, d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim)
+        lib().delta_rule_step(u, o, s_state, slots, d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim, bool(d.decay_rank))
         return o
     return delta_rule_step_ref(u, d, s_state, slots)
 
 
-def gated_head_norm_ref(o, w, gate, eps, out_dtype):
+def gated_head_norm_ref(o, w, gate, eps, out_dtype, act="silu"):
     T, H, dv = o.shape
     n = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w.float()
-    gt = gate.float().view(T, H, dv)
-    return (n * gt * torch.sigmoid(gt)).reshape(T, H * dv).to(out_dtype)
+    gt = gate.float().reshape(T, H, dv)
+    return (n * (F.silu(gt) if act == "silu" else torch.sigmoid(gt))).reshape(T, H * dv).to(out_dtype)
 
 
-def gated_head_norm(o, w, gate, eps: float, out_dtype):
-    """o [T, H, dv] fp32, w [dv], gate [T, H * dv] (a column slice of the projection output; unit column stride)."""
+def gated_head_norm(o, w, gate, eps: float, out_dtype, act: str = "silu"):
+    """o [T, H, dv] fp32, w [dv], gate [T, H * dv] (a column slice of the projection output; unit column stride), act silu or sigmoid."""
     if use_native(o):
         out = torch.empty(o.shape[0], o.shape[1] * o.shape[2], dtype=out_dtype, device=o.device)
-        lib().gated_head_norm(o, w, gate, out, eps)
+        lib().gated_head_norm(o, w, gate, out, eps, act == "sigmoid")
         return out
-    return gated_head_norm_ref(o, w, gate, eps, out_dtype)
+    return gated_head_norm_ref(o, w, gate, eps, out_dtype, act)
 
 
 # ------------------------------------------------------------------------------------------------ matrix-memory LSTM
@@ -287,11 +318,12 @@ def decay_table(d, device) -> torch.Tensor:
     return hit
 
 
-def _rotate_heads_ref(x, p, rot, inv_freq):
-    """x [T, H, d] fp32: the first rot.dims dimensions of every head turn by p * f_i; pairs (i, i + dims / 2) or (2i, 2i + 1)."""
+def _rotate_heads_ref(x, p, rot, inv_freq, mscale: float = 1.0):
+    """x [T, H, d] fp32: the first rot.dims dimensions of every head turn by p * f_i (cos and sin times mscale); pairs (i, i + dims / 2)
+    or (2i, 2i + 1)."""
     n = rot.dims
     ang = p.float().unsqueeze(-1) * inv_freq                 # fp32 product, as the kernels form it
-    cs, sn = torch.cos(ang).unsqueeze(1), torch.sin(ang).unsqueeze(1)
+    cs, sn = (torch.cos(ang) * mscale).unsqueeze(1), (torch.sin(ang) * mscale).unsqueeze(1)
     out = x.clone()
     if rot.interleaved:
         a, b = x[..., 0:n:2], x[..., 1:n:2]
