@@ -38,10 +38,10 @@ def silu(x):
 
 def distance_bucket(n: int, rows: int, bias_max: float) -> int:
     """Row of the bias table for distance n: exact below rows / 2, then logarithmic up to bias_max, the last row beyond."""
-    half = rows / 2
+    half = rows // 2
     if n < half:
         return n
-    return min(rows - 1, math.floor(half + math.floor(math.log(n / half) / math.log(bias_max / half) * (rows - half))))
+    return min(rows - 1, half + math.floor(math.log(n / half) / math.log(bias_max / half) * (rows - half)))
 
 
 def frequencies(rot: dict):
@@ -70,7 +70,7 @@ def rotate_half(x: torch.Tensor, rot: dict) -> torch.Tensor:
 
 
 def attend(q, k, v, scale, window=None, bias=None, sink=None) -> torch.Tensor:
-    """q [T, H, d], k [T, G, d], v [T, G, dv] -> [T, H, dv].  bias(n, h): what is added to the scaled score at distance n; sink [H]."""
+    """q [T, H, d], k [T, G, d], v [T, G, dv] -> [T, H, dv].  bias [T, H]: what is added to the scaled score at every distance; sink [H]."""
     T, H, _ = q.shape
     G = k.shape[1]
     i, j = torch.arange(T).unsqueeze(1), torch.arange(T).unsqueeze(0)
@@ -82,7 +82,7 @@ def attend(q, k, v, scale, window=None, bias=None, sink=None) -> torch.Tensor:
         g = h // (H // G)
         s = (q[:, h] @ k[:, g].T) * scale
         if bias is not None:
-            s = s + torch.tensor([bias(n, h) for n in range(T)], dtype=F64)[(i - j).clamp(min=0)]
+            s = s + bias[(i - j).clamp(min=0), h]
         s = s.masked_fill(~ok, -math.inf)
         mx = s.max(-1, keepdim=True).values
         if sink is not None:
@@ -101,7 +101,7 @@ def biased_attention(w, m: dict, h: torch.Tensor) -> torch.Tensor:
     H, G, d = m["heads"], m["kv_heads"], m["dim"]
     rel = w["rel"]
     q, k = (h @ w["q"].T).view(T, H, d), (h @ w["k"].T).view(T, G, d)
-    bias = lambda n, hh: float(rel[distance_bucket(n, rel.shape[0], m["bias_max"]), hh])
+    bias = rel[torch.tensor([distance_bucket(n, rel.shape[0], m["bias_max"]) for n in range(T)])]
     mask = m.get("mask")
     o = attend(q, k, k, m["scale"], mask["size"] if mask else None, bias, w["sink"])
     return o.reshape(T, -1) @ w["o"].T
@@ -137,16 +137,14 @@ def unit(x):
 def delta_core(q, k, v, beta, decay) -> torch.Tensor:
     """q, k [T, G, d], v [T, H, dv], beta [T, H], decay [T, H, d] (one factor per row of S).  S starts at zero; returns o [T, H, dv]."""
     T, H, dv = v.shape
-    G, d = q.shape[1], q.shape[2]
+    q, k = (x.repeat_interleave(H // x.shape[1], 1) for x in (q, k))      # head h reads q / k head floor(h / (H / G))
     o = torch.zeros(T, H, dv, dtype=F64)
-    for h in range(H):
-        g = h // (H // G)
-        S = torch.zeros(d, dv, dtype=F64)
-        for t in range(T):
-            S = decay[t, h].unsqueeze(1) * S
-            u = beta[t, h] * (v[t, h] - S.T @ k[t, g])
-            S = S + torch.outer(k[t, g], u)
-            o[t, h] = S.T @ q[t, g]
+    S = torch.zeros(H, q.shape[2], dv, dtype=F64)
+    for t in range(T):
+        S = decay[t].unsqueeze(-1) * S
+        u = beta[t].unsqueeze(-1) * (v[t] - (k[t].unsqueeze(1) @ S).squeeze(1))
+        S = S + k[t].unsqueeze(-1) * u.unsqueeze(1)
+        o[t] = (q[t].unsqueeze(1) @ S).squeeze(1)
     return o
 
 
@@ -242,8 +240,8 @@ def greedy(sd, cfg, prompt: List[int], n_new: int) -> List[int]:
 
 
 def tensor_shapes(cfg: dict) -> Dict[str, tuple]:
-    """Shapes of every tensor; the two ranks of `parallel`'s right side and the rows of its bias table are no part of the checkpoint's
-    config: `_rank_a`, `_rank_g` (of the right side) and `_rel_rows` (of the left side) name them in a test's config."""
+    """Shapes of every tensor.  The inner ranks of `parallel`'s right side and the rows of its bias table are not part of a checkpoint's
+    config; a test's config names them `decay_rank`, `gate_rank` and `bias_rows`."""
     W = cfg["width"]
     s = {"embed": (cfg["vocab"], W), "final.norm": (W,)}
     if cfg.get("loop"):
@@ -254,7 +252,7 @@ def tensor_shapes(cfg: dict) -> Dict[str, tuple]:
         q = p + "mix.left."
         s.update({q + "q": (l["heads"] * l["dim"], W), q + "k": (l["kv_heads"] * l["dim"], W), q + "o": (W, l["heads"] * l["vdim"])})
         if lay["type"] == "parallel":
-            s.update({q + "rel": (l["_rel_rows"], l["heads"]), q + "sink": (l["heads"],), q + "out": (W,)})
+            s.update({q + "rel": (l["bias_rows"], l["heads"]), q + "sink": (l["heads"],), q + "out": (W,)})
         else:
             s[q + "v"] = (l["kv_heads"] * l["vdim"], W)
         q = p + "mix.right."
@@ -262,7 +260,7 @@ def tensor_shapes(cfg: dict) -> Dict[str, tuple]:
         s.update({q + "q": (G * d, W), q + "q.conv": (G * d, t), q + "k": (G * d, W), q + "k.conv": (G * d, t), q + "v": (H * dv, W),
                   q + "v.conv": (H * dv, t), q + "b": (H, W), q + "A_log": (H,), q + "norm": (dv,), q + "o": (W, H * dv)})
         if lay["type"] == "parallel":
-            ra, rg = r["_rank_a"], r["_rank_g"]
+            ra, rg = r["decay_rank"], r["gate_rank"]
             s.update({q + "a1": (ra, W), q + "a2": (H * d, ra), q + "dt_bias": (H * d,), q + "g1": (rg, W), q + "g2": (H * dv, rg), q + "out": (W,)})
         else:
             s.update({q + "a": (H, W), q + "dt_bias": (H,), q + "g": (H * dv, W)})
