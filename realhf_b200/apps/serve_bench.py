@@ -1,7 +1,8 @@
 """Prefill / decode throughput of a heterogeneous-stack design next to the closest homogeneous model of equal size, and the
 roofline position of its kernels next to the like kernels of that model.  Reached through `bench.py --serve-bench rapodra`,
-`--serve-bench tizodra`, `--serve-bench defilorn`, `--serve-bench buvesun` or `--serve-bench tokatar` (the default workload of bench.py
-is unaffected).  Buvesun and Tokatar are also timed beside a Defilorn of equal size, the closest heterogeneous stack (window attention,
+`--serve-bench tizodra`, `--serve-bench defilorn`, `--serve-bench buvesun`, `--serve-bench tokatar` or `--serve-bench nufatar` (the default
+workload of bench.py is unaffected).  Nufatar is also timed beside a Tizodra of equal size (window attention with a sink, the delta rule),
+Buvesun and Tokatar beside a Defilorn of equal size, the closest heterogeneous stack (window attention,
 rotated latent attention, a matrix-state mixer, dense and routed feed-forwards).
 
 Both models run through `models.generation`: prefill = `prefill_into_state` (the packed prefill `generate` performs) into a
@@ -128,11 +129,32 @@ def tokatar_config(s: dict, n_layers: int = 4) -> dict:
                 vocab=s["vocab"], width=s["width"])
 
 
+NUFATAR_SIZES = {
+    # the Tizodra sizes plus: rows and reach of the bias table, inner rank of the two-factor projections, rotated dimensions
+    "1b-like": dict(TIZODRA_SIZES["1b-like"], rows=32, bias_max=400, rank=128, rot_dims=64),
+    "7b-like": dict(TIZODRA_SIZES["7b-like"], rows=32, bias_max=800, rank=128, rot_dims=64),
+}
+
+
+def nufatar_config(s: dict, n_layers: int = 4) -> dict:
+    """The two mixers in turn, every block with a feed-forward; the inner blocks in a loop of one pass (so the step vector is on the path)."""
+    left = dict(dim=s["dim"], heads=s["heads"], kv_heads=s["kv_heads"], vdim=s["vdim"], scale=s["dim"] ** -0.5)
+    right = dict(conv=s["conv"], dim=s["dim"], heads=s["heads"], kv_heads=s["kv_heads"], vdim=s["vdim"])
+    par = dict(type="parallel", mlp=dict(kind="dense", ff=s["ff"]),
+               mixer=dict(left=dict(left, bias_max=s["bias_max"], bias_rows=s["rows"], mask=dict(size=s["window"])),
+                          right=dict(right, decay_rank=s["rank"], gate_rank=s["rank"])))
+    par2 = dict(type="parallel_2", mlp=dict(kind="dense", ff=s["ff"]),
+                mixer=dict(left=dict(left, rot=dict(base=5e5, dims=s["rot_dims"], scaling=dict(factor=8.0, fast=32.0, original=4096, slow=1.0))),
+                           left_scale=0.7, right=right, right_scale=0.6))
+    return dict(architecture="Nufatar", layers=[par2 if i % 2 else par for i in range(n_layers)], loop=dict(start=1, stop=max(2, n_layers - 1), times=1),
+                norm=dict(eps=1e-5), vocab=s["vocab"], width=s["width"])
+
+
 def _hetero_model(design: str, s: dict, n_layers: int, dev):
     from realhf_b200.models import hf_io
     from realhf_b200.models.real_model import ReaLModel
     cfg = {"rapodra": rapodra_config, "tizodra": tizodra_config, "defilorn": defilorn_config, "buvesun": buvesun_config,
-           "tokatar": tokatar_config}[design](s, n_layers)
+           "tokatar": tokatar_config, "nufatar": nufatar_config}[design](s, n_layers)
     m = ReaLModel(hf_io.family(design).config_from_dict(cfg, False), dtype=torch.bfloat16, device=dev).init_random_fast()
     for p in m.parameters():
         p.requires_grad_(False)
@@ -185,6 +207,8 @@ def model_numbers(name: str, s: dict, n_layers: int, batch: int, prompt_len: int
     arms = [(design, new), ("llama-equal-size", old)]
     if design in ("buvesun", "tokatar"):
         arms.insert(1, ("defilorn-equal-size", _hetero_model("defilorn", s, n_layers, dev)))
+    if design == "nufatar":
+        arms.insert(1, ("tizodra-equal-size", _hetero_model("tizodra", s, n_layers, dev)))
     for label, m in arms:
         # prefill: the packed prefill into a standing decode state (`prefill_into_state`, what `generate` calls), so that the
         # number is the model's and not the caching allocator's (a fresh multi-GB state per `generate` call can fall into
@@ -792,8 +816,157 @@ def tokatar_kernel_numbers(name: str, s: dict, batch: int, prompt_len: int, ctx:
     return rows
 
 
+def nufatar_kernel_numbers(name: str, s: dict, batch: int, prompt_len: int, ctx: int, dev, peaks: Dict[str, float]) -> List[dict]:
+    """The Nufatar kernels next to the like kernels of the closest models at the same token count and head sizes: Tizodra's window
+    attention, delta rule and head norm, Tokatar's row preparation, Buvesun's two-branch norm, LLaMA's norm and attention.  Attention
+    FLOPs count the visible (query, key) pairs; the fp32 recurrences are held against the nominal fp32 CUDA-core rate or their bytes."""
+    import dataclasses
+
+    from realhf_b200.models import hf_io
+    from realhf_b200.models.hetero_block import packed_meta
+    from realhf_b200.models.sharding import delta_sections
+    from realhf_b200.ops import attention as A
+    from realhf_b200.ops import functional as OF
+    from realhf_b200.ops import recurrent as RC
+    bf = torch.bfloat16
+    rc = hf_io.family("nufatar").config_from_dict(nufatar_config(s, 2), False)
+    tz = hf_io.family("tizodra").config_from_dict(tizodra_config(s, 3), False)
+    w1, d1, w2, d2 = rc.blocks[0].wattn, rc.blocks[0].delta, rc.blocks[1].wattn, rc.blocks[1].delta
+    wt = next(b.wattn for b in tz.blocks if b.wattn is not None)
+    wt = dataclasses.replace(wt, out_gate=False)
+    W, H, G, d, dv, win = s["width"], s["heads"], s["kv_heads"], s["dim"], s["vdim"], s["window"]
+    T = batch * prompt_len
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    fp32_tflops = 148 * 128 * 2 * 1.9e9 / 1e12
+    rows = []
+
+    def add(kernel, like, ms, nbytes, flops, simt_fp32=False):
+        peak = fp32_tflops if simt_fp32 else peaks["bf16_tflops"]
+        floor_ms = max(nbytes / (peaks["hbm_gbs"] * 1e9), flops / (peak * 1e12)) * 1e3
+        rows.append(dict(bench="kernel", size=name, kernel=kernel, like=like, ms=round(ms, 4), gbytes=round(nbytes / 1e9, 4),
+                         gflop=round(flops / 1e9, 2), roofline_ms=round(floor_ms, 4), frac_of_measured_roofline=round(floor_ms / ms, 4),
+                         flop_peak="fp32 CUDA cores (nominal)" if simt_fp32 else "bf16 tensor (measured)"))
+
+    def t(fn, iters=10):
+        return _time(fn, iters, flush=flush)
+    rb = lambda *n: torch.randn(*n, device=dev).to(bf)
+    cu = torch.arange(0, batch + 1, device=dev, dtype=torch.int32) * prompt_len
+    slots = torch.arange(batch, dtype=torch.int32, device=dev)
+    meta = packed_meta(cu, T, slots, None, prompt_len)
+    # ---- row-wise
+    x32, y1, y2, y3 = torch.randn(T, W, device=dev), rb(T, W), rb(T, W), rb(T, W)
+    vec = torch.ones(W, device=dev, dtype=bf)
+    for T_, label in ((T, "prefill"), (batch, "decode")):
+        x_, a_, b_, c_ = x32[:T_], y1[:T_], y2[:T_], y3[:T_]
+        add(f"branch_add_norm_ (two normalised sides + feed-forward into the fp32 stream, next norm; {label})", False,
+            t(lambda: OF.branch_add_norm_(x_, a_, b_, c_, 1e-5, 0.5, 0.5, vec, vec, None, vec, 1.0, bf)), T_ * W * 16, 0)
+        add(f"branch_add_norm_ (two weighed sides + feed-forward + step vector, next norm; {label})", False,
+            t(lambda: OF.branch_add_norm_(x_, a_, b_, c_, 1e-5, 0.7, 0.6, None, None, vec, vec, 1.0, bf)), T_ * W * 16, 0)
+        add(f"residual_add_centred_norm_ (buvesun: two branches, output norm, add, next norm; {label})", True,
+            t(lambda: OF.residual_add_centred_norm_(x_, a_, vec, 1e-5, vec, 0.7, b_, 0.6, 1.1, vec, bf)), T_ * W * 14, 0)
+        add(f"add_rms_norm_ (tizodra: fp32 stream += branch, next norm; {label})", True, t(lambda: OF.add_rms_norm_(x_, a_, vec, 1e-5, bf)), T_ * W * 12, 0)
+    del x32, y1, y2, y3
+    # ---- attention rows and caches
+    rows1, rows2 = w1.cache_rows(prompt_len + 64), w2.cache_rows(prompt_len + 64)
+    wide1, wide2 = rb(T, (H + G) * d), rb(T, (H + G) * d + G * dv)
+    c1, kc2, vc2 = (torch.zeros(batch, G, r, n, device=dev, dtype=bf) for r, n in ((rows1, d), (rows2, d), (rows2, dv)))
+    kw = dict(pos=meta.pos, tok_slot=meta.tok_slot, remain=meta.remain)
+    kept = lambda r, n: batch * min(prompt_len, r) * G * n * 4
+    add("window_prepare_ (parallel: cache fill only; prefill)", False, t(lambda: A.window_prepare_(wide1, w1, None, None, 1e-5, k_cache=c1, v_cache=c1, **kw)),
+        kept(rows1, d), 0)
+    add("window_prepare_ (parallel_2: rotate q and k with a factor, cache fill; prefill)", False,
+        t(lambda: A.window_prepare_(wide2, w2, None, None, 1e-5, k_cache=kc2, v_cache=vc2, **kw)), T * (H + G) * d * 4 + kept(rows2, dv) + kept(rows2, d) // 2, 0)
+    kt, vt = (torch.zeros(batch, G, wt.cache_rows(prompt_len + 64), n, device=dev, dtype=bf) for n in (d, dv))
+    add("value_norm_store (tizodra: value norm, cache fill; prefill)", True,
+        t(lambda: A.value_norm_store(wide2, wt, 1e-5, kt, vt, meta.tok_slot, meta.pos, meta.remain)), T * G * (d + 3 * dv) * 2, 0)
+    ta = hf_io.family("tokatar").config_from_dict(tokatar_config(TOKATAR_SIZES[name], 2), False).blocks[0].wattn
+    tk, tv = (torch.zeros(batch, G, ta.cache_rows(prompt_len + 64), n, device=dev, dtype=bf) for n in (d, dv))
+    add("window_prepare_ (tokatar attention: rotate q and k, cache fill; prefill)", True,
+        t(lambda: A.window_prepare_(wide2, ta, None, None, 1e-5, k_cache=tk, v_cache=tv, **kw)),
+        T * ((H + G) * d * 4 + G * dv * 2) + kept(ta.cache_rows(prompt_len + 64), d), 0)
+    one = wide2[:batch].clone()
+    lens = torch.full((batch,), ctx, dtype=torch.int32, device=dev)
+    add("window_prepare_ (parallel_2; decode)", False, t(lambda: A.window_prepare_(one, w2, None, None, 1e-5, cache_lens=lens)), batch * (H + G) * d * 4, 0)
+    add("window_prepare_ (tokatar attention; decode)", True, t(lambda: A.window_prepare_(one, ta, None, None, 1e-5, cache_lens=lens)), batch * (H + G) * d * 4, 0)
+    del c1, kc2, vc2, kt, vt, tk, tv
+    # ---- attention
+    rel, sink, temp = rb(s["rows"], H), torch.zeros(H, device=dev, dtype=bf), torch.ones(H, device=dev, dtype=bf)
+    pairs = lambda wn: batch * sum(min(p + 1, wn) for p in range(prompt_len))
+    full = batch * prompt_len * (prompt_len + 1) // 2
+    add("sink_window_attention (parallel: shared keys / values, distance bias, sink, window; prefill, tcgen05)", False,
+        t(lambda: A.sink_window_attention(wide1, A.window_values(wide1, w1), w1, None, sink, meta.pos, cu, prompt_len, rel=rel), 5),
+        T * (H * (d + dv) + G * d) * 2, 2.0 * pairs(win) * H * (d + dv))
+    v_n = wide2[:, (H + G) * d:].contiguous()
+    kp = batch * sum(min(p + 1, win) + max(0, min(s["keep"], p + 1 - win)) for p in range(prompt_len))
+    add("sink_window_attention (tizodra: temperature, slope, sink, window + kept keys; prefill, tcgen05)", True,
+        t(lambda: A.sink_window_attention(wide2, v_n, wt, temp, sink, meta.pos, cu, prompt_len), 5), T * (H + G) * (d + dv) * 2, 2.0 * kp * H * (d + dv))
+    add("sink_window_attention (parallel_2: every earlier key; prefill, tcgen05)", False,
+        t(lambda: A.sink_window_attention(wide2, A.window_values(wide2, w2), w2, None, None, meta.pos, cu, prompt_len), 5), T * (H + G) * (d + dv) * 2,
+        2.0 * full * H * (d + dv))
+    for dq, dvv in ((64, 128), (128, 64)):
+        a = dataclasses.replace(w2, qk_dim=dq, v_dim=dvv, rotary=None)
+        xq = rb(T, (H + G) * dq + G * dvv)
+        add(f"sink_window_attention (parallel_2, query / key size {dq}, value size {dvv}; prefill, tcgen05)", False,
+            t(lambda: A.sink_window_attention(xq, A.window_values(xq, a), a, None, None, meta.pos, cu, prompt_len), 5), T * (H + G) * (dq + dvv) * 2,
+            2.0 * full * H * (dq + dvv))
+    qkv = rb(T, (H + 2 * G) * d)
+    add("varlen attention tcgen05 (llama, prefill, full causal)", True, t(lambda: A.varlen_attention_qkv(qkv, cu, prompt_len, H, G, d, None, True), 5),
+        T * (2 * H + 2 * G) * d * 2, 4.0 * full * H * d)
+    del wide1, wide2, v_n, qkv, xq
+    keys = min(ctx + 1, win)
+    q1, q2 = rb(batch, (H + G) * d), rb(batch, (H + G) * d + G * dv)
+    kc = rb(batch, G, w1.cache_rows(ctx + 64), d)
+    add(f"sink_window_decode_attention (parallel: one shared cache, bias, sink; {keys} keys)", False,
+        t(lambda: A.sink_window_decode_attention(q1, w1, None, sink, kc, kc, lens, None, 1e-5, rel=rel)), batch * keys * G * d * 2, 2.0 * batch * H * keys * (d + dv))
+    kt, vt = rb(batch, G, wt.cache_rows(ctx + 64), d), rb(batch, G, wt.cache_rows(ctx + 64), dv)
+    tkeys = keys + max(0, min(s["keep"], ctx + 1 - win))
+    add(f"sink_window_decode_attention (tizodra; {tkeys} keys)", True, t(lambda: A.sink_window_decode_attention(q2, wt, temp, sink, kt, vt, lens, None, 1e-5)),
+        batch * tkeys * G * (d + dv) * 2, 2.0 * batch * H * tkeys * (d + dv))
+    k2, v2 = rb(batch, G, ctx + 64, d), rb(batch, G, ctx + 64, dv)
+    add(f"sink_window_decode_attention (parallel_2; all {ctx + 1} keys)", False,
+        t(lambda: A.sink_window_decode_attention(q2, w2, None, None, k2, v2, lens, None, 1e-5)), batch * (ctx + 1) * G * (d + dv) * 2,
+        2.0 * batch * H * (ctx + 1) * (d + dv))
+    kl, vl = (torch.zeros(batch, G, ctx + 64, d, device=dev, dtype=bf).permute(0, 2, 1, 3) for _ in range(2))
+    cos, sin = OF.rope_tables(ctx + 64, d, 10000.0, dev)
+    ql = rb(batch, (H + 2 * G) * d)
+    add(f"decode_attention (llama, all {ctx + 1} keys)", True, t(lambda: A.decode_attention(ql, kl, vl, lens, H, G, d, None, cos, sin)),
+        batch * (ctx + 1) * G * d * 4, 4.0 * batch * H * (ctx + 1) * d)
+    del k2, v2, kl, vl
+    # ---- delta rule: a decay per channel beside one per head
+    conv_w, A_log = rb(d1.conv_channels, d1.conv_taps) * 0.5, torch.zeros(H, device=dev, dtype=bf)
+    C = d1.conv_channels
+    conv_state, s_state = torch.zeros(batch, d1.conv_taps - 1, C, device=dev), torch.zeros(batch, H, d, dv, device=dev)
+    wo = torch.ones(dv, device=dev, dtype=bf)
+    for dl, like, label in ((d1, False, "parallel: a decay per channel"), (d2, True, "tizodra, parallel_2: a decay per head")):
+        N, act = dl.n_decays, dl.gate
+        dtb = torch.zeros(N, device=dev, dtype=bf)
+        for n, form in ((T, "prefill"), (batch, "decode")):
+            proj = rb(n, sum(delta_sections(dl)))
+            low_w = rb(dl.low_rank_width, 2 * s["rank"]) * 0.05 if dl.low_rank_width else None
+            low = RC.delta_low(proj, dl, low_w)
+            if low is not None:
+                add(f"delta_low (second factors of decay and gate, one product; {form})", False, t(lambda: RC.delta_low(proj, dl, low_w)),
+                    (n * (2 * s["rank"] + dl.low_rank_width) + low_w.numel()) * 2, 2.0 * n * low_w.numel())
+            io = n * (C * (2 + 4) + (H + N) * (2 + 4)) + (n * C * 8 * (dl.conv_taps - 1) if form == "decode" else 0)
+            if form == "prefill":
+                prep = lambda: RC.delta_prepare(proj, conv_w, A_log, dtb, dl, meta.pos, conv_state, meta.tok_slot, meta.remain, low=low)
+                scan = lambda: RC.delta_rule_scan(u, dl, cu, s_state, meta.seq_slot)
+            else:
+                prep = lambda: RC.delta_prepare_step(proj, conv_w, A_log, dtb, dl, conv_state, None, low=low)
+                scan = lambda: RC.delta_rule_step(u, dl, s_state, None)
+            add(f"delta_prepare ({label}; {form})", like, t(prep), io, n * C * 2.0 * dl.conv_taps, simt_fp32=True)
+            u = prep()
+            add(f"delta_rule ({label}; {form})", like, t(scan, 3), n * (C + H + N + H * dv) * 4 + (batch * H * d * dv * 8 if form == "decode" else 0),
+                n * H * 8.0 * d * dv, simt_fp32=True)
+            o = scan()
+            gate = RC.delta_gate(proj, low, dl)
+            add(f"gated_head_norm ({act}; {form})", like, t(lambda: RC.gated_head_norm(o, wo, gate, 1e-5, bf, act)), n * H * dv * 8, 0)
+            del proj, low, u, o, gate
+    return rows
+
+
 def run(design: str, sizes: List[str] = None, n_layers: int = 4) -> List[dict]:
-    assert design in ("rapodra", "tizodra", "defilorn", "buvesun", "tokatar")
+    assert design in ("rapodra", "tizodra", "defilorn", "buvesun", "tokatar", "nufatar")
     dev = torch.device("cuda:0")
     torch.cuda.set_device(dev)
     peaks = dict(hbm_gbs=6650.0, bf16_tflops=1590.0, source="fallback")
@@ -805,12 +978,12 @@ def run(design: str, sizes: List[str] = None, n_layers: int = 4) -> List[dict]:
             peaks = dict(hbm_gbs=float(d["hbm_gbs"]), bf16_tflops=float(d["bf16_tflops"]), source="measured")
     results = [dict(bench="peaks", **peaks)]
     table = {"rapodra": SIZES, "tizodra": TIZODRA_SIZES, "defilorn": DEFILORN_SIZES, "buvesun": BUVESUN_SIZES,
-             "tokatar": TOKATAR_SIZES}[design]
+             "tokatar": TOKATAR_SIZES, "nufatar": NUFATAR_SIZES}[design]
     for name in sizes or list(table):
         s = table[name]
         results += model_numbers(name, s, n_layers, batch=32, prompt_len=1024, new_tokens=33, dev=dev, design=design)
         kn = {"rapodra": kernel_numbers, "tizodra": tizodra_kernel_numbers, "defilorn": defilorn_kernel_numbers,
-              "buvesun": buvesun_kernel_numbers, "tokatar": tokatar_kernel_numbers}[design]
+              "buvesun": buvesun_kernel_numbers, "tokatar": tokatar_kernel_numbers, "nufatar": nufatar_kernel_numbers}[design]
         results += kn(name, s, batch=32, prompt_len=1024, ctx=2048, dev=dev, peaks=peaks)
     for r in results:
         print(json.dumps(r), flush=True)

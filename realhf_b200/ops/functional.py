@@ -462,8 +462,7 @@ def linear_f32(x, w):
         from realhf_b200.ops import gemm as G
         x2 = x.reshape(-1, x.shape[-1])
         if gemm_impl() is G.linear and G.supported(x2, w):
-            if x2.stride(-1) != 1 or x2.stride(0) % 8 != 0 or x2.data_ptr() % 16 != 0:
-                x2 = x2.contiguous()
+            x2 = G.tma_rows(x2)
             return G.gemm(x2, w, out_dtype=torch.float32).view(*x.shape[:-1], w.shape[0])
     return F.linear(x, w).float()
 
@@ -777,8 +776,7 @@ def clamped_gated_linear(x, w_gate_up, limit: float, alpha: float = 1.702):
         from realhf_b200.ops import gemm as G
         if gemm_impl() is G.linear and G.gated_linear_supported(x, w_gate_up):
             x2 = x.reshape(-1, x.shape[-1])
-            if x2.stride(-1) != 1 or x2.stride(0) % 8 != 0 or x2.data_ptr() % 16 != 0:
-                x2 = x2.contiguous()
+            x2 = G.tma_rows(x2)
             out = lib().gemm_glu_clamped(x2, w_gate_up, limit, alpha, G._sms(x.device))
             return out.view(*x.shape[:-1], w_gate_up.shape[0] // 2)
     return clamped_glu(linear(x, w_gate_up), limit, alpha)
@@ -852,8 +850,7 @@ def relu2_linear(x, w_up, bias=None, act_cols: Optional[int] = None):
         x2 = x.reshape(-1, x.shape[-1])
         if (gemm_impl() is G.linear and G.supported(x2, w_up) and x2.shape[0] > 128 and w_up.shape[0] % 8 == 0 and w_up.is_contiguous()
                 and os.environ.get("REAL_GEMM_GLU", "1") == "1"):
-            if x2.stride(-1) != 1 or x2.stride(0) % 8 != 0 or x2.data_ptr() % 16 != 0:
-                x2 = x2.contiguous()
+            x2 = G.tma_rows(x2)
             out = lib().gemm_relu2(x2, w_up, G._sms(x.device), bias, act_cols or 0)
             return out.view(*x.shape[:-1], w_up.shape[0])
     y = linear(x, w_up, bias)

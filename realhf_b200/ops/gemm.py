@@ -62,12 +62,19 @@ def supported(x: torch.Tensor, w: torch.Tensor) -> bool:
             and w.shape[0] % 8 == 0 and w.stride(-1) == 1 and w.stride(0) % 8 == 0)
 
 
+def tma_rows(x: torch.Tensor) -> torch.Tensor:
+    """x [M, K] itself if a TMA descriptor can describe it (unit column stride, 16-byte aligned rows), else a packed copy.  (Not
+    `contiguous()`: a one-row slice counts as contiguous wherever it starts.)"""
+    if x.stride(-1) != 1 or x.stride(0) % 8 != 0 or x.data_ptr() % 16 != 0:
+        return x.clone(memory_format=torch.contiguous_format)
+    return x
+
+
 class _Linear(torch.autograd.Function):
     @staticmethod
     def forward(ctx, x, w, bias):
         x2 = x.reshape(-1, x.shape[-1])
-        if x2.stride(-1) != 1 or x2.stride(0) % 8 != 0 or x2.data_ptr() % 16 != 0:
-            x2 = x2.contiguous()
+        x2 = tma_rows(x2)
         ctx.save_for_backward(x2, w)
         ctx.has_bias = bias is not None
         ctx.x_shape = x.shape
@@ -88,8 +95,7 @@ def _linear_backward(x2, w, dy, need_dx: bool, need_dw: bool, x_shape):
     """dgrad and wgrad of y = x2 @ w^T on the tcgen05 kernel (no transposed copies); the weight gradient accumulates straight
     into the flat gradient buffer when the parameter lives in one (returns dw = None then)."""
     dy2 = dy.reshape(-1, dy.shape[-1])
-    if dy2.stride(-1) != 1 or dy2.stride(0) % 8 != 0 or dy2.data_ptr() % 16 != 0:
-        dy2 = dy2.contiguous()
+    dy2 = tma_rows(dy2)
     dx = dw = None
     if need_dx:
         dx = gemm(dy2, w, b_mn=True).view(x_shape)                     # [T,N] x [N,K] -> [T,K]
@@ -112,8 +118,7 @@ class _GatedLinear(torch.autograd.Function):
     @staticmethod
     def forward(ctx, x, w, kind: int):
         x2 = x.reshape(-1, x.shape[-1])
-        if x2.stride(-1) != 1 or x2.stride(0) % 8 != 0 or x2.data_ptr() % 16 != 0:
-            x2 = x2.contiguous()
+        x2 = tma_rows(x2)
         need_raw = any(ctx.needs_input_grad[:2])
         res = lib().gemm_glu(x2, w, kind, need_raw, _sms(x.device))
         if need_raw:
