@@ -222,11 +222,16 @@ void sink_window_decode_attention(const Tensor& qkvg, Tensor out, const OptT& te
   if (qkvg.scalar_type() != at::kFloat && out.scalar_type() == qkvg.scalar_type() && (d == 64 || d == 128) && (dv == 64 || dv == 128) &&
       (rep == 1 || rep == 2 || rep == 3 || rep == 4 || rep == 6 || rep == 8) && qkvg.stride(0) % 8 == 0 &&
       reinterpret_cast<uintptr_t>(qkvg.data_ptr()) % 16 == 0) {
-    // enough CTAs for two per SM, at least 128 keys per split (the cache's row count bounds the visible keys).  Measured at 32 rows x
-    // 4 kv heads x 576 keys with a cold L2: 65 us with 3 splits + merge, 74 us as one split
-    const int64_t rows = kc.size(2);
-    int splits = (int)std::min<int64_t>(std::max<int64_t>(1, (2 * 148 + B * G - 1) / (B * G)), std::max<int64_t>(1, rows / 128));
-    splits = std::min(splits, 32);
+    // CTAs come in waves of about two per SM: of the split counts with at least 128 keys per split (the cache's row count bounds the
+    // visible keys), the one with the least work per wave slot, a split more costing a little (the merge)
+    const int64_t rows = kc.size(2), ctas = B * G;
+    const int64_t most = std::min<int64_t>(32, std::max<int64_t>(1, rows / 128));
+    int splits = 1;
+    double best = 1e30;
+    for (int64_t n = 1; n <= most; ++n) {
+      const double cost = (double)((ctas * n + 2 * 148 - 1) / (2 * 148)) / (double)n + 0.01 * (double)(n - 1);
+      if (cost < best) { best = cost; splits = (int)n; }
+    }
     Tensor pa, pm;
     if (splits > 1) {
       pa = at::empty({B, H, splits, dv}, qkvg.options().dtype(at::kFloat));

@@ -17,7 +17,7 @@ namespace {
 using rb::ld_any;
 using rb::st_any;
 
-constexpr int kThreads = 256;
+constexpr int kThreads = 256;      // of the shared-memory form
 
 struct BranchParams {
   void* res; int dtr;                       // [T, W] updated in place
@@ -29,7 +29,7 @@ struct BranchParams {
   int W; float eps;
 };
 
-// sums of two values over the CTA (one round); `red` holds >= 16 float2
+// sums of two values over the CTA (one round); `red` holds >= 32 float2
 RB_DEVICE float2 block_sum2(float x, float y, float2* red) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   x = rb::warp_sum(x);
@@ -37,7 +37,7 @@ RB_DEVICE float2 block_sum2(float x, float y, float2* red) {
   __syncthreads();
   if (lane == 0) red[warp] = make_float2(x, y);
   __syncthreads();
-  const float2 v = lane < kThreads / 32 ? red[lane] : make_float2(0.f, 0.f);
+  const float2 v = lane < (blockDim.x >> 5) ? red[lane] : make_float2(0.f, 0.f);
   return make_float2(rb::warp_sum(v.x), rb::warp_sum(v.y));
 }
 
@@ -45,9 +45,9 @@ RB_DEVICE float inv_rms(float ss, int W, float eps) { return 1.f / sqrtf(ss / (f
 RB_DEVICE float dot4(float4 v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); }
 RB_DEVICE float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 
-// NV float4 per thread: rows of up to NV * 1024 elements
-template <int NV>
-__global__ void __launch_bounds__(kThreads) branch_norm_reg_kernel(BranchParams p) {
+// NV float4 per thread, NT threads (many threads with few elements each keep more loads in flight than the reverse: four streams are read)
+template <int NV, int NT>
+__global__ void __launch_bounds__(NT) branch_norm_reg_kernel(BranchParams p) {
   __shared__ float2 red2[32];
   __shared__ float red[32];
   const int64_t t = blockIdx.x;
@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(kThreads) branch_norm_reg_kernel(BranchParams 
   float s1 = 0.f, s2 = 0.f;
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
-    const int e = (threadIdx.x + j * kThreads) * 4;
+    const int e = (threadIdx.x + j * NT) * 4;
     r[j] = m1[j] = m2[j] = f[j] = zero;
     if (e < W) {
       r[j] = rb::ld4_any(p.res, p.dtr, t * (int64_t)W + e);
@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(kThreads) branch_norm_reg_kernel(BranchParams 
   float ss = 0.f;
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
-    const int e = (threadIdx.x + j * kThreads) * 4;
+    const int e = (threadIdx.x + j * NT) * 4;
     if (e < W) {
       float4 u = m1[j], v = m2[j];
       if (p.w1 != nullptr) { const float4 w = rb::ld4_any(p.w1, p.dtw, e); u = make_float4(u.x * w.x, u.y * w.y, u.z * w.z, u.w * w.w); }
@@ -97,7 +97,7 @@ __global__ void __launch_bounds__(kThreads) branch_norm_reg_kernel(BranchParams 
   const float rs = inv_rms(rb::block_reduce<false>(ss, red), W, p.eps);
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
-    const int e = (threadIdx.x + j * kThreads) * 4;
+    const int e = (threadIdx.x + j * NT) * 4;
     if (e < W) {
       const float4 w = rb::ld4_any(p.w_next, p.dtw, e);
       rb::st4_any(p.out, p.dto, t * (int64_t)W + e, make_float4(r[j].x * rs * (w.x + p.w_off), r[j].y * rs * (w.y + p.w_off), r[j].z * rs * (w.z + p.w_off),
@@ -155,8 +155,10 @@ extern "C" int rb_branch_norm(void* res, int dtr, const void* y1, int64_t ld1, c
   const bool vec = W % 4 == 0 && W <= 8192 && al_ld(y1, ld1) && al_ld(y2, ld2) && al_ld(y3, ld3) && al16(res) && al16(y1) && al16(y2) && al16(y3) &&
                    al16(w1) && al16(w2) && al16(step) && al16(w_next) && al16(out);
   if (vec) {
-    auto kern = W <= 1024 ? branch_norm_reg_kernel<1> : W <= 2048 ? branch_norm_reg_kernel<2> : W <= 4096 ? branch_norm_reg_kernel<4> : branch_norm_reg_kernel<8>;
-    return rb::launch_pdl(kern, dim3((unsigned)T), dim3(kThreads), 0, s, p) == cudaSuccess ? 0 : 2;
+    auto kern = W <= 1024 ? branch_norm_reg_kernel<1, 256> : W <= 2048 ? branch_norm_reg_kernel<1, 512> : W <= 4096 ? branch_norm_reg_kernel<1, 1024>
+                                                                                                        : branch_norm_reg_kernel<2, 1024>;
+    const int nt = W <= 1024 ? 256 : W <= 2048 ? 512 : 1024;
+    return rb::launch_pdl(kern, dim3((unsigned)T), dim3(nt), 0, s, p) == cudaSuccess ? 0 : 2;
   }
   const size_t smem = (size_t)W * sizeof(float);
   if (smem > 160 * 1024) return -1;

@@ -517,6 +517,8 @@ template <int N, typename T> RB_DEVICE void f_store(T* p, const float* f) {
   }
 }
 
+template <int N> struct Int { static constexpr int value = N; };
+
 struct FastParams {
   DecodeParams d;
   float* part_acc;   // [B, H, splits, DV]
@@ -596,50 +598,77 @@ __global__ void __launch_bounds__(kFastThreads) sink_window_decode_fast_kernel(F
   }
   const float cap2 = p.softcap > 0.f ? 2.f / p.softcap : 0.f;
   const unsigned gmask = (LPR == 32) ? 0xffffffffu : (((1u << LPR) - 1u) << (rsel * LPR));
-  auto consume = [&](const float* kf, const float* vf, int idx) {
-    const int dist = n - pos_of(idx);
+  // bias of a key: lane r of the row's lanes loads head r's and puts it into its part of the dot product
+  auto bias_of = [&](int idx) { return p.bias != nullptr && sub < REP ? dist_bias(p.bias, p.n_bias, g * REP + sub, n - pos_of(idx)) : 0.f; };
+  // N keys at once (indices idx + u * stride): their scores first, then one maximum and one correction per head
+  auto consume = [&](auto n_keys, const auto& kf, const auto& vf, const float* bv, int idx, int stride) {
+    constexpr int N = decltype(n_keys)::value;
 #pragma unroll
     for (int r = 0; r < REP; ++r) {
-      float s = 0.f;
+      float s[N], mn = m[r];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) s = fmaf(q[r][i], kf[i], s);
+      for (int u = 0; u < N; ++u) {
+        s[u] = sub == r ? bv[u] : 0.f;
 #pragma unroll
-      for (int o = LPR / 2; o > 0; o >>= 1) s += __shfl_xor_sync(gmask, s, o, LPR);
-      if (p.softcap > 0.f) s = p.softcap - __fdividef(2.f * p.softcap, 1.f + __expf(fminf(s * cap2, 80.f)));   // cap tanh(s / cap)
-      s += dist_bias(p.bias, p.n_bias, g * REP + r, dist) - slope[r] * (float)dist;
-      const float mn = fmaxf(m[r], s);
-      const float corr = (m[r] == -INFINITY) ? 0.f : __expf(m[r] - mn), pr = __expf(s - mn);
-      l[r] = l[r] * corr + pr;
+        for (int i = 0; i < 8; ++i) s[u] = fmaf(q[r][i], kf[u][i], s[u]);
+      }
 #pragma unroll
-      for (int i = 0; i < VPL; ++i) acc[r][i] = fmaf(acc[r][i], corr, pr * vf[i]);
+      for (int o = LPR / 2; o > 0; o >>= 1)
+#pragma unroll
+        for (int u = 0; u < N; ++u) s[u] += __shfl_xor_sync(gmask, s[u], o, LPR);
+#pragma unroll
+      for (int u = 0; u < N; ++u) {
+        if (p.softcap > 0.f) s[u] = p.softcap - __fdividef(2.f * p.softcap, 1.f + __expf(fminf(s[u] * cap2, 80.f)));   // cap tanh(s / cap)
+        s[u] -= slope[r] * (float)(n - pos_of(idx + u * stride));
+        mn = fmaxf(mn, s[u]);
+      }
+      const float corr = (m[r] == -INFINITY) ? 0.f : __expf(m[r] - mn);
+      float sum = 0.f;
+#pragma unroll
+      for (int u = 0; u < N; ++u) { s[u] = __expf(s[u] - mn); sum += s[u]; }
+      l[r] = fmaf(l[r], corr, sum);
       m[r] = mn;
+#pragma unroll
+      for (int i = 0; i < VPL; ++i) {
+        float v = s[0] * vf[0][i];
+#pragma unroll
+        for (int u = 1; u < N; ++u) v = fmaf(s[u], vf[u][i], v);
+        acc[r][i] = fmaf(acc[r][i], corr, v);
+      }
     }
   };
   constexpr int UNROLL = REP * VPL >= 96 ? 2 : 4;      // (register budget)
   const int step = kFastWarps * RPW;
   int s0 = i0 + warp * RPW + rsel;
   for (; s0 + (UNROLL - 1) * step < i1; s0 += UNROLL * step) {
-    float kf[UNROLL][8], vf[UNROLL][kShared ? 1 : VPL];
+    float kf[UNROLL][8], vf[kShared ? 1 : UNROLL][VPL], bv[UNROLL];
 #pragma unroll
     for (int u = 0; u < UNROLL; ++u) {
       const int64_t rr = row_of(s0 + u * step);
       f_load<8>(kc + rr * HD + sub * 8, kf[u]);
       if constexpr (!kShared) f_load<VPL>(vc + rr * DV + sub * VPL, vf[u]);
+      bv[u] = bias_of(s0 + u * step);
     }
-#pragma unroll
-    for (int u = 0; u < UNROLL; ++u) consume(kf[u], kShared ? kf[u] : vf[u], s0 + u * step);
+    if constexpr (kShared) consume(Int<UNROLL>{}, kf, kf, bv, s0, step);
+    else consume(Int<UNROLL>{}, kf, vf, bv, s0, step);
   }
   for (; s0 < i1; s0 += step) {
-    float kf[8], vf[kShared ? 1 : VPL];
+    float kf[1][8], vf[1][VPL];
     const int64_t rr = row_of(s0);
-    f_load<8>(kc + rr * HD + sub * 8, kf);
-    if constexpr (!kShared) f_load<VPL>(vc + rr * DV + sub * VPL, vf);
-    consume(kf, kShared ? kf : vf, s0);
+    f_load<8>(kc + rr * HD + sub * 8, kf[0]);
+    if constexpr (!kShared) f_load<VPL>(vc + rr * DV + sub * VPL, vf[0]);
+    const float bv = bias_of(s0);
+    if constexpr (kShared) consume(Int<1>{}, kf, kf, &bv, s0, 0);
+    else consume(Int<1>{}, kf, vf, &bv, s0, 0);
   }
   if (split == fp.splits - 1 && warp == 0 && rsel == 0) {
+    float kf[1][8], vf[1][VPL];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) kn[i] = rb::to_f(rb::from_f<T>(kn[i]));
-    consume(kn, vn, nk - 1);
+    for (int i = 0; i < 8; ++i) kf[0][i] = rb::to_f(rb::from_f<T>(kn[i]));
+#pragma unroll
+    for (int i = 0; i < VPL; ++i) vf[0][i] = vn[i];
+    const float bv = bias_of(nk - 1);
+    consume(Int<1>{}, kf, vf, &bv, nk - 1, 0);
   }
   __syncwarp();
   __shared__ float sm_acc[kFastWarps][REP][DV];

@@ -9,6 +9,7 @@
 //                    the last rows - keep of the sequence) also go to their cache row (a row without a v section, whose values are its
 //                    keys, has one cache).  Step form: position lens[slot of row t]; the
 //                    decode kernel stores the row.
+//   cache_store      the same call without norm and rotation: the cache rows only
 //   turn_gate        attention output [T, H dv] in place: every head turned BACK by the position over its first `dims` columns (the
 //                    inverse of the values' rotation), then times sigmoid of a gate logit per head or per element.
 //
@@ -182,6 +183,29 @@ __global__ void __launch_bounds__(kThreads) window_prepare_kernel(PrepareParams 
     walk<V>(p.x, dt, base + nq + nk, p.G, p.dv, p.vdims, p.vinter, false, vcs, vsn, norm(nullptr, 1.f), emit(base + nq + nk, vc, p.dv));
 }
 
+// Nothing to turn or norm: only the cache rows are written.  A warp per token; tokens that leave no row end at once.
+template <int V>
+__global__ void __launch_bounds__(kThreads) cache_store_kernel(PrepareParams p, int64_t T) {
+  const int64_t t = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
+  rb::pdl_trigger();
+  rb::pdl_wait();
+  if (t >= T) return;
+  const int64_t slot = p.tok_slot[t];
+  const int n = p.pos[t], ring = max(p.rows - p.keep, 1);
+  if (slot < 0 || !(n < p.keep || p.remain[t] < p.rows - p.keep)) return;
+  const int row = n < p.keep ? n : p.keep + (n - p.keep) % ring;
+  auto copy = [&](int64_t b0, void* cache, int hd) {
+    for (int e = (threadIdx.x & 31) * V; e < p.G * hd; e += 32 * V) {
+      float a[V];
+      ldn<V>(p.x, p.dt, b0 + e, a);
+      stn<V>(cache, p.dt, ((slot * p.G + e / hd) * p.rows + row) * hd + e % hd, a);
+    }
+  };
+  const int64_t k0 = t * p.ld + (int64_t)p.H * p.d;
+  copy(k0, p.kc, p.d);
+  if (p.vc != nullptr) copy(k0 + (int64_t)p.G * p.d, p.vc, p.dv);
+}
+
 template <int V>
 __global__ void __launch_bounds__(kThreads) turn_gate_kernel(void* __restrict__ x, int dt, const void* __restrict__ gate, int64_t gld, int gmode,
                                                              const float* __restrict__ freq, const int* __restrict__ pos, const int* __restrict__ lens,
@@ -221,6 +245,12 @@ extern "C" int rb_window_prepare(void* x, int64_t ld, int dt, const void* wq, co
   if ((wq == nullptr) != (wk == nullptr) || (kc == nullptr && vc != nullptr)) return -1;
   PrepareParams p{x, ld, dt, wq, wk, freq, vfreq, pos, lens, slots, tok_slot, remain, kc, vc, H, G, d, dv, dims, inter, vdims, vinter, keep, rows, eps, mscale};
   const bool vec = d % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && rot_vec(dims, inter) && rot_vec(vdims, vinter) && al16(x) && al16(kc) && al16(vc);
+  if (wq == nullptr && dims == 0 && vdims == 0) {
+    if (kc == nullptr) return 0;
+    const bool v4 = d % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && al16(x) && al16(kc) && al16(vc);
+    return rb::launch_pdl(v4 ? cache_store_kernel<4> : cache_store_kernel<1>, dim3((unsigned)((T + kThreads / 32 - 1) / (kThreads / 32))), dim3(kThreads), 0, s,
+                          p, T) == cudaSuccess ? 0 : 2;
+  }
   return rb::launch_pdl(vec ? window_prepare_kernel<4> : window_prepare_kernel<1>, dim3((unsigned)T), dim3(kThreads), 0, s, p) == cudaSuccess ? 0 : 2;
 }
 
