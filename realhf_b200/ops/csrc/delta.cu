@@ -36,10 +36,11 @@ struct GateParams {
   int N;
 };
 
-RB_DEVICE float decay_of(const GateParams& gp, int dt, int64_t t, int i, int h) {
+// decay of input i; rate = exp(A_log) of its head
+RB_DEVICE float decay_of(const GateParams& gp, int dt, int64_t t, int i, float rate) {
   const float a = ld_any(gp.a, dt, t * gp.lda + i) + ld_any(gp.dt_bias, dt, i);
   const float sp = a > 20.f ? a : log1pf(expf(a));
-  return expf(-expf(ld_any(gp.A_log, dt, h)) * sp);
+  return expf(-rate * sp);
 }
 
 // Gate units of the prepare kernels (grid.y from 2 G + H on): the first one writes the strengths, and the decays when there is one
@@ -51,15 +52,16 @@ RB_DEVICE void gate_unit(const GateParams& gp, float* u, int dt, int unit, int64
       const int64_t t = t0 + idx / H;
       const int h = idx % H;
       u[t * UW + C + h] = 1.f / (1.f + expf(-ld_any(gp.b, dt, t * gp.ldb + h)));
-      if (per == 1) u[t * UW + C + H + h] = decay_of(gp, dt, t, h, h);
+      if (per == 1) u[t * UW + C + H + h] = decay_of(gp, dt, t, h, expf(ld_any(gp.A_log, dt, h)));
     }
     return;
   }
   const int h = unit - 1;
+  const float rate = expf(ld_any(gp.A_log, dt, h));
   for (int idx = threadIdx.x; idx < nt * per; idx += blockDim.x) {
     const int64_t t = t0 + idx / per;
     const int i = h * per + idx % per;
-    u[t * UW + C + H + i] = decay_of(gp, dt, t, i, h);
+    u[t * UW + C + H + i] = decay_of(gp, dt, t, i, rate);
   }
 }
 
