@@ -202,7 +202,7 @@ TC_SHAPES = {
     "shared-64-no-window-short-bias": lambda: par(heads=2, kv_heads=2, dim=64, window=None, rows=8, bias_max=16),
     "shared-128-rep6": lambda: par(heads=6, kv_heads=1, dim=128, window=200, rows=24, bias_max=150),
     "64-64": lambda: par2(heads=4, kv_heads=2, dim=64, vdim=64, dims=64),
-    "64-128": lambda: par2(heads=6, kv_heads=1, dim=64, vdim=128, dims=24),
+    "64-128-rep6": lambda: par2(heads=12, kv_heads=2, dim=64, vdim=128, dims=24),
     "64-128-rep8": lambda: par2(heads=8, kv_heads=1, dim=64, vdim=128, dims=16),
     "128-64": lambda: par2(heads=3, kv_heads=1, dim=128, vdim=64, dims=128, scaling=False),
     "128-128-rep12": lambda: par2(heads=12, kv_heads=1, dim=128, vdim=128, dims=32),
@@ -459,7 +459,7 @@ def test_rotation_with_a_factor_at_far_positions(device, dtype):
     pos = torch.tensor([0, 1, 2, 63, 64, 500, 2999], dtype=torch.int32)
     lens = torch.tensor([5, 2999, 64], dtype=torch.int32)
     slots = torch.tensor([1, 2, 1, 0, 2, 2, 0], dtype=torch.int32)
-    for H, G, d, dv, dims in ((3, 1, 12, 8, 8), (2, 2, 10, 6, 10), (4, 2, 64, 128, 16)):
+    for H, G, d, dv, dims in ((3, 1, 12, 8, 8), (2, 2, 10, 6, 10), (4, 2, 64, 128, 32)):
         rot = dict(base=700.0, dims=dims, scaling=dict(factor=8.0, fast=16.0, original=128, slow=2.0))
         a = WindowAttentionConfig(n_heads=H, n_kv_heads=G, qk_dim=d, v_dim=dv, scale=1.0, qkv_bias=False, value_norm=False, head_temp=False, slope_base=None,
                                   sink=False, out_gate=False,
